@@ -8,6 +8,8 @@ group has its own pool of pages and its own block table per request:
   * a windowed group (window w) gives a page back as soon as every key in it is
     out of reach of all future queries; the table keeps a -1 in its place so
     that logical page i still sits at index i;
+  * a chunked group (chunk c: a query sees the keys of its own run of c positions) gives back
+    the pages of every chunk that has ended, in the same way;
   * a fixed-state group holds no pages: the request's *state slot* indexes a
     fixed-size record per layer.  The slot pool exists even when no layer asks
     for state, and is taken and returned with the pages.
@@ -22,6 +24,7 @@ device here).  Prefix matching, swap and offload are not part of this engine.
 
 from __future__ import annotations
 
+import math
 from collections import deque
 from dataclasses import dataclass
 from typing import Callable, Dict, List, Optional, Sequence, Tuple
@@ -32,7 +35,8 @@ from typing import Callable, Dict, List, Optional, Sequence, Tuple
 class PagedKVRequest:
     """Keys and values of ``num_kv_heads`` x ``head_dim`` per token, paged.
     ``window`` None: all earlier tokens stay readable; else only the last
-    ``window`` positions (the current one included).  ``tied_values``: the values are
+    ``window`` positions (the current one included).  ``chunk``: only the positions of the
+    query's own chunk, p with p // chunk == query // chunk, stay readable.  ``tied_values``: the values are
     the keys themselves (or a prefix of every key row), so only keys are stored
     (``LayerCache.v`` is ``LayerCache.k``).  ``value_dim``: the size of a value row where it
     differs from the keys' ``head_dim`` (None: the same)."""
@@ -41,6 +45,7 @@ class PagedKVRequest:
     window: Optional[int] = None
     tied_values: bool = False
     value_dim: Optional[int] = None
+    chunk: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -67,6 +72,13 @@ def state_part(request) -> Optional[FixedStateRequest]:
     return next((r for r in request_parts(request) if isinstance(r, FixedStateRequest)), None)
 
 
+def record_floats(request) -> int:
+    """Floats of a request's fixed-size record, rounded up to 4 (so that records laid side by side in
+    a larger one start on 16-byte boundaries)."""
+    st = state_part(request)
+    return 0 if st is None else -(-math.prod(st.shape) // 4) * 4
+
+
 class CacheError(RuntimeError):
     pass
 
@@ -75,12 +87,16 @@ class CacheError(RuntimeError):
 class PagePool:
     """Pages of one layer group and the block tables that point into them."""
 
-    def __init__(self, num_pages: int, page_size: int, window: Optional[int] = None):
+    def __init__(self, num_pages: int, page_size: int, window: Optional[int] = None,
+                 chunk: Optional[int] = None):
         if num_pages < 1 or page_size < 1:
             raise ValueError("num_pages and page_size must be >= 1")
+        if window is not None and chunk is not None:
+            raise ValueError("a group has a window or a chunk, not both")
         self.num_pages = num_pages
         self.page_size = page_size
         self.window = window
+        self.chunk = chunk
         self.free: deque = deque(range(num_pages))
         self.tables: Dict[str, List[int]] = {}
         self._first_live: Dict[str, int] = {}
@@ -102,9 +118,18 @@ class PagePool:
         """Most pages a request of ``total_tokens`` can hold at once when fed in
         portions of at most ``max_portion`` tokens."""
         full = self.pages_for(total_tokens)
-        if self.window is None:
+        reach = self.window if self.window is not None else self.chunk
+        if reach is None:
             return full
-        return min(full, self.pages_for(self.window + max_portion) + 1)
+        return min(full, self.pages_for(reach + max_portion) + 1)
+
+    def first_needed(self, next_position: int) -> int:
+        """The earliest position that a query at a position >= ``next_position`` can read."""
+        if self.window is not None:
+            return max(0, next_position - self.window + 1)
+        if self.chunk is not None:
+            return next_position - next_position % self.chunk
+        return 0
 
     def open(self, req: str) -> None:
         if req in self.tables:
@@ -129,12 +154,10 @@ class PagePool:
 
     def trim(self, req: str, next_position: int) -> List[int]:
         """Give back pages no query at position >= ``next_position`` can read."""
-        if self.window is None:
+        if self.window is None and self.chunk is None:
             return []
         table = self.tables[req]
-        # keys needed: r >= next_position - window + 1
-        dead_pages = max(0, (next_position - self.window + 1) // self.page_size)
-        dead_pages = min(dead_pages, len(table))
+        dead_pages = min(self.first_needed(next_position) // self.page_size, len(table))
         freed = []
         for lp in range(self._first_live[req], dead_pages):
             if table[lp] >= 0:
@@ -201,13 +224,17 @@ class CacheManager:
     trimmed and released across every group at once (all or nothing)."""
 
     def __init__(self, group_windows: Sequence[Optional[int]], num_pages, page_size: int,
-                 num_state_slots: int, reserve_pages: int = 0):
+                 num_state_slots: int, reserve_pages: int = 0,
+                 group_chunks: Optional[Sequence[Optional[int]]] = None):
         if isinstance(num_pages, int):
             num_pages = [num_pages] * len(group_windows)
         if len(num_pages) != len(group_windows):
             raise ValueError("one page count per group is needed")
         self.page_size = page_size
-        self.pools = [PagePool(n, page_size, w) for n, w in zip(num_pages, group_windows)]
+        chunks = list(group_chunks) if group_chunks is not None else [None] * len(group_windows)
+        if len(chunks) != len(group_windows):
+            raise ValueError("one chunk size (or None) per group is needed")
+        self.pools = [PagePool(n, page_size, w, c) for n, w, c in zip(num_pages, group_windows, chunks)]
         self.slots = StateSlotPool(num_state_slots)
         self.reserve_pages = reserve_pages
         self.alloc_fails = 0

@@ -1,7 +1,7 @@
 """Device memory of the cache: pages per layer group, state records per layer.
 
 ``plan_groups`` sorts the cache requests of the run order's entries into groups:
-paged requests with equal (kv heads, head size, window) share a group (one page
+paged requests with equal (kv heads, head size, window or chunk) share a group (one page
 pool, one block table per request); runs that read an earlier run's cache own
 nothing; a mixer may ask for pages and a fixed-size state record at once, and a paged
 request with tied values stores keys only.  "layer" below means an entry of the run order.  Page
@@ -121,6 +121,10 @@ class CacheStorage:
     @property
     def group_windows(self) -> List[Optional[int]]:
         return [g.request.window for g in self.groups]
+
+    @property
+    def group_chunks(self) -> List[Optional[int]]:
+        return [g.request.chunk for g in self.groups]
 
     def clear_state_slots(self, slots: Sequence[int]) -> None:
         """Zero the state records of freshly taken slots (before their first step)."""

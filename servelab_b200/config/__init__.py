@@ -5,13 +5,15 @@ from .daferax import DaferaxConfig
 from .dezelorn import DezelornConfig
 from .qwen2 import ConfigError, Qwen2Config
 from .sumolorn import SumolornConfig
+from .vufadra import VufadraConfig
 from .zimupel import ZimupelConfig
 from .registry import (config_from_dict, load_config, model_spec_from_config,
                        register_architecture, registered_architectures,
                        resolve_architecture)
-from .specs import (AttentionSpec, BlockSpec, ConvTalkAttentionSpec, DecayAttentionSpec,
-                    DifferentialAttentionSpec, DynamicTanhSpec, GatedMLPSpec,
-                    LatentAttentionSpec, LayerNormSpec, LayerRun, ModelSpec, NoPositionSpec,
+from .specs import (AttentionSpec, BigramSpec, BlockSpec, ConvTalkAttentionSpec, DecayAttentionSpec,
+                    DeltaRuleSpec, DifferentialAttentionSpec, DynamicTanhSpec, GatedMLPSpec,
+                    GatedRecurrenceSpec, LatentAttentionSpec, LayerNormSpec, LayerRun, LoopEntrySpec,
+                    ModelSpec, NoPositionSpec,
                     NormedAttentionSpec, PairRotarySpec, ParallelMixersSpec, PartSpec, RMSNormSpec,
                     RotarySpec, RoutedExpertsSpec)
 
@@ -20,14 +22,18 @@ register_architecture(DezelornConfig.architecture, DezelornConfig, model_type=De
 register_architecture(DaferaxConfig.architecture, DaferaxConfig, model_type=DaferaxConfig.model_type)
 register_architecture(ZimupelConfig.architecture, ZimupelConfig, model_type=ZimupelConfig.model_type)
 register_architecture(SumolornConfig.architecture, SumolornConfig, model_type=SumolornConfig.model_type)
+register_architecture(VufadraConfig.architecture, VufadraConfig, model_type=VufadraConfig.model_type)
 
 __all__ = [
-    "AttentionSpec", "BlockSpec", "CacheConfig", "ConfigError", "ConvTalkAttentionSpec",
-    "DaferaxConfig", "DecayAttentionSpec", "DezelornConfig", "DifferentialAttentionSpec", "DynamicTanhSpec",
+    "AttentionSpec", "BigramSpec", "BlockSpec", "CacheConfig", "ConfigError", "ConvTalkAttentionSpec",
+    "DaferaxConfig", "DecayAttentionSpec", "DeltaRuleSpec", "DezelornConfig", "DifferentialAttentionSpec",
+    "DynamicTanhSpec",
     "EngineConfig",
-    "GatedMLPSpec", "LatentAttentionSpec", "LayerNormSpec", "LayerRun", "ModelSpec", "NoPositionSpec",
+    "GatedMLPSpec", "GatedRecurrenceSpec", "LatentAttentionSpec", "LayerNormSpec", "LayerRun", "LoopEntrySpec",
+    "ModelSpec", "NoPositionSpec",
     "NormedAttentionSpec", "PairRotarySpec", "ParallelMixersSpec", "PartSpec",
-    "Qwen2Config", "RMSNormSpec", "RotarySpec", "RoutedExpertsSpec", "SchedulerConfig", "SumolornConfig", "ZimupelConfig",
+    "Qwen2Config", "RMSNormSpec", "RotarySpec", "RoutedExpertsSpec", "SchedulerConfig", "SumolornConfig",
+    "VufadraConfig", "ZimupelConfig",
     "config_from_dict", "load_config", "model_spec_from_config",
     "register_architecture", "registered_architectures", "resolve_architecture",
 ]

@@ -44,6 +44,12 @@ class RotarySpec(PartSpec):
     stretch_high: float = 4.0
     stretch_original: float = 8192.0
     precise: bool = False      # the frequencies are formed in float64 and rounded to float32 once
+    # Interpolation by a ramp over the pairs and a factor on cos and sin, as ``PairRotarySpec``
+    # describes it (None: none).
+    yarn_factor: Optional[float] = None
+    yarn_original: float = 0.0
+    yarn_fast: float = 32.0
+    yarn_slow: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -200,7 +206,12 @@ class NormedAttentionSpec(PartSpec):
                      the mixed values being what the cache holds.  ``value_mix_key`` names the
                      source among the layers of a model;
     ``head_gate``    head h's result is multiplied by sigmoid((W_g x)_h), one number a head;
-    ``window``       None: every earlier key; else the last ``window`` keys (own included).
+    ``window``       None: every earlier key; else the last ``window`` keys (own included);
+    ``chunk``        None, or: a query at position i sees the keys j <= i of its own chunk,
+                     j // chunk == i // chunk (not together with a window);
+    ``weight_fn``    "softmax", or "sigmoid": the weight of a visible key is sigmoid(score) and
+                     the weights are not normalized (no soft cap, sink or gate with it);
+    ``score_bias``   (sigmoid) a learned number a head added to the scaled score.
     """
     kind: str = "normed_attention"
     hidden_size: int = 0
@@ -230,6 +241,10 @@ class NormedAttentionSpec(PartSpec):
     value_mix_name: str = "vmix"
     conv_suffix: str = ".conv"             # the taps of a projection: <projection><conv_suffix>
     sink_name: str = "sink"
+    chunk: Optional[int] = None
+    weight_fn: str = "softmax"
+    score_bias: bool = False
+    score_bias_name: str = "pb"
 
 
 @dataclass(frozen=True)
@@ -292,6 +307,14 @@ class DecayAttentionSpec(PartSpec):
     S_t = diag(alpha_t) S_{t-1} + k_t v_t^T.  ``query_scale``: a factor on the queries (None: 1).
     ``out_norm_per_head``: with ``out_norm`` "head" and a weight, the weight has ``value_dim``
     elements and is shared by the heads.
+
+    ``decay_gate_kind`` "exp_exp": the learned decay is exp(-exp(z)) instead (no tau).
+    ``decay_gate_tanh``: a tanh inside the bottleneck, z = W_a2 tanh(W_a1 x) + b.
+    ``bonus``: the current token enters its own result with a learned factor per head and key
+    channel instead of through the state, o_t = (S_{t-1} + diag(bonus) k_t v_t^T)^T q_t.
+    ``token_mix``: each of q, k, v, gate and the decay reads its own mix h + (h' - h) * mu of the
+    token's input h and the previous token's h' (zeros for a sequence's first), with a learned
+    vector mu for each; the previous input is per-request state.
     """
     kind: str = "decay_attention"
     hidden_size: int = 0
@@ -319,6 +342,73 @@ class DecayAttentionSpec(PartSpec):
     decay_down_name: str = "a1"
     decay_up_name: str = "a2"
     decay_bias_name: str = "a2.b"
+    decay_gate_kind: str = "sigmoid_root"
+    decay_gate_tanh: bool = False
+    bonus: bool = False
+    bonus_name: str = "u"
+    token_mix: bool = False
+    # the mixing vectors of q, k, v, the gate and the decay
+    token_mix_names: Tuple[str, ...] = ("mu.r", "mu.k", "mu.v", "mu.g", "mu.w")
+
+
+@dataclass(frozen=True)
+class DeltaRuleSpec(PartSpec):
+    """Linear attention whose per-request state forgets by channel and unlearns along the key: with
+    the unit key u = k / sqrt(sum k^2 + ``unit_eps``) of a head,
+
+        S_t = diag(w_t) S_{t-1} - (a_t u_t) (u_t^T S_{t-1}) + k_t v_t^T,    o_t = S_t^T r_t
+
+    (both terms read the old state), decays w = exp(-``decay_coef`` sigmoid(W_w2 tanh(W_w1 x) + b))
+    through a bottleneck of ``decay_rank`` elements (-1: the checkpoint's tensor decides) and removal
+    rates a = sigmoid(W_a x + b_a), both per head and key channel.  Every head's result is divided by
+    its root mean square (``out_norm_eps``); the row is multiplied by a learned weight and by
+    sigmoid(W_g x) before the output projection.  S: ``head_dim`` x ``value_dim`` float32 a head."""
+    kind: str = "delta_rule"
+    hidden_size: int = 0
+    num_heads: int = 0
+    head_dim: int = 0
+    value_dim: int = 0
+    decay_coef: float = 1.0
+    decay_rank: int = -1
+    unit_eps: float = 1e-6
+    out_norm_eps: float = 1e-6
+    r_name: str = "r"
+    k_name: str = "k"
+    v_name: str = "v"
+    gate_name: str = "g"
+    o_name: str = "o"
+    removal_name: str = "a"
+    removal_bias_name: str = "a.b"
+    decay_down_name: str = "w1"
+    decay_up_name: str = "w2"
+    decay_bias_name: str = "w0"
+    out_norm_name: str = "norm"
+
+
+@dataclass(frozen=True)
+class GatedRecurrenceSpec(PartSpec):
+    """A recurrent block of two branches of ``width`` channels: y = gelu_tanh(W_y x + b_y), and
+    u = a causal convolution per channel (``conv_taps``, bias) of W_x x + b_x.  With ``blocks`` equal
+    parts of the channels, r = sigmoid(ra[b] u_b + ra_b[b]) and i = sigmoid(ri[b] u_b + ri_b[b]),
+
+        log a = -``decay_coef`` r softplus(lambda),   S_t = a S_{t-1} + sqrt(1 - a^2) i u,
+
+    S = 0 before a sequence's first token; the result is W_o (S y).  Per-request state: S and the
+    convolution's last ``conv_taps`` - 1 inputs, float32."""
+    kind: str = "gated_recurrence"
+    hidden_size: int = 0
+    width: int = 0
+    blocks: int = 1
+    conv_taps: int = 1
+    decay_coef: float = 8.0
+    y_name: str = "y"
+    x_name: str = "x"
+    conv_name: str = "conv"
+    r_name: str = "ra"
+    i_name: str = "ri"
+    lambda_name: str = "lam"
+    o_name: str = "o"
+    bias_suffix: str = ".b"
 
 
 @dataclass(frozen=True)
@@ -435,7 +525,11 @@ class BlockSpec(PartSpec):
     ``hyper_connections`` keeps ``streams`` copies of the residual: a sublayer reads
     u = sum_s in[s] x_s, and x_t <- sum_s mix[s, t] x_s + out[t] f(norm(u)) for all streams at once
     (tensors ``<layer>.<mixer_hyper_name>.{in,out,mix}`` and the same for the feed-forward, which
-    may be None)."""
+    may be None).
+    ``parallel_norm`` runs both sublayers on the same stream, each behind a norm of its own:
+    x += mixer(norm1(x)) + ff(norm2(x)) (``feed_forward`` None: the mixer alone); with
+    ``token_shift`` the mixer's input h becomes h + (h' - h) * shift, h' the previous token's h
+    before this (zeros for a sequence's first), which is per-request state of the block."""
     kind: str = "pre_norm"
     mixer: PartSpec = None
     feed_forward: PartSpec = None
@@ -453,6 +547,8 @@ class BlockSpec(PartSpec):
     streams: int = 1                       # (hyper_connections)
     mixer_hyper_name: str = "hc1"
     ff_hyper_name: str = "hc2"
+    token_shift: bool = False              # (parallel_norm)
+    shift_name: str = "shift"
 
 
 @dataclass(frozen=True)
@@ -465,9 +561,34 @@ class LayerRun:
     ``cache_of``   index of an EARLIER RUN whose cache this run reads instead of
                    owning one: such a run writes no keys, values or state.  None
                    means the run owns (and fills) its cache.
+    ``loop_entry`` None, or the number t of the pass of a loop that begins with this
+                   run: the stream is first replaced by W_in [x; x0] + step_t
+                   (``ModelSpec.loop``).
     """
     layer: int
     cache_of: Optional[int] = None
+    loop_entry: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class BigramSpec:
+    """A second embedding, added to the token's: row (previous * ``mul_prev`` + token * ``mul_cur``)
+    mod ``buckets`` of a table of ``buckets`` + 1 rows, whose last row serves a sequence's first
+    token.  The previous token is per-request state."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+    name: str = "bigram"
+
+
+@dataclass(frozen=True)
+class LoopEntrySpec:
+    """What happens to the stream where a pass of a loop begins: x <- W_in [x; x0] + step_t, with
+    x0 the embedding output and t the number of the pass (tensors ``in_name`` [w, 2 w] and
+    ``step_name`` [``times``, w])."""
+    times: int
+    in_name: str = "loop.in"
+    step_name: str = "loop.step"
 
 
 @dataclass(frozen=True)
@@ -500,5 +621,7 @@ class ModelSpec:
     # a number: the residual is kept as that many streams [tokens, streams, hidden], all equal to the
     # embedding at the start and summed before the final norm (blocks of kind hyper_connections)
     residual_streams: Optional[int] = None
+    bigram: Optional[BigramSpec] = None
+    loop: Optional[LoopEntrySpec] = None         # (runs with a ``loop_entry``)
     logit_scale: Optional[float] = None          # logits are multiplied by it ...
     logit_softcap: Optional[float] = None        # ... and then become cap * tanh(logits / cap)

@@ -15,6 +15,10 @@
 // and a sink, one number a head whose exponential is added to the softmax's denominator once (it
 // has no key and no value and is neither scaled nor capped).
 //
+// Instead of the softmax (`sig_bias`, one number a head): the weight of a visible key is
+// sigmoid(s + sig_bias_h) and the weights are not normalized.  Instead of the window (`chunk` > 0): a query
+// at position i sees the keys j <= i with j / chunk == i / chunk.
+//
 // Several attention maps a head (`maps`, the differential form): every query head and every kv
 // head carries `maps` query / key vectors side by side ([head][map][Dk], key rows `ldk` apart),
 // each map is an attention of its own over the kv head's one set of values, and the results are
@@ -45,7 +49,8 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
     const int* __restrict__ cu_q, const int* __restrict__ ctx_len,
     const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
     int H, int Hkv, int Dk, int Dv, int ps, int num_pages, float scale, int window,
-    const T* __restrict__ gate, int ldg, float softcap, const float* __restrict__ sink) {
+    const T* __restrict__ gate, int ldg, float softcap, const float* __restrict__ sink, int chunk,
+    const float* __restrict__ sig_bias) {
     extern __shared__ float ak_smem[];
     pdl_wait();
     const int ldq_s = Dk + 1;
@@ -84,6 +89,10 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
     const int p_last = pos_base + (row0 + nrows - 1) / g;
     int kbeg = 0;
     if (window > 0) kbeg = max(0, p_first - window + 1) / AK_BN * AK_BN;
+    if (chunk > 0) kbeg = p_first / chunk * chunk / AK_BN * AK_BN;
+    // the first key of this thread's row, and what its head adds to a score
+    const int my_first = window > 0 ? my_pos - window + 1 : chunk > 0 && my_pos >= 0 ? my_pos - my_pos % chunk : 0;
+    const float my_bias = sig_bias != nullptr && row_valid ? sig_bias[kvh * g + (row0 + r) % g] : 0.f;
     const int kend = p_last + 1;
     const int nvc = (Dv + AK_DC - 1) / AK_DC;
 
@@ -134,7 +143,7 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int kp = k0 + c0 + 8 * j;
-            const bool vis = row_valid && kp <= my_pos && (window <= 0 || my_pos - kp < window);
+            const bool vis = row_valid && kp <= my_pos && kp >= my_first;
             float sv = sc[j] * scale;
             if (softcap > 0.f) sv = softcap * tanhf(sv / softcap);
             sc[j] = vis ? sv : -INFINITY;
@@ -146,7 +155,11 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
         const float m_new = fmaxf(m, tmax);
         float alpha = 1.f, psum = 0.f;
         float p[4] = {0.f, 0.f, 0.f, 0.f};
-        if (m_new != -INFINITY) {
+        if (sig_bias != nullptr) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                p[j] = (sc[j] == -INFINITY) ? 0.f : 1.0f / (1.0f + expf(-(sc[j] + my_bias)));
+        } else if (m_new != -INFINITY) {
             alpha = (m == -INFINITY) ? 0.f : expf(m - m_new);
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
@@ -195,6 +208,7 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
         const int head = (kvh * g + hg) * maps + map;
         if (sink != nullptr) l += (m == -INFINITY) ? 1.f : expf(sink[head] - m);
         float inv = l > 0.f ? 1.0f / l : 0.f;
+        if (sig_bias != nullptr) inv = 1.0f;
         if (gate != nullptr) {
             const float z = to_float(gate[(size_t)(q0 + tl) * ldg + head]);
             inv *= 1.0f / (1.0f + expf(-z));
@@ -216,8 +230,10 @@ static int launch_attention_kv(const T* q, int ldq, const T* kc, int ldk, int ma
                                const int* ctx_len, const int* tile_seq, const int* tile_row0,
                                int num_tiles, int H, int Hkv, int Dk, int Dv, int ps, int num_pages,
                                float scale, int window, const T* gate, int ldg, float softcap,
-                               const float* sink, cudaStream_t st) {
+                               const float* sink, cudaStream_t st, int chunk = 0, const float* sig_bias = nullptr) {
     if (num_tiles <= 0) return 0;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sig_bias != nullptr && (sink != nullptr || maps != 1)))
+        return SLB_ERR_BAD_ARG;
     if (softcap < 0.f || (sink != nullptr && maps != 1)) return SLB_ERR_BAD_ARG;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dv <= 0 || ps <= 0 || max_pages <= 0 ||
         num_pages <= 0 || ldv < Dv || maps <= 0 || ldk < maps * Dk)
@@ -231,7 +247,7 @@ static int launch_attention_kv(const T* q, int ldq, const T* kc, int ldk, int ma
     if (rc != 0) return rc;
     return slb_launch(attention_kv_kernel<T, TO>, dim3(num_tiles, Hkv * maps), dim3(AK_THREADS), smem, st, q, ldq,
                       kc, ldk, maps, vc, ldv, out, ldo, block_table, max_pages, cu_q, ctx_len, tile_seq, tile_row0,
-                      H, Hkv, Dk, Dv, ps, num_pages, scale, window, gate, ldg, softcap, sink);
+                      H, Hkv, Dk, Dv, ps, num_pages, scale, window, gate, ldg, softcap, sink, chunk, sig_bias);
 }
 
 extern "C" {
@@ -240,19 +256,21 @@ int slb_attention_kv_f32(const float* q, int ldq, const float* kc, const float* 
                          int ldo, const int* block_table, int max_pages, const int* cu_q,
                          const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                          int H, int Hkv, int Dk, int Dv, int ps, int num_pages, float scale, int window,
-                         const float* gate, int ldg, float softcap, const float* sink, cudaStream_t st) {
+                         const float* gate, int ldg, float softcap, const float* sink, int chunk,
+                         const float* sig_bias, cudaStream_t st) {
     return launch_attention_kv<float, float>(q, ldq, kc, Dk, 1, vc, ldv, out, ldo, block_table, max_pages, cu_q,
                                       ctx_len, tile_seq, tile_row0, num_tiles, H, Hkv, Dk, Dv, ps,
-                                      num_pages, scale, window, gate, ldg, softcap, sink, st);
+                                      num_pages, scale, window, gate, ldg, softcap, sink, st, chunk, sig_bias);
 }
 int slb_attention_kv_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int ldv, bf16* out,
                           int ldo, const int* block_table, int max_pages, const int* cu_q,
                           const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                           int H, int Hkv, int Dk, int Dv, int ps, int num_pages, float scale, int window,
-                          const bf16* gate, int ldg, float softcap, const float* sink, cudaStream_t st) {
+                         const bf16* gate, int ldg, float softcap, const float* sink, int chunk,
+                         const float* sig_bias, cudaStream_t st) {
     return launch_attention_kv<bf16, bf16>(q, ldq, kc, Dk, 1, vc, ldv, out, ldo, block_table, max_pages, cu_q,
                                      ctx_len, tile_seq, tile_row0, num_tiles, H, Hkv, Dk, Dv, ps,
-                                     num_pages, scale, window, gate, ldg, softcap, sink, st);
+                                     num_pages, scale, window, gate, ldg, softcap, sink, st, chunk, sig_bias);
 }
 // several maps a head (see the top of the file); the results are float32 in both forms
 int slb_attention_kv_maps_f32(const float* q, int ldq, const float* kc, int ldk, int maps, const float* vc, int ldv,

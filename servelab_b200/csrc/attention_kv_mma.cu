@@ -23,6 +23,10 @@
 // long product of a tile is spread over the warps; the Q tile takes 16 rows of shared memory, so
 // that two blocks fit an SM at the largest sizes.
 //
+// Instead of the softmax (`sig_bias`, one number a head): a visible key's weight is sigmoid(score +
+// sig_bias_h), the weights are not normalized, and key splits simply add up.  Instead of the window
+// (`chunk` > 0): a query at position i sees the keys j <= i with j / chunk == i / chunk.
+//
 // Several attention maps a head (`maps`; not with `tied`): every query head and every kv head
 // carries `maps` query / key vectors side by side ([head][map][DK]; a cached key row is
 // [map][DK]), each map is an attention of its own over the kv head's one set of values, and a
@@ -97,7 +101,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
     const int* __restrict__ tile_row0, int H, int Hkv, int ps, int num_pages, float scale_log2,
     int window, const bf16* __restrict__ gate, int ldg, int splits, float* __restrict__ part_o,
     float* __restrict__ part_ml, int maps, float* __restrict__ out_f32, int q_rows, int fold,
-    float softcap, float scale, const float* __restrict__ sink) {
+    float softcap, float scale, const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias) {
     // softcap > 0: a scaled score s becomes softcap tanh(s / softcap); sink: one number a head whose
     // exponential joins the softmax's denominator (added where the row is finished: here without
     // key splits, in the combine kernel with them)
@@ -144,6 +148,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
     const int p_last = pos_base + (row0 + nrows - 1) / g;
     int kbeg = 0;
     if (window > 0) kbeg = max(0, p_first - window + 1) / BN * BN;
+    if (chunk > 0) kbeg = p_first / chunk * chunk / BN * BN;
     const int kend = p_last + 1;
     int ntiles = (kend - kbeg + BN - 1) / BN;
     if (splits > 1) {                                      // this block's share of the key tiles
@@ -165,6 +170,16 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
     const int warp_pos_max = wrow * 16 < nrows ? pos_base + (row0 + wr_last) / g : -1;
     const int warp_pos_min = pos_base + (row0 + wrow * 16) / g;
     const int tig = lane & 3;
+    // the first key each of the two rows sees (and the warp's lowest row), and what a head adds to a score
+    auto first_key = [&](int pos) {
+        return window > 0 ? pos - window + 1 : chunk > 0 && pos >= 0 ? pos - pos % chunk : 0;
+    };
+    const int first_lo = first_key(pos_lo), first_hi = first_key(pos_hi), warp_first = first_key(warp_pos_min);
+    float bias2[2] = {0.f, 0.f};
+    if (sig_bias != nullptr) {
+        if (r_lo < nrows) bias2[0] = sig_bias[kvh * g + (row0 + r_lo) % g] * 1.4426950408889634f;
+        if (r_hi < nrows) bias2[1] = sig_bias[kvh * g + (row0 + r_hi) % g] * 1.4426950408889634f;
+    }
 
     float o[NO][4];
 #pragma unroll
@@ -190,7 +205,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
         __syncthreads();
         const int k0 = kbeg + t * BN;
         // (a warp whose rows all lie before the tile, or beyond the window's reach of it, skips it)
-        if (k0 <= warp_pos_max && (window <= 0 || warp_pos_min - (k0 + BN - 1) < window)) {
+        if (k0 <= warp_pos_max && k0 + BN - 1 >= warp_first) {
             float sc[NT_S][4];
 #pragma unroll
             for (int j = 0; j < NT_S; ++j)
@@ -235,11 +250,20 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
                 for (int e = 0; e < 4; ++e) {
                     const int kp = k0 + j * 8 + tig * 2 + (e & 1);
                     const int pos = (e < 2) ? pos_lo : pos_hi;
-                    const bool vis = kp < kend && kp <= pos && (window <= 0 || pos - kp < window);
+                    const bool vis = kp < kend && kp <= pos && kp >= ((e < 2) ? first_lo : first_hi);
                     if (!vis) sc[j][e] = -INFINITY;
                     mx[e >> 1] = fmaxf(mx[e >> 1], sc[j][e]);
                 }
-            float alpha[2];
+            float alpha[2] = {1.f, 1.f};
+            if (sig_bias != nullptr) {
+                // sigmoid(x) = 1 / (1 + 2^(-x log2 e)); a masked score (-inf) gives 0
+#pragma unroll
+                for (int j = 0; j < NT_S; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        sc[j][e] = __fdividef(1.f, 1.f + exp2f(fminf(fmaf(sc[j][e], -scale_log2, -bias2[e >> 1]), 126.f)))
+                                   * (sc[j][e] == -INFINITY ? 0.f : 1.f);
+            } else
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
@@ -322,7 +346,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
         if (splits > 1) {
             const size_t pi = ((size_t)(q0 + tl) * H * maps + head) * splits + blockIdx.y;
             if (tig == 0 && (!NARROW || warp == 0)) {
-                part_ml[2 * pi] = m[h];
+                part_ml[2 * pi] = sig_bias != nullptr ? 0.f : m[h];
                 part_ml[2 * pi + 1] = l[h];
             }
             float* po = part_o + pi * DV + tig * 2;
@@ -336,6 +360,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
         if (sink != nullptr)
             l[h] += (m[h] == -INFINITY) ? 1.f : exp2f(sink[head] * 1.4426950408889634f - m[h]);
         float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
+        if (sig_bias != nullptr) inv = 1.f;
         if (gate != nullptr) {
             const float z = __bfloat162float(gate[(size_t)(q0 + tl) * ldg + head]);
             inv *= 1.0f / (1.0f + __expf(-z));
@@ -364,7 +389,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
 __global__ void __launch_bounds__(128) attention_kv_combine_kernel(
     const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits, bf16* __restrict__ out,
     int ldo, int H, const bf16* __restrict__ gate, int ldg, float* __restrict__ out_f32,
-    const float* __restrict__ sink) {
+    const float* __restrict__ sink, int plain_sum) {
     __shared__ float wgt[32];
     __shared__ float inv_s;
     pdl_wait();
@@ -383,6 +408,7 @@ __global__ void __launch_bounds__(128) attention_kv_combine_kernel(
         if (s == 0) {
             if (sink != nullptr) L += (M == -INFINITY) ? 1.f : exp2f(sink[head] * 1.4426950408889634f - M);
             float inv = L > 0.f ? 1.f / L : 0.f;
+            if (plain_sum) inv = 1.f;                      // (weights that are not normalized)
             if (gate != nullptr) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[t * ldg + head])));
             inv_s = inv;
         }
@@ -441,7 +467,7 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
                                    int H, int Hkv, int maps, int ps, int num_pages, float scale, int window,
                                    const bf16* gate, int ldg, int splits, float* part_o, float* part_ml,
                                    int narrow, int fold, cudaStream_t st, float softcap = 0.f,
-                                   const float* sink = nullptr) {
+                                   const float* sink = nullptr, int chunk = 0, const float* sig_bias = nullptr) {
     // `fold` > 1: H counts (head, map) pairs, `maps` is 1, DK is fold times a map's key size.
     // `narrow`: every tile of the list holds at most 16 rows (a step of single tokens with at most
     // 16 query heads a kv head).
@@ -452,6 +478,8 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
         return SLB_ERR_BAD_ARG;
     if (narrow && H / Hkv > 16) return SLB_ERR_BAD_ARG;
     if (softcap < 0.f || (sink != nullptr && (maps != 1 || fold != 1))) return SLB_ERR_BAD_ARG;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sig_bias != nullptr && (maps != 1 || fold != 1 || sink != nullptr)))
+        return SLB_ERR_BAD_ARG;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || ps <= 0 || max_pages <= 0 || num_pages <= 0 || scale <= 0.f ||
         (tied && DV > DK) || ldq % 8 != 0 || ldo % 2 != 0 || maps < 1 || (maps > 1 && tied) || fold < 1 ||
         (fold > 1 && (maps != 1 || tied || DK % (8 * fold) != 0 || H % fold != 0)))
@@ -470,11 +498,12 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
                              dim3(num_tiles * Hkv * maps, splits), dim3(NTHREADS), smem, st,
                              q, ldq, kc, tied ? kc : vc, tied, out, ldo, block_table, max_pages, cu_q, ctx_len,
                              tile_seq, tile_row0, H, Hkv, ps, num_pages, scale * 1.4426950408889634f, window,
-                             gate, ldg, splits, part_o, part_ml, maps, out_f32, q_rows, fold, softcap, scale, sink);
+                             gate, ldg, splits, part_o, part_ml, maps, out_f32, q_rows, fold, softcap, scale, sink, chunk, sig_bias);
     if (e != 0 || splits == 1) return e;
     // (one tile a token: num_tiles is the number of tokens)
     return slb_launch(attention_kv_combine_kernel, dim3(num_tiles, H * maps), dim3(128), 0, st, (const float*)part_o,
-                      (const float*)part_ml, splits, out, ldo, H * maps, gate, ldg, out_f32, sink);
+                      (const float*)part_ml, splits, out, ldo, H * maps, gate, ldg, out_f32, sink,
+                      sig_bias != nullptr ? 1 : 0);
 }
 // `tied`: the values are the first DV elements of the key rows (vc is ignored).
 int slb_attention_kv_mma_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int tied, bf16* out,
@@ -488,16 +517,18 @@ int slb_attention_kv_mma_bf16(const bf16* q, int ldq, const bf16* kc, const bf16
                                    ldg, splits, part_o, part_ml, narrow, 1, st);
 }
 // The same with a soft cap on the scaled scores (`softcap` > 0: s <- softcap tanh(s / softcap)) and a
-// sink a head (`sink` [H] float32 or null) in the softmax's denominator.
+// sink a head (`sink` [H] float32 or null) in the softmax's denominator; with `chunk` > 0 instead of the
+// window and `sig_bias` ([H] float32 or null) instead of the softmax.
 int slb_attention_kv_mma_capped_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int tied, bf16* out,
                                      int ldo, const int* block_table, int max_pages, const int* cu_q,
                                      const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                                      int H, int Hkv, int ps, int num_pages, float scale, int window,
                                      const bf16* gate, int ldg, int splits, float* part_o, float* part_ml,
-                                     int narrow, float softcap, const float* sink, cudaStream_t st) {
+                                     int narrow, float softcap, const float* sink, int chunk,
+                                     const float* sig_bias, cudaStream_t st) {
     return launch_attention_kv_mma(q, ldq, kc, vc, tied, out, nullptr, ldo, block_table, max_pages, cu_q, ctx_len,
                                    tile_seq, tile_row0, num_tiles, H, Hkv, 1, ps, num_pages, scale, window, gate,
-                                   ldg, splits, part_o, part_ml, narrow, 1, st, softcap, sink);
+                                   ldg, splits, part_o, part_ml, narrow, 1, st, softcap, sink, chunk, sig_bias);
 }
 // `maps` attention maps a head; float32 results [token][head][map][DV] with rows `ldo` floats apart
 int slb_attention_kv_mma_maps_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int maps, float* out,

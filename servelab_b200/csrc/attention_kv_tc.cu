@@ -8,7 +8,10 @@
 //   * `tied`: the values are the first SLB_VALUE_DIM elements of the key rows (the absorbed form
 //     of a latent attention).  The K tile is then also the V operand: nothing is fetched twice,
 //     there is no value ring, and a key stage is given back when the tile's P.V has run;
-//   * optional epilogue: head h's row times sigmoid(gate[token][h]).
+//   * optional epilogue: head h's row times sigmoid(gate[token][h]);
+//   * `sig_bias` (one number a head) instead of the softmax: a visible key's weight is
+//     sigmoid(score + sig_bias_h), not normalized, so the accumulator is never rescaled; `chunk` > 0
+//     instead of the window: a query at position i sees the keys j <= i with j / chunk == i / chunk.
 //
 // Work unit: 128 query rows x one kv head (rho = local_token * g + head_in_group, whole tokens per
 // tile).  Per 64-key tile: loader warps bring the pages' rows by TMA (128-byte swizzle) into
@@ -180,7 +183,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
     const int* __restrict__ ctx_len, const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
     int H, int Hkv, int ps, int box_rows, float scale_log2, int window, int* __restrict__ status, int tied,
     const bf16* __restrict__ gate, int ldg, int maps, float* __restrict__ out32, int ldo32,
-    float cap_in, float cap_back, const float* __restrict__ sink) {
+    float cap_in, float cap_back, const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias) {
     // cap_in > 0: a soft cap c on the scaled scores.  With s the raw score, cap_in = 2 log2(e) scale / c
     // and cap_back = c / scale, the raw score becomes cap_back tanh(s scale / c), so that what follows
     // (which multiplies by scale log2 e) sees the capped score; tanh(x) = 1 - 2 / (e^(2x) + 1).
@@ -227,6 +230,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
     const int p_last = pos_base + tok0 + (nrows - 1) / g;
     int kbeg = 0;
     if (window > 0) kbeg = max(0, p_first - window + 1) / BN * BN;
+    if (chunk > 0) kbeg = p_first / chunk * chunk / BN * BN;
     const int kend = p_last + 1;
     const int ntiles = (kend - kbeg + BN - 1) / BN;
 
@@ -377,7 +381,11 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
         const int r = quarter * 32 + lane;
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const int pos = r < nrows ? pos_base + tok0 + r / g : -1;
+        const int pos_first = window > 0 ? pos - window + 1 : chunk > 0 && pos >= 0 ? pos - pos % chunk : 0;
+        // the first key that every row of the block sees (rows are in the order of their positions)
+        const int all_first = window > 0 ? p_last - window + 1 : chunk > 0 ? p_last - p_last % chunk : 0;
         float m_ref = -INFINITY, l = 0.f;
+        const float bias2 = sig_bias != nullptr && r < nrows ? sig_bias[kvh * g + r % g] * 1.4426950408889634f : 0.f;
         bool ok = true;
         for (int j = 0; j < ntiles && ok; ++j) {
             if (!mbar_spin(&s_full[j & 1], (j >> 1) & 1)) { if (lane == 0) gave_up(status, 0x301, 2, j, ntiles); ok = false; break; }
@@ -399,7 +407,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
             // raw scores stay unscaled; masked ones become -inf.  A tile that every row of
             // the block sees completely needs no mask (rows of padding compute garbage that
             // is never stored).
-            const bool open = k0 + BN - 1 <= p_first && (window <= 0 || p_last - k0 < window);
+            const bool open = k0 + BN - 1 <= p_first && k0 >= all_first;
             float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four chains, not one
             if (open) {
 #pragma unroll
@@ -408,7 +416,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
                     for (int i = 0; i < 32; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(raw[h][i]));
             } else {
                 const int hi = min(BN, min(kend, pos + 1) - k0);      // visible keys: [lo, hi)
-                const int lo = window > 0 ? max(0, pos - window + 1 - k0) : 0;
+                const int lo = max(0, pos_first - k0);
 #pragma unroll
                 for (int h = 0; h < 2; ++h)
 #pragma unroll
@@ -420,13 +428,24 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
             }
             const float mt = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2;   // scale > 0
             float alpha = 1.f;
+            float sm[4] = {0.f, 0.f, 0.f, 0.f};
+            uint32_t packed[32];
+            if (sig_bias != nullptr) {
+                // sigmoid(x) = 1 / (1 + 2^(-x log2 e)); a masked score (-inf) gives 2^inf and so 0
+#pragma unroll
+                for (int h = 0; h < 2; ++h)
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2) {
+                        const float e0 = fast_exp2(fmaf(__uint_as_float(raw[h][i]), -scale_log2, -bias2));
+                        const float e1 = fast_exp2(fmaf(__uint_as_float(raw[h][i + 1]), -scale_log2, -bias2));
+                        packed[h * 16 + i / 2] = pack2(__frcp_rn(1.f + e0), __frcp_rn(1.f + e1));
+                    }
+            } else {
             if (mt > m_ref + RESCALE_THRESHOLD || (m_ref == -INFINITY && mt != -INFINITY)) {
                 alpha = (m_ref == -INFINITY) ? 0.f : exp2f(m_ref - mt);
                 m_ref = mt;
             }
             const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
-            float sm[4] = {0.f, 0.f, 0.f, 0.f};
-            uint32_t packed[32];
 #pragma unroll
             for (int h = 0; h < 2; ++h)
 #pragma unroll
@@ -437,6 +456,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
                     packed[h * 16 + i / 2] = pack2(p0, p1);
                 }
             l = l * alpha + ((sm[0] + sm[1]) + (sm[2] + sm[3]));
+            }
             if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
                 // the accumulator is rescaled (rarely): P.V of the previous tile must be done
                 if (!mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1)) { if (lane == 0) gave_up(status, 0x302, 2, j, ntiles); ok = false; break; }
@@ -466,6 +486,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
         if (sink != nullptr && r < nrows)
             l += (m_ref == -INFINITY) ? 1.f : exp2f(sink[kvh * g + hg] * 1.4426950408889634f - m_ref);
         float inv = l > 0.f ? 1.f / l : 0.f;
+        if (sig_bias != nullptr) inv = 1.f;
         if (gate != nullptr && r < nrows)
             inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)(q0 + tok0 + tl) * ldg + kvh * g + hg])));
         bf16* dst = out + (size_t)(q0 + tok0 + tl) * ldo + (size_t)(kvh * g + hg) * DV;
@@ -522,9 +543,11 @@ static int launch_attention_kv_tc(const bf16* q, int ldq, const bf16* kc, const 
                                   const int* tile_seq, const int* tile_row0, int num_tiles, int H, int Hkv, int ps,
                                   int num_pages, float scale, int window, const bf16* gate, int ldg, int maps,
                                   float* out32, int ldo32, cudaStream_t st, float softcap = 0.f,
-                                  const float* sink = nullptr) {
+                                  const float* sink = nullptr, int chunk = 0, const float* sig_bias = nullptr) {
     if (num_tiles <= 0) return 0;
     if (softcap < 0.f || (sink != nullptr && maps != 1)) return SLB_ERR_BAD_ARG;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sig_bias != nullptr && (maps != 1 || sink != nullptr)))
+        return SLB_ERR_BAD_ARG;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || max_pages <= 0 || num_pages <= 0 || !(scale > 0.f) || maps < 1 ||
         maps > 64)
         return SLB_ERR_BAD_ARG;
@@ -560,7 +583,7 @@ static int launch_attention_kv_tc(const bf16* q, int ldq, const bf16* kc, const 
                       map_k, map_v, out, ldo, block_table, max_pages, cu_q, ctx_len, tile_seq, tile_row0, H, Hkv,
                       ps, box_rows, scale * 1.4426950408889634f, window, status, tied, gate, ldg, maps, out32, ldo32,
                       softcap > 0.f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.f,
-                      softcap > 0.f ? softcap / scale : 0.f, sink);
+                      softcap > 0.f ? softcap / scale : 0.f, sink, chunk, sig_bias);
 }
 
 extern "C" {
@@ -575,15 +598,17 @@ int slb_attention_kv_tc_bf16(const bf16* q, int ldq, const bf16* kc, const bf16*
                                   0, st);
 }
 // The same with a soft cap on the scaled scores (`softcap` > 0: s <- softcap tanh(s / softcap)) and a
-// sink a head (`sink` [H] float32 or null) in the softmax's denominator.
+// sink a head (`sink` [H] float32 or null) in the softmax's denominator; with `chunk` > 0 instead of the
+// window and `sig_bias` ([H] float32 or null) instead of the softmax.
 int slb_attention_kv_tc_capped_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int tied, bf16* out,
                                     int ldo, const int* block_table, int max_pages, const int* cu_q,
                                     const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                                     int H, int Hkv, int ps, int num_pages, float scale, int window, const bf16* gate,
-                                    int ldg, float softcap, const float* sink, cudaStream_t st) {
+                                    int ldg, float softcap, const float* sink, int chunk, const float* sig_bias,
+                                    cudaStream_t st) {
     return launch_attention_kv_tc(q, ldq, kc, vc, tied, out, ldo, block_table, max_pages, cu_q, ctx_len, tile_seq,
                                   tile_row0, num_tiles, H, Hkv, ps, num_pages, scale, window, gate, ldg, 1, nullptr,
-                                  0, st, softcap, sink);
+                                  0, st, softcap, sink, chunk, sig_bias);
 }
 // `maps` attention maps a head: q [T][H][maps][DK], k_cache [num_pages][Hkv][ps][maps * DK], one set
 // of values a kv head, float32 results per map out32 [T][H][maps][DV].
@@ -626,7 +651,7 @@ int slb_attention_kv_tc_bf16(const bf16*, int, const bf16*, const bf16*, int, bf
 }
 int slb_attention_kv_tc_capped_bf16(const bf16*, int, const bf16*, const bf16*, int, bf16*, int, const int*, int,
                                     const int*, const int*, const int*, const int*, int, int, int, int, int, float,
-                                    int, const bf16*, int, float, const float*, cudaStream_t) {
+                                    int, const bf16*, int, float, const float*, int, const float*, cudaStream_t) {
     return SLB_ERR_BAD_ARG;
 }
 int slb_attention_kv_tc_maps_bf16(const bf16*, int, const bf16*, const bf16*, float*, int, const int*, int, const int*,

@@ -53,6 +53,7 @@ __global__ void __launch_bounds__(DA_EV * DA_PARTS, R <= 16 ? 4 : 2) decay_atten
     float* vs = ks + DA_TT * LD;                 // [DA_TT][DA_EV]
     float* part = vs + DA_TT * DA_EV;            // [DA_TT][DA_PARTS][DA_EV]
     float* as = part + DA_TT * DA_PARTS * DA_EV; // [DA_TT][LD]: the decays of a token's key channels (gated form)
+    float* bs = as + DA_TT * LD;                 // [LD]: the bonus of the head's key channels (if any)
     const bool gated = a.gate_z != nullptr;
     const int tid = threadIdx.x, p = tid >> 5, e = tid & 31;
     const int col = e0 + e;
@@ -67,6 +68,13 @@ __global__ void __launch_bounds__(DA_EV * DA_PARTS, R <= 16 ? 4 : 2) decay_atten
         st[i] = (live && i < Dp && d < D) ? srow[(size_t)d * Dv + col] : 0.f;
     }
     const T* proj = reinterpret_cast<const T*>(a.proj);
+    const bool bonus = a.bonus != nullptr;
+    if (bonus) {
+        for (int c = tid; c < LD; c += DA_EV * DA_PARTS) {
+            const int pp = c / Dpad, i = c - pp * Dpad, d = pp * Dp + i;
+            bs[c] = (i < Dp && d < D) ? a.bonus[h * D + d] : 0.f;
+        }
+    }
     for (int t0 = 0; t0 < qlen; t0 += DA_TT) {
         const int n = min(DA_TT, qlen - t0);
         for (int idx = tid; idx < n * LD; idx += DA_EV * DA_PARTS) {
@@ -82,8 +90,7 @@ __global__ void __launch_bounds__(DA_EV * DA_PARTS, R <= 16 ? 4 : 2) decay_atten
                 if (gated) {
                     float z = a.gate_z[(size_t)(q0 + t0 + j) * a.ld_gate + h * D + d];
                     if (a.gate_bias != nullptr) z += a.gate_bias[h * D + d];
-                    // log sigmoid(z) = min(z, 0) - log(1 + exp(-|z|))
-                    av = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * a.gate_inv_tau);
+                    av = expf(da_log_decay(z, a.gate_kind, a.gate_inv_tau));
                 }
             }
             qs[idx] = qv;
@@ -105,6 +112,27 @@ __global__ void __launch_bounds__(DA_EV * DA_PARTS, R <= 16 ? 4 : 2) decay_atten
             const float4* qj = reinterpret_cast<const float4*>(qs + j * LD + p * Dpad);
             const float4* kj = reinterpret_cast<const float4*>(ks + j * LD + p * Dpad);
             float acc = 0.f;
+            if (bonus) {
+                // the result reads the state before the update, and the token itself through its bonus
+                const float4* aj = reinterpret_cast<const float4*>(as + j * LD + p * Dpad);
+                const float4* bj = reinterpret_cast<const float4*>(bs + p * Dpad);
+#pragma unroll
+                for (int i4 = 0; i4 < R / 4; ++i4) {
+                    if (i4 * 4 < Dp) {
+                        const float4 k4 = kj[i4], q4 = qj[i4], a4 = aj[i4], b4 = bj[i4];
+                        const float kv[4] = {k4.x * v, k4.y * v, k4.z * v, k4.w * v};
+                        const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, aa[4] = {a4.x, a4.y, a4.z, a4.w};
+                        const float bb[4] = {b4.x, b4.y, b4.z, b4.w};
+#pragma unroll
+                        for (int u = 0; u < 4; ++u) {
+                            acc = fmaf(fmaf(bb[u], kv[u], st[4 * i4 + u]), qq[u], acc);
+                            st[4 * i4 + u] = fmaf(aa[u], st[4 * i4 + u], kv[u]);
+                        }
+                    }
+                }
+                part[(j * DA_PARTS + p) * DA_EV + e] = acc;
+                continue;
+            }
             if (gated) {
                 const float4* aj = reinterpret_cast<const float4*>(as + j * LD + p * Dpad);
 #pragma unroll
@@ -169,6 +197,7 @@ static int launch_decay_attention(const DecayAttnArgs* a_in, int num_seqs, cudaS
     if (a->state_stride < (long long)a->H * a->D * a->Dv) return SLB_ERR_BAD_ARG;
     if ((a->gate_z == nullptr) == (a->decay == nullptr)) return SLB_ERR_BAD_ARG;      // one of the two
     if (a->gate_z != nullptr && (a->ld_gate < a->H * a->D || !(a->gate_inv_tau > 0.f))) return SLB_ERR_BAD_ARG;
+    if (a->gate_kind < 0 || a->gate_kind > 1 || (a->bonus != nullptr && a->gate_z == nullptr)) return SLB_ERR_BAD_ARG;
     if (a->H <= 0 || a->D <= 0 || a->Dv <= 0 || a->num_slots <= 0 || (a->rot_dims & 1) || a->rot_dims < 0 ||
         a->rot_dims > a->D || (a->rot_dims > 0 && a->freq == nullptr) || a->act < 0 || a->act > 1)
         return SLB_ERR_BAD_ARG;
@@ -177,7 +206,7 @@ static int launch_decay_attention(const DecayAttnArgs* a_in, int num_seqs, cudaS
     if (vz > 65535) return SLB_ERR_TOO_LARGE;
     const int dpad = ((a->D + DA_PARTS - 1) / DA_PARTS + 3) / 4 * 4;
     const size_t smem = ((size_t)(a->gate_z != nullptr ? 3 : 2) * DA_TT * DA_PARTS * dpad + DA_TT * DA_EV +
-                         DA_TT * DA_PARTS * DA_EV) * sizeof(float);
+                         DA_TT * DA_PARTS * DA_EV + (a->bonus != nullptr ? DA_PARTS * dpad : 0)) * sizeof(float);
     if (a->D <= 16 * DA_PARTS)
         return slb_launch(decay_attention_kernel<T, 16>, dim3(num_seqs, a->H, vz), dim3(DA_EV * DA_PARTS), smem, st, *a);
     return slb_launch(decay_attention_kernel<T, DA_MAX_D / DA_PARTS>, dim3(num_seqs, a->H, vz), dim3(DA_EV * DA_PARTS),

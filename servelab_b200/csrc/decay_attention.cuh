@@ -22,7 +22,21 @@ struct DecayAttnArgs {
     const float* gate_z; int ld_gate; const float* gate_bias; float gate_inv_tau;
     float q_scale;
     long long state_stride;
+    // appended: how a learned decay is formed from its logit (below), and a factor per head and key
+    // channel with which the current token enters its own result instead of through the state:
+    // o_t = (S_{t-1} + diag(bonus) k_t v_t^T)^T q_t
+    int gate_kind;
+    const float* bonus;            // [H * D] or null
 };
+
+// The logarithm of a learned decay, never positive.
+//   kind 0: sigmoid(z)^p: log sigmoid(z) = min(z, 0) - log(1 + exp(-|z|)), times p
+//   kind 1: exp(-exp(z)), bounded below where the decay is zero in float32 anyway (so that sums and
+//           differences of logarithms stay finite)
+__device__ __forceinline__ float da_log_decay(float z, int kind, float p) {
+    if (kind == 1) return -fminf(expf(z), 110.f);
+    return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * p;
+}
 
 __device__ __forceinline__ float da_silu(float z) { return z / (1.0f + expf(-z)); }
 

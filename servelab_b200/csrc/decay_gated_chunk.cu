@@ -10,6 +10,10 @@
 //     A[t][j] = sum_d q_t[d] k_j[d] e^(L_t[d] - L_j[d]),
 //     S_out = diag(e^(L_last)) S + sum_j diag(e^(L_last - L_j)) k_j v_j^T.
 //
+// With a bonus the result reads the state before the token's own update and the token itself through a
+// learned factor per key channel, o_t = (S_{t-1} + diag(bonus) k_t v_t^T)^T q_t: then e^(L_{t-1}[d])
+// takes the place of e^(L_t[d]) in o_t and in A[t][j] for j < t, and A[t][t] = sum_d q_t bonus k_t.
+//
 // Every exponent is a difference L_t - L_j with j <= t, or L_t itself: never positive, so nothing
 // overflows however fast a channel decays (a factorised form q e^L . k e^-L would).  All
 // arithmetic is float32 on the CUDA cores: the logarithms of the decays, their sums, the
@@ -75,7 +79,7 @@ __global__ void __launch_bounds__(256) gated_chunk_prep_kernel(const GatedChunkA
         const int j = idx / D, d = idx - j * D;
         float z = a.gate_z[(size_t)(t0 + j) * a.ld_gate + h * D + d];
         if (a.gate_bias != nullptr) z += a.gate_bias[h * D + d];
-        Ls[j * LD + d] = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * a.gate_inv_tau;      // log sigmoid(z) / tau
+        Ls[j * LD + d] = da_log_decay(z, a.gate_kind, a.gate_inv_tau);
     }
     __syncthreads();
     // ... then their running sums, a channel a thread, in the order of the tokens
@@ -99,7 +103,8 @@ __global__ void __launch_bounds__(256) gated_chunk_prep_kernel(const GatedChunkA
         const float L = Ls[j * LD + d];
         qs[j * LD + d] = qv;
         ks[j * LD + d] = kv;
-        c.qdec[(size_t)(t0 + j) * ldl + h * D + d] = qv * expf(L);
+        const float Lq = a.bonus == nullptr ? L : (j > 0 ? Ls[(j - 1) * LD + d] : 0.f);
+        c.qdec[(size_t)(t0 + j) * ldl + h * D + d] = qv * expf(Lq);
         c.kdec[(size_t)(t0 + j) * ldl + h * D + d] = kv * expf(Ls[(n - 1) * LD + d] - L);
     }
     __syncthreads();
@@ -115,9 +120,15 @@ __global__ void __launch_bounds__(256) gated_chunk_prep_kernel(const GatedChunkA
         const int j = e - t * (t + 1) / 2;
         const float* qt = qs + t * LD;
         const float* kj = ks + j * LD;
-        const float* Lt = Ls + t * LD;
+        const float* Lt = Ls + (a.bonus == nullptr ? t : t - 1) * LD;      // (t > j >= 0 where it is read)
         const float* Lj = Ls + j * LD;
         float sum = 0.f;
+        if (a.bonus != nullptr && t == j) {
+            const float* bn = a.bonus + h * D;
+            for (int d = 0; d < D; ++d) sum = fmaf(qt[d] * kj[d], bn[d], sum);
+            A[t * GC_CHUNK + j] = sum;
+            continue;
+        }
         // (the exponent is <= 0; the one-instruction 2^x is exact to 2 ulp there, and its argument's
         // rounding weighs on terms that are small by the same factor)
         for (int d = 0; d < D; ++d) sum = fmaf(qt[d] * kj[d], __expf(Lt[d] - Lj[d]), sum);
@@ -358,7 +369,8 @@ static int launch_gated_chunk(const GatedChunkArgs* c_in, int num_seqs, cudaStre
     if (a.state_stride <= 0) a.state_stride = (long long)a.H * a.D * a.Dv;
     if (a.H <= 0 || a.D <= 0 || a.Dv <= 0 || a.num_slots <= 0 || (a.rot_dims & 1) || a.rot_dims < 0 ||
         a.rot_dims > a.D || (a.rot_dims > 0 && a.freq == nullptr) || a.act < 0 || a.act > 1 ||
-        a.gate_z == nullptr || a.ld_gate < a.H * a.D || !(a.gate_inv_tau > 0.f) ||
+        a.gate_z == nullptr || a.ld_gate < a.H * a.D || !(a.gate_inv_tau > 0.f) || a.gate_kind < 0 ||
+        a.gate_kind > 1 ||
         a.state_stride < (long long)a.H * a.D * a.Dv || c.work == nullptr || c.qdec == nullptr || c.kdec == nullptr ||
         c.dtot == nullptr || c.scores == nullptr || c.tile_seq == nullptr || c.tile_row0 == nullptr)
         return SLB_ERR_BAD_ARG;

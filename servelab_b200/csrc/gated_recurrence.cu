@@ -1,0 +1,123 @@
+// A gated linear recurrence, one number of state a channel (float32, in a state slot):
+//
+//     log a_t = rate r_t,   S_t = a_t S_{t-1} + sqrt(1 - a_t^2) i_t u_t,   out_t = S_t gelu_tanh(y_t + b_y)
+//
+// with r_t = sigmoid(z^r_t + b_r), i_t = sigmoid(z^i_t + b_i) and rate = -coef softplus(lambda) <= 0 per
+// channel.  u (behind its convolution) and y have the compute type; the gates' logits z are float32 and
+// come from block-diagonal products: block b of n channels has its logits at z + b * z_block +
+// token * z_token, n for r and then n for i.  Everything here is float32; S is zero for a new request.
+//
+// A block owns 16 channels of a request and takes its tokens 64 at a time: all threads form a and the
+// update of every (token, channel), 16 threads walk the tokens (one multiply-add each, in order, so the
+// result of a token does not depend on how the request was cut), all threads finish the outputs.
+#include "common.cuh"
+
+#define GR_EC 16
+#define GR_TT 64
+
+struct GatedRecArgs {
+    const void* u; int ldu;
+    const float* z; long long z_block, z_token;
+    const float* r_bias; const float* i_bias; const float* rate;
+    const void* y; int ldy; const float* y_bias;
+    float* state; long long state_stride; int num_slots;
+    const int* cu_q; const int* state_slots;
+    int width, n;
+    void* out; int ldo;
+};
+
+__device__ __forceinline__ float gr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gr_gelu_tanh(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+// a and sqrt(1 - a^2) from log a (1 - a^2 = -expm1(2 log a): no cancellation for a near 1)
+__device__ __forceinline__ void gr_decay(float log_a, float& a, float& gain) {
+    a = expf(log_a);
+    gain = sqrtf(-expm1f(2.0f * log_a));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) gated_recurrence_kernel(const GatedRecArgs g) {
+    __shared__ float sa[GR_TT][GR_EC], sb[GR_TT][GR_EC];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.x, c0 = blockIdx.y * GR_EC;
+    const int q0 = g.cu_q[s];
+    const int qlen = g.cu_q[s + 1] - q0;
+    if (qlen <= 0) return;
+    const int slot = g.state_slots[s];
+    if (slot < 0 || slot >= g.num_slots) return;
+    const int tid = threadIdx.x, ch = tid % GR_EC, tk = tid / GR_EC;
+    const int c = c0 + ch;
+    const bool live = c < g.width;
+    const T* u = reinterpret_cast<const T*>(g.u);
+    const T* y = reinterpret_cast<const T*>(g.y);
+    T* out = reinterpret_cast<T*>(g.out);
+    float rb = 0.f, ib = 0.f, rate = 0.f, yb = 0.f;
+    const float* z = g.z;
+    if (live) {
+        rb = g.r_bias[c]; ib = g.i_bias[c]; rate = g.rate[c]; yb = g.y_bias[c];
+        const int b = c / g.n;
+        z += (size_t)b * g.z_block + (c - b * g.n);
+    }
+    float* sp = g.state + (size_t)slot * g.state_stride + c;
+    float S = live && tk == 0 ? *sp : 0.f;
+    constexpr int PER = 256 / GR_EC;             // tokens in flight
+    for (int t0 = 0; t0 < qlen; t0 += GR_TT) {
+        const int n = min(GR_TT, qlen - t0);
+#pragma unroll
+        for (int i = 0; i < GR_TT / PER; ++i) {
+            const int j = tk + i * PER;
+            if (j < n && live) {
+                const size_t t = q0 + t0 + j;
+                const float r = gr_sigmoid(z[t * g.z_token] + rb);
+                const float in = gr_sigmoid(z[t * g.z_token + g.n] + ib);
+                float a, gain;
+                gr_decay(rate * r, a, gain);
+                sa[j][ch] = a;
+                sb[j][ch] = gain * in * to_float(u[t * g.ldu + c]);
+            }
+        }
+        __syncthreads();
+        if (tk == 0 && live) {
+#pragma unroll 8
+            for (int j = 0; j < n; ++j) {
+                S = fmaf(sa[j][ch], S, sb[j][ch]);
+                sb[j][ch] = S;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < GR_TT / PER; ++i) {
+            const int j = tk + i * PER;
+            if (j < n && live) {
+                const size_t t = q0 + t0 + j;
+                out[t * g.ldo + c] = from_float<T>(sb[j][ch] * gr_gelu_tanh(to_float(y[t * g.ldy + c]) + yb));
+            }
+        }
+        // (a thread overwrites only the elements of sa and sb that it has just read itself, and the
+        // walk over them comes after the next barrier)
+    }
+    if (tk == 0 && live) *sp = S;
+}
+
+template <typename T>
+static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, cudaStream_t st) {
+    if (num_seqs <= 0) return 0;
+    if (g.width <= 0 || g.n <= 0 || g.width % g.n || g.u == nullptr || g.z == nullptr || g.y == nullptr ||
+        g.state == nullptr || g.state_stride < g.width || g.num_slots <= 0 || g.r_bias == nullptr ||
+        g.i_bias == nullptr || g.rate == nullptr || g.y_bias == nullptr || g.out == nullptr)
+        return SLB_ERR_BAD_ARG;
+    const int gy = (g.width + GR_EC - 1) / GR_EC;
+    if (gy > 65535) return SLB_ERR_TOO_LARGE;
+    return slb_launch(gated_recurrence_kernel<T>, dim3(num_seqs, gy), dim3(256), 0, st, g);
+}
+
+extern "C" {
+int slb_gated_recurrence_f32(const GatedRecArgs* g, int num_seqs, cudaStream_t st) {
+    return launch_gated_recurrence<float>(*g, num_seqs, st);
+}
+int slb_gated_recurrence_bf16(const GatedRecArgs* g, int num_seqs, cudaStream_t st) {
+    return launch_gated_recurrence<bf16>(*g, num_seqs, st);
+}
+}

@@ -15,7 +15,8 @@
 #define GS_BN 64
 #define GS_BK 16
 
-template <typename TA, typename TW, typename TC>
+// ACT 1: tanh on every element of A as it is loaded (the second product of a bottleneck).
+template <typename TA, typename TW, typename TC, int ACT = 0>
 __global__ void __launch_bounds__(256) gemm_tn_simt_kernel(
     const TA* __restrict__ A, int lda, const TW* __restrict__ W, int ldw, TC* __restrict__ C,
     int ldc, const float* __restrict__ bias, int M, int N, int K, long long batch_a,
@@ -41,7 +42,9 @@ __global__ void __launch_bounds__(256) gemm_tn_simt_kernel(
             const int idx = tid + i * 256;
             const int row = idx >> 4, kk = idx & 15;
             const int gm = m0 + row, gn = n0 + row, gk = k0 + kk;
-            As[kk][row] = (gm < M && gk < K) ? to_float(A[(size_t)gm * lda + gk]) : 0.f;
+            float av = (gm < M && gk < K) ? to_float(A[(size_t)gm * lda + gk]) : 0.f;
+            if (ACT == 1) av = tanhf(av);
+            As[kk][row] = av;
             Ws[kk][row] = (gn < N && gk < K) ? to_float(W[(size_t)gn * ldw + gk]) : 0.f;
         }
         __syncthreads();
@@ -71,7 +74,7 @@ __global__ void __launch_bounds__(256) gemm_tn_simt_kernel(
     }
 }
 
-template <typename TA, typename TW, typename TC>
+template <typename TA, typename TW, typename TC, int ACT = 0>
 static int launch_gemm(const TA* A, int lda, const TW* W, int ldw, TC* C, int ldc,
                        const float* bias, int M, int N, int K, cudaStream_t st, int batch = 1,
                        long long batch_a = 0, long long batch_w = 0, long long batch_c = 0) {
@@ -79,7 +82,7 @@ static int launch_gemm(const TA* A, int lda, const TW* W, int ldw, TC* C, int ld
     if (K <= 0 || lda < K || ldw < K || ldc < N) return SLB_ERR_BAD_ARG;
     const int gy = (M + GS_BM - 1) / GS_BM;
     if (gy > 65535 || batch > 65535) return SLB_ERR_TOO_LARGE;
-    return slb_launch(gemm_tn_simt_kernel<TA, TW, TC>, dim3((N + GS_BN - 1) / GS_BN, gy, batch), dim3(256),
+    return slb_launch(gemm_tn_simt_kernel<TA, TW, TC, ACT>, dim3((N + GS_BN - 1) / GS_BN, gy, batch), dim3(256),
                       0, st, A, lda, W, ldw, C, ldc, bias, M, N, K, batch_a, batch_w, batch_c);
 }
 
@@ -105,6 +108,21 @@ int slb_gemm_simt_batched_bf16(const bf16* A, int lda, const bf16* W, int ldw, b
                                long long batch_c, cudaStream_t st) {
     return launch_gemm<bf16, bf16, bf16>(A, lda, W, ldw, C, ldc, nullptr, M, N, K, st, batch, batch_a,
                                          batch_w, batch_c);
+}
+int slb_gemm_simt_batched_bf16_f32out(const bf16* A, int lda, const bf16* W, int ldw, float* C, int ldc, int M,
+                                      int N, int K, int batch, long long batch_a, long long batch_w,
+                                      long long batch_c, cudaStream_t st) {
+    return launch_gemm<bf16, bf16, float>(A, lda, W, ldw, C, ldc, nullptr, M, N, K, st, batch, batch_a, batch_w,
+                                          batch_c);
+}
+// C = tanh(A) . W^T (+ bias), float32 results
+int slb_gemm_simt_tanh_f32(const float* A, int lda, const float* W, int ldw, float* C, int ldc,
+                           const float* bias, int M, int N, int K, cudaStream_t st) {
+    return launch_gemm<float, float, float, 1>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
+}
+int slb_gemm_simt_tanh_bf16(const bf16* A, int lda, const bf16* W, int ldw, float* C, int ldc,
+                            const float* bias, int M, int N, int K, cudaStream_t st) {
+    return launch_gemm<bf16, bf16, float, 1>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
 }
 int slb_gemm_simt_bf16_f32out(const bf16* A, int lda, const bf16* W, int ldw, float* C, int ldc,
                               const float* bias, int M, int N, int K, cudaStream_t st) {

@@ -21,7 +21,9 @@
 //
 // With no key heads (Hkv = 0) every channel is a "query" channel: the kernel is then a plain
 // convolution of the first q_size columns into q_out, which a mixer runs on q | k | v before its
-// head kernel.  The records of two requests lie `state_stride` floats apart (a record may be part of
+// head kernel.  Two biases are optional: one on the projected rows (`in_bias`: what the record holds
+// then includes it, so the zeros before a sequence's start stay zeros) and one on the result.  The
+// records of two requests lie `state_stride` floats apart (a record may be part of
 // a larger one).
 #include "common.cuh"
 
@@ -78,7 +80,8 @@ __global__ void __launch_bounds__(256) qk_conv_cache_kernel(
     const int* __restrict__ seq_of_token, const int* __restrict__ positions,
     const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
     float temp_coef, int temp_every, T* __restrict__ q_out, int ldq, T* __restrict__ k_cache,
-    int q_size, int Hkv, int D, int update_inline, long long state_stride) {
+    int q_size, int Hkv, int D, int update_inline, long long state_stride,
+    const float* __restrict__ in_bias, const float* __restrict__ out_bias) {
     const int C = q_size + Hkv * D;
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     pdl_launch_dependents();
@@ -93,12 +96,16 @@ __global__ void __launch_bounds__(256) qk_conv_cache_kernel(
     float* st = state != nullptr ? state + (size_t)state_slots[s] * state_stride + c : nullptr;
     float y[VEC];
 #pragma unroll
-    for (int v = 0; v < VEC; ++v) y[v] = 0.f;
+    for (int v = 0; v < VEC; ++v) y[v] = out_bias != nullptr ? out_bias[c + v] : 0.f;
     for (int i = 0; i < taps; ++i) {
         const int jj = j - hist + i;
         float u[VEC], w[VEC];
         if (jj >= 0) {
             load_vec<T, VEC>(proj + (size_t)(q0 + jj) * ldp + c, u);
+            if (in_bias != nullptr) {
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) u[v] += in_bias[c + v];
+            }
         } else if (st != nullptr) {
             load_vec<float, VEC>(st + (size_t)(hist + jj) * C, u);
         } else {
@@ -133,7 +140,8 @@ __global__ void __launch_bounds__(256) qk_conv_cache_kernel(
 template <typename T>
 __global__ void __launch_bounds__(256) conv_state_update_kernel(
     const T* __restrict__ proj, int ldp, int taps, float* __restrict__ state,
-    const int* __restrict__ state_slots, const int* __restrict__ cu_q, int C, long long state_stride) {
+    const int* __restrict__ state_slots, const int* __restrict__ cu_q, int C, long long state_stride,
+    const float* __restrict__ in_bias) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -143,10 +151,11 @@ __global__ void __launch_bounds__(256) conv_state_update_kernel(
     if (n <= 0) return;
     const int hist = taps - 1;
     float* st = state + (size_t)state_slots[s] * state_stride + c;
+    const float add = in_bias != nullptr ? in_bias[c] : 0.f;
     // ascending i: row i + n of the old record is read before any row >= i + 1 is written
     for (int i = 0; i < hist; ++i) {
         const int src = i + n - hist;              // index into the portion, or before it
-        st[(size_t)i * C] = src >= 0 ? to_float(proj[(size_t)(q0 + src) * ldp + c]) : st[(size_t)(i + n) * C];
+        st[(size_t)i * C] = src >= 0 ? to_float(proj[(size_t)(q0 + src) * ldp + c]) + add : st[(size_t)(i + n) * C];
     }
 }
 
@@ -156,7 +165,7 @@ static int launch_conv(const T* proj, int ldp, const float* taps_w, int taps, fl
                        const int* positions, const int* block_table, int max_pages, int page_size,
                        int num_pages, float temp_coef, int temp_every, T* q_out, int ldq, T* k_cache,
                        int T_tokens, int S, int q_size, int Hkv, int D, int decode_only, long long state_stride,
-                       cudaStream_t st) {
+                       cudaStream_t st, const float* in_bias = nullptr, const float* out_bias = nullptr) {
     if (T_tokens <= 0) return 0;
     if (state_stride <= 0) state_stride = (long long)(taps - 1) * (q_size + Hkv * D);
     if (state_stride < (long long)(taps - 1) * (q_size + Hkv * D)) return SLB_ERR_BAD_ARG;
@@ -179,19 +188,36 @@ static int launch_conv(const T* proj, int ldp, const float* taps_w, int taps, fl
         rc = slb_launch(qk_conv_cache_kernel<T, V>, dim3((C / V + threads - 1) / threads, T_tokens), dim3(threads),
                         0, st, proj, ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions,
                         block_table, max_pages, page_size, num_pages, temp_coef, temp_every, q_out, ldq,
-                        k_cache, q_size, Hkv, D, inline_update, state_stride);
+                        k_cache, q_size, Hkv, D, inline_update, state_stride, in_bias, out_bias);
     } else {
         rc = slb_launch(qk_conv_cache_kernel<T, 1>, dim3((C + 255) / 256, T_tokens), dim3(256), 0, st, proj,
                         ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions, block_table,
                         max_pages, page_size, num_pages, temp_coef, temp_every, q_out, ldq, k_cache, q_size,
-                        Hkv, D, inline_update, state_stride);
+                        Hkv, D, inline_update, state_stride, in_bias, out_bias);
     }
     if (rc != 0 || taps == 1 || inline_update) return rc;
     return slb_launch(conv_state_update_kernel<T>, dim3((C + 255) / 256, S), dim3(256), 0, st, proj, ldp,
-                      taps, state, state_slots, cu_q, C, state_stride);
+                      taps, state, state_slots, cu_q, C, state_stride, in_bias);
 }
 
 extern "C" {
+// the convolution alone of the first C columns of proj, with biases (null: none)
+int slb_short_conv_f32(const float* proj, int ldp, const float* taps_w, int taps, float* state,
+                       const int* state_slots, const int* cu_q, const int* seq_of_token, const int* positions,
+                       float* out, int ldo, int T_tokens, int S, int C, int decode_only, long long state_stride,
+                       const float* in_bias, const float* out_bias, cudaStream_t st) {
+    return launch_conv<float>(proj, ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions, nullptr, 0,
+                              1, 0, 0.f, 1, out, ldo, nullptr, T_tokens, S, C, 0, 0, decode_only, state_stride, st,
+                              in_bias, out_bias);
+}
+int slb_short_conv_bf16(const bf16* proj, int ldp, const float* taps_w, int taps, float* state,
+                        const int* state_slots, const int* cu_q, const int* seq_of_token, const int* positions,
+                        bf16* out, int ldo, int T_tokens, int S, int C, int decode_only, long long state_stride,
+                        const float* in_bias, const float* out_bias, cudaStream_t st) {
+    return launch_conv<bf16>(proj, ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions, nullptr, 0,
+                             1, 0, 0.f, 1, out, ldo, nullptr, T_tokens, S, C, 0, 0, decode_only, state_stride, st,
+                             in_bias, out_bias);
+}
 int slb_qk_conv_cache_f32(const float* proj, int ldp, const float* taps_w, int taps, float* state,
                           const int* state_slots, const int* cu_q, const int* seq_of_token,
                           const int* positions, const int* block_table, int max_pages, int page_size,

@@ -62,14 +62,17 @@ class ModelRunner:
         self.storage = CacheStorage(requests, num_pages, self.page_size, max_num_seqs, self.dtype,
                                     device, poison=cache_config.poison_cache)
         self.cache = CacheManager(self.storage.group_windows, num_pages, self.page_size,
-                                  max_num_seqs, reserve_pages=cache_config.reserve_blocks)
+                                  max_num_seqs, reserve_pages=cache_config.reserve_blocks,
+                                  group_chunks=self.storage.group_chunks)
         if cache_config.poison_cache:
             storage = self.storage             # (the pools must not keep the runner alive)
             for g, pool in enumerate(self.cache.pools):
                 pool.on_free = (lambda pages, g=g, storage=storage: storage.poison_pages(g, pages))
         self.num_groups = len(self.storage.groups)
         self.max_model_len = min(max_model_len or self.spec.max_position_embeddings,
-                                 self.spec.max_position_embeddings, num_pages * self.page_size)
+                                 self.spec.max_position_embeddings)
+        if groups:                        # (a model that keeps state only is not bounded by pages)
+            self.max_model_len = min(self.max_model_len, num_pages * self.page_size)
         # decode-only steps replay a CUDA graph per batch size (fixed addresses,
         # block tables padded to the longest request the engine admits)
         self.cuda_graphs = cuda_graphs
@@ -86,7 +89,7 @@ class ModelRunner:
         # only if every such mixer says that a padded step is safe for it (``padded_steps_safe``:
         # requests without tokens and tokens that belong to no request leave every record alone).
         self._padded_state_safe = all(
-            getattr(getattr(b, "mixer", None), "padded_steps_safe", False)
+            getattr(b, "padded_steps_safe", getattr(getattr(b, "mixer", None), "padded_steps_safe", False))
             for run, b in ((r, self.model.blocks[r.layer]) for r in self.spec.run_order)
             if run.cache_of is None and state_part(b.cache_request(b.spec)) is not None)
         self.graph_replays = 0

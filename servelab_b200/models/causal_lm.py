@@ -22,8 +22,10 @@ import torch
 from ..config.specs import ModelSpec
 from ..ops import kernels as K
 from ..ops.linear import linear
+from ..cache.manager import FixedStateRequest
 from ..parts import BLOCKS, NORMS, POSITIONS, BuildEnv, LayerCache, build_part, part_class
-from ..weights.source import MATRIX, TensorDecl, WeightSource
+from ..parts.norm import PendingUpdate, pending_parts
+from ..weights.source import BIAS, MATRIX, TensorDecl, WeightSource
 from ..weights.store import WeightStore
 
 
@@ -33,6 +35,11 @@ def declare_tensors(spec: ModelSpec) -> List[TensorDecl]:
                                                                   spec.embedding_position_prefix)
     if spec.embedding_norm is not None:
         out += part_class(NORMS, spec.embedding_norm).declare(spec.embedding_norm, spec.embedding_norm_prefix)
+    if spec.bigram is not None:
+        out.append(TensorDecl(spec.bigram.name, (spec.bigram.buckets + 1, spec.hidden_size), MATRIX))
+    if spec.loop is not None:
+        out += [TensorDecl(spec.loop.in_name, (spec.hidden_size, 2 * spec.hidden_size), MATRIX),
+                TensorDecl(spec.loop.step_name, (spec.loop.times, spec.hidden_size), BIAS)]
     for i, block in enumerate(spec.layers):
         out += part_class(BLOCKS, block).declare(block, spec.layer_prefix.format(i))
     out += part_class(NORMS, spec.final_norm).declare(spec.final_norm, spec.final_norm_prefix)
@@ -65,16 +72,31 @@ class CausalLM:
                                                          b.streams == spec.residual_streams for b in spec.layers):
             raise ValueError("a residual kept as several streams needs blocks of kind hyper_connections "
                              "with that many streams")
+        entries = [run.loop_entry for run in spec.run_order if run.loop_entry is not None]
+        if entries and (spec.loop is None or not all(0 <= t < spec.loop.times for t in entries)):
+            raise ValueError("a run that begins a pass of a loop needs ModelSpec.loop with that many steps")
+        if (entries or spec.bigram is not None) and spec.residual_streams is not None:
+            raise ValueError("a bigram embedding or a loop's entry together with several residual streams is not built")
+        if spec.bigram is not None and (spec.embedding_norm is not None or spec.embedding_scale is not None):
+            raise ValueError("a bigram embedding together with an embedding norm or scale is not built")
+        if entries and spec.embedding_position.kind != "none":
+            raise ValueError("a loop's entry together with positions on the embedding is not built")
+        self.loops = bool(entries)
+        self.bigram_table = self.loop_in = self.loop_step = None
         self.embed_tokens: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
 
     # ------------------------------------------------------------ caches
     def cache_requests(self) -> List[Optional[object]]:
         """Per run of the run order, what its mixer asks of the cache; None for
-        runs that read an earlier run's cache."""
-        return [part_class(BLOCKS, self.spec.layers[run.layer]).cache_request(
-                    self.spec.layers[run.layer]) if run.cache_of is None else None
-                for run in self.spec.run_order]
+        runs that read an earlier run's cache.  A bigram embedding adds one more entry: the
+        previous token of a request."""
+        out = [part_class(BLOCKS, self.spec.layers[run.layer]).cache_request(
+                   self.spec.layers[run.layer]) if run.cache_of is None else None
+               for run in self.spec.run_order]
+        if self.spec.bigram is not None:
+            out.append(FixedStateRequest((1,)))
+        return out
 
     # ----------------------------------------------------------- weights
     def load(self, source: WeightSource) -> None:
@@ -85,6 +107,11 @@ class CausalLM:
         self.embedding_position.load(store)
         if self.embedding_norm is not None:
             self.embedding_norm.load(store)
+        if self.spec.bigram is not None:
+            self.bigram_table = store.get(self.spec.bigram.name)
+        if self.spec.loop is not None:
+            self.loop_in = store.get(self.spec.loop.in_name)
+            self.loop_step = store.get(self.spec.loop.step_name)
         for b in self.blocks:
             b.load(store)
         self.final_norm.load(store)
@@ -105,7 +132,7 @@ class CausalLM:
         for b in self.blocks:
             walk(b)
         walk(self.final_norm)
-        for t in (self.embed_tokens, self.lm_head):
+        for t in (self.embed_tokens, self.lm_head, self.bigram_table, self.loop_in, self.loop_step):
             if t is not None and t.data_ptr() not in seen:
                 seen.add(t.data_ptr())
                 total += t.numel() * t.element_size()
@@ -119,7 +146,15 @@ class CausalLM:
         n = self.spec.residual_streams
         shape = (T, self.spec.hidden_size) if n is None else (T, n, self.spec.hidden_size)
         resid = torch.empty(shape, dtype=torch.float32, device=self.env.device)
-        if self.embedding_norm is None and n is None:
+        w = self.spec.hidden_size
+        both = None                            # [x | x0] in the compute type: what a pass of a loop begins with
+        if self.loops:
+            both = torch.empty((T, 2 * w), dtype=self.env.dtype, device=self.env.device)
+        if self.spec.bigram is not None:
+            b = self.spec.bigram
+            K.embed_bigram(ctx, self.embed_tokens, self.bigram_table, b.buckets, b.mul_prev, b.mul_cur,
+                           caches[len(self.spec.run_order)].state, resid, None if both is None else both[:, w:])
+        elif self.embedding_norm is None and n is None:
             K.embedding(ctx.token_ids, self.embed_tokens, resid,
                         1.0 if self.spec.embedding_scale is None else self.spec.embedding_scale)
         else:
@@ -129,11 +164,20 @@ class CausalLM:
             norm = self.embedding_norm
             K.embed_norm_streams(ctx.token_ids, self.embed_tokens, None if norm is None else norm.weight,
                                  0.0 if norm is None else norm.spec.eps, resid)
+        if self.loops and self.spec.bigram is None:
+            K.stream_rows(resid, (), None, both[:, w:])
         self.embedding_position.apply_to_embedding(ctx, resid)
         delta = None
         for i, run in enumerate(self.spec.run_order):
             owner = i if run.cache_of is None else run.cache_of
             block = self.blocks[run.layer]
+            if run.loop_entry is not None:
+                # x <- W_in [x; x0] (float32 results); the step's vector is added with the next update
+                K.stream_rows(resid, *pending_parts(delta), both[:, :w])
+                resid = linear(both, self.loop_in, out_dtype=torch.float32)
+                delta = PendingUpdate((), self.loop_step[run.loop_entry])
+                if not getattr(block, "accepts_pending_update", False):
+                    resid, delta = resid + delta.row, None
             # (an update may travel as the partial sums of a K-split product; a block that
             # does not say it accepts that form gets the plain tensor)
             resid, delta = block.forward(ctx, resid, K.plain_unless(block, delta), caches[owner],

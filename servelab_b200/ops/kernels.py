@@ -351,20 +351,21 @@ def qk_conv_cache(proj: torch.Tensor, taps_w: torch.Tensor, state: Optional[torc
 
 
 def short_conv(proj: torch.Tensor, taps_w: torch.Tensor, state: Optional[torch.Tensor], ctx,
-               out: torch.Tensor) -> None:
+               out: torch.Tensor, in_bias: Optional[torch.Tensor] = None,
+               out_bias: Optional[torch.Tensor] = None) -> None:
     """The convolution alone: y_t = sum_i taps_w[i] u_(t - taps + 1 + i) on the first C = out.shape[1]
     columns of ``proj`` into ``out`` [T, C]; the rows before a portion come from ``state`` (float32
     [slots, >= (taps - 1) * C], a request's record at ``ctx.state_slots``; rows of the record may be
     ``state.stride(0)`` apart, so it can be a slice of a larger record), which is left holding the
-    last taps - 1 projected rows."""
-    fn = getattr(L.core(), "slb_qk_conv_cache_" + _suffix(proj.dtype))
+    last taps - 1 projected rows.  ``in_bias`` / ``out_bias`` float32 [C]: added to the projected rows
+    (and so part of the record) / to the result."""
+    fn = getattr(L.core(), "slb_short_conv_" + _suffix(proj.dtype))
     n = 1 if (taps_w.shape[0] == 1 or ctx.decode_only) else 2
     L.check(fn(proj.data_ptr(), proj.stride(0), taps_w.data_ptr(), taps_w.shape[0], _p(state),
                ctx.state_slots.data_ptr(), ctx.cu_q.data_ptr(), ctx.seq_of_token.data_ptr(),
-               ctx.positions.data_ptr(), None, 0, 1, 0, 0.0, 1, out.data_ptr(), out.stride(0),
-               None, proj.shape[0], ctx.num_seqs, out.shape[1], 0, 0,
-               1 if ctx.decode_only else 0, state.stride(0) if state is not None else 0, _stream()),
-            "short_conv")
+               ctx.positions.data_ptr(), out.data_ptr(), out.stride(0), proj.shape[0], ctx.num_seqs, out.shape[1],
+               1 if ctx.decode_only else 0, state.stride(0) if state is not None else 0, _p(in_bias), _p(out_bias),
+               _stream()), "short_conv")
     global launch_count
     launch_count += n - 1
 
@@ -932,12 +933,15 @@ def attention_kv_status(reset: bool = False) -> int:
 def attention_kv(ctx, q, k_cache, v_cache, v_row_stride: int, out, block_table, num_heads: int,
                  num_kv_heads: int, k_dim: int, v_dim: int, page_size: int, scale: float, window: int,
                  head_gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                 sink: Optional[torch.Tensor] = None) -> None:
+                 sink: Optional[torch.Tensor] = None, chunk: int = 0,
+                 sigmoid_bias: Optional[torch.Tensor] = None) -> None:
     """The plain kernel: float32 arithmetic; keys of ``k_dim``, values of ``v_dim`` elements at
     ``v_cache`` with rows ``v_row_stride`` apart (the key cache itself for values that are a
     prefix of the keys); ``head_gate`` [T, >= H]: head h's row times sigmoid(head_gate[t, h]);
     ``softcap`` > 0: a scaled score s becomes softcap tanh(s / softcap); ``sink`` float32 [H]: its
-    exponential joins the softmax's denominator."""
+    exponential joins the softmax's denominator; ``chunk`` > 0 (instead of ``window``): a query at i sees
+    the keys j <= i with j // chunk == i // chunk; ``sigmoid_bias`` float32 [H] (instead of the
+    softmax): a visible key's weight is sigmoid(score + sigmoid_bias[h]), not normalized."""
     tile_seq, tile_row0, n = ctx.attention_tiles(num_heads // num_kv_heads, attention_kv_tile_rows())
     fn = getattr(L.core(), "slb_attention_kv_" + _suffix(q.dtype))
     L.check(fn(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), v_row_stride,
@@ -945,7 +949,7 @@ def attention_kv(ctx, q, k_cache, v_cache, v_row_stride: int, out, block_table, 
                ctx.cu_q.data_ptr(), ctx.ctx_len.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), n,
                num_heads, num_kv_heads, k_dim, v_dim, page_size, k_cache.shape[0], float(scale),
                int(window), _p(head_gate), head_gate.stride(0) if head_gate is not None else 0,
-               float(softcap), _p(sink), _stream()), "attention_kv")
+               float(softcap), _p(sink), int(chunk), _p(sigmoid_bias), _stream()), "attention_kv")
 
 
 def attention_kv_splits(num_seqs: int, num_kv_heads: int, longest_context: int, window: int,
@@ -979,17 +983,21 @@ def attention_kv_resident(lib, k_dim: int, v_dim: int, narrow: bool, group: int)
 def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num_heads: int,
                      num_kv_heads: int, k_dim: int, v_dim: int, page_size: int, scale: float, window: int,
                      head_gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                     sink: Optional[torch.Tensor] = None) -> None:
+                     sink: Optional[torch.Tensor] = None, chunk: int = 0,
+                     sigmoid_bias: Optional[torch.Tensor] = None) -> None:
     """The tensor-core kernel (bfloat16), for prompt portions and single tokens; in a step of
     single tokens the keys of a request are split over several blocks when the requests alone
-    would not fill the device.  ``softcap`` and ``sink`` as in ``attention_kv``."""
+    would not fill the device.  ``softcap``, ``sink``, ``chunk`` and ``sigmoid_bias`` as in
+    ``attention_kv``."""
     lib = L.attention_kv(k_dim, v_dim)
     rows = lib.slb_attention_kv_mma_tile_rows()
     tile_seq, tile_row0, n = ctx.attention_tiles(num_heads // num_kv_heads, rows)
     splits, part_o, part_ml = 1, None, None
     if ctx.decode_only and attention_kv_split and num_heads // num_kv_heads <= rows:
         narrow = attention_kv_narrow and num_heads // num_kv_heads <= 16
-        splits = attention_kv_splits(ctx.num_seqs, num_kv_heads, ctx.split_hint_len, window,
+        # (a chunk's keys fill up from its start: at most ``chunk`` of them, half on average)
+        splits = attention_kv_splits(ctx.num_seqs, num_kv_heads,
+                                     min(ctx.split_hint_len, chunk) if chunk else ctx.split_hint_len, window,
                                      max_splits=lib.slb_attention_kv_mma_max_splits(),
                                      resident=attention_kv_resident(lib, k_dim, v_dim, narrow,
                                                                     num_heads // num_kv_heads))
@@ -1003,9 +1011,9 @@ def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num
             page_size, k_cache.shape[0], float(scale), int(window), _p(head_gate),
             head_gate.stride(0) if head_gate is not None else 0, splits, _p(part_o), _p(part_ml),
             1 if ctx.decode_only and attention_kv_narrow and num_heads // num_kv_heads <= 16 else 0)
-    if softcap or sink is not None:
-        L.check(lib.slb_attention_kv_mma_capped_bf16(*args, float(softcap or 0.0), _p(sink), _stream()),
-                "attention_kv_mma")
+    if softcap or sink is not None or chunk or sigmoid_bias is not None:
+        L.check(lib.slb_attention_kv_mma_capped_bf16(*args, float(softcap or 0.0), _p(sink), int(chunk),
+                                                     _p(sigmoid_bias), _stream()), "attention_kv_mma")
         return
     L.check(lib.slb_attention_kv_mma_bf16(*args, _stream()), "attention_kv_mma")
 
@@ -1041,10 +1049,11 @@ def attention_kv_tc_takes(k_dim: int, v_dim: int, page_size: int, group: int, ti
 def attention_kv_tc(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num_heads: int,
                     num_kv_heads: int, k_dim: int, v_dim: int, page_size: int, scale: float, window: int,
                     head_gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                    sink: Optional[torch.Tensor] = None) -> None:
+                    sink: Optional[torch.Tensor] = None, chunk: int = 0,
+                    sigmoid_bias: Optional[torch.Tensor] = None) -> None:
     """The tcgen05 kernel (bfloat16; key and value sizes multiples of 64; steps with prompt
-    portions): 128 flattened rows a block, accumulators in tensor memory.  ``softcap`` and ``sink``
-    as in ``attention_kv``."""
+    portions): 128 flattened rows a block, accumulators in tensor memory.  ``softcap``, ``sink``,
+    ``chunk`` and ``sigmoid_bias`` as in ``attention_kv``."""
     lib = L.attention_kv(k_dim, v_dim)
     group = num_heads // num_kv_heads
     tile_seq, tile_row0, n = ctx.attention_tiles(group, lib.slb_attention_kv_tc_tile_rows(group))
@@ -1053,9 +1062,9 @@ def attention_kv_tc(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num_
             ctx.ctx_len.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), n, num_heads, num_kv_heads,
             page_size, k_cache.shape[0], float(scale), int(window), _p(head_gate),
             head_gate.stride(0) if head_gate is not None else 0)
-    if softcap or sink is not None:
-        L.check(lib.slb_attention_kv_tc_capped_bf16(*args, float(softcap or 0.0), _p(sink), _stream()),
-                "attention_kv_tc")
+    if softcap or sink is not None or chunk or sigmoid_bias is not None:
+        L.check(lib.slb_attention_kv_tc_capped_bf16(*args, float(softcap or 0.0), _p(sink), int(chunk),
+                                                    _p(sigmoid_bias), _stream()), "attention_kv_tc")
         return
     L.check(lib.slb_attention_kv_tc_bf16(*args, _stream()), "attention_kv_tc")
 
@@ -1089,7 +1098,8 @@ def gemm_simt_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> No
     any row stride; the last dimension contiguous), on CUDA cores with float32 accumulation."""
     M, B, Kd = a.shape
     N = w.shape[1]
-    fn = getattr(L.core(), "slb_gemm_simt_batched_" + _suffix(a.dtype))
+    kind = "bf16_f32out" if a.dtype == _BF16 and out.dtype == _F32 else _suffix(a.dtype)
+    fn = getattr(L.core(), "slb_gemm_simt_batched_" + kind)
     L.check(fn(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(1), out.data_ptr(), out.stride(0),
                M, N, Kd, B, a.stride(1), w.stride(0), out.stride(1), _stream()), "gemm_simt_batched")
 
@@ -1309,7 +1319,11 @@ class _DecayAttnArgs(_ct.Structure):
         ("out", _ct.c_void_p), ("ldo", _ct.c_int),
         ("gate_z", _ct.c_void_p), ("ld_gate", _ct.c_int), ("gate_bias", _ct.c_void_p),
         ("gate_inv_tau", _ct.c_float), ("q_scale", _ct.c_float), ("state_stride", _ct.c_longlong),
+        ("gate_kind", _ct.c_int), ("bonus", _ct.c_void_p),
     ]
+
+
+DECAY_GATE_KINDS = {"sigmoid_root": 0, "exp_exp": 1}
 
 
 class _DecayChunkArgs(_ct.Structure):
@@ -1346,13 +1360,16 @@ def decay_attention(proj: torch.Tensor, ctx, state: torch.Tensor, decay: Optiona
                     q_off: int, k_off: int, v_off: int, num_heads: int, head_dim: int, value_dim: int,
                     activation: Optional[str] = None, freq: Optional[torch.Tensor] = None, rot_dims: int = 0,
                     key_scale: float = 1.0, query_scale: float = 1.0, gate_z: Optional[torch.Tensor] = None,
-                    gate_bias: Optional[torch.Tensor] = None, gate_tau: float = 1.0) -> None:
+                    gate_bias: Optional[torch.Tensor] = None, gate_tau: float = 1.0,
+                    gate_kind: str = "sigmoid_root", bonus: Optional[torch.Tensor] = None) -> None:
     """o_t = S_t^T q_t with S_t = decay_h S_{t-1} + k_t v_t^T per head over the tokens of every request
     of the step, in order; q, k, v are columns of ``proj`` [T, ...]; ``state`` float32
     [slots, H, D, Dv] (or [slots, >= H * D * Dv]: a slice of a larger record) is read at
     ``ctx.state_slots`` and left advanced; ``out`` float32 [T, H * Dv].  With ``gate_z`` (float32
     [T, H * D]; ``decay`` None) every key channel of every token has its own decay
-    sigmoid(gate_z + gate_bias)^(1 / gate_tau): S_t = diag(alpha_t) S_{t-1} + k_t v_t^T."""
+    sigmoid(gate_z + gate_bias)^(1 / gate_tau): S_t = diag(alpha_t) S_{t-1} + k_t v_t^T; ``gate_kind``
+    "exp_exp": exp(-exp(gate_z + gate_bias)).  ``bonus`` float32 [H * D] (learned decays only): the result
+    reads the state before the token, o_t = (S_{t-1} + diag(bonus) k_t v_t^T)^T q_t."""
     a = _DecayAttnArgs()
     a.proj, a.ld = proj.data_ptr(), proj.stride(0)
     a.q_off, a.k_off, a.v_off = q_off, k_off, v_off
@@ -1366,6 +1383,7 @@ def decay_attention(proj: torch.Tensor, ctx, state: torch.Tensor, decay: Optiona
     a.gate_z, a.ld_gate = _p(gate_z), (gate_z.stride(0) if gate_z is not None else 0)
     a.gate_bias, a.gate_inv_tau, a.q_scale = _p(gate_bias), 1.0 / float(gate_tau), float(query_scale)
     a.state_stride = state.stride(0)
+    a.gate_kind, a.bonus = DECAY_GATE_KINDS[gate_kind], _p(bonus)
     if gate_z is not None and gate_z.dtype != _F32:
         raise L.KernelError("decay_attention: the decays' logits must be float32")
     plain = (gate_z is None and query_scale == 1.0
@@ -1468,3 +1486,198 @@ def attention_kv_mma_maps(ctx, q, k_cache, v_cache, out, block_table, num_heads:
         float(scale), int(window), splits, _p(part_o), _p(part_ml),
         1 if ctx.decode_only and attention_kv_narrow and num_heads // num_kv_heads <= 16 else 0, _stream()),
         "attention_kv_mma")
+
+
+# ------------------------------- two sublayers on one stream behind Dynamic Tanh norms
+class _DytParallelArgs(_ct.Structure):
+    _fields_ = [
+        ("resid", _ct.c_void_p), ("ldr", _ct.c_int),
+        ("d1", _ct.c_void_p), ("ldd1", _ct.c_int), ("d2", _ct.c_void_p), ("ldd2", _ct.c_int), ("d_is_f32", _ct.c_int),
+        ("row", _ct.c_void_p),
+        ("resid_out", _ct.c_void_p), ("ldx", _ct.c_int),
+        ("alpha1", _ct.c_void_p), ("w1", _ct.c_void_p), ("b1", _ct.c_void_p), ("out1", _ct.c_void_p), ("ldo1", _ct.c_int),
+        ("shift", _ct.c_void_p),
+        ("alpha2", _ct.c_void_p), ("w2", _ct.c_void_p), ("b2", _ct.c_void_p), ("out2", _ct.c_void_p), ("ldo2", _ct.c_int),
+        ("prev", _ct.c_void_p), ("prev_stride", _ct.c_longlong), ("num_slots", _ct.c_int),
+        ("cu_q", _ct.c_void_p), ("seq_of_token", _ct.c_void_p), ("state_slots", _ct.c_void_p),
+        ("row_map", _ct.c_void_p), ("rows", _ct.c_int), ("dim", _ct.c_int),
+    ]
+
+
+def _stream_args(resid, terms, row):
+    if len(terms) > 2:
+        raise L.KernelError("at most two pending updates")
+    a = _DytParallelArgs()
+    a.resid, a.ldr, a.dim = resid.data_ptr(), resid.stride(0), resid.shape[1]
+    for i, t in enumerate(terms):
+        setattr(a, f"d{i + 1}", t.data_ptr())
+        setattr(a, f"ldd{i + 1}", t.stride(0))
+        if t.dtype == _F32:
+            a.d_is_f32 |= 1 << i
+    a.row = _p(row)
+    return a
+
+
+def dyt_parallel(ctx, resid: torch.Tensor, terms, row: Optional[torch.Tensor], norm1, out1: torch.Tensor,
+                 norm2=None, out2: Optional[torch.Tensor] = None, resid_out: Optional[torch.Tensor] = None,
+                 shift: Optional[torch.Tensor] = None, prev: Optional[torch.Tensor] = None,
+                 row_map: Optional[torch.Tensor] = None) -> None:
+    """x = resid (+ the pending ``terms``, up to two [T, w], + ``row`` [w]); out1 = dyt_1(x), mixed with the
+    previous token's by ``shift`` [w]: n + (n_prev - n) * shift; out2 = dyt_2(x); x into
+    ``resid_out``.  ``norm1`` / ``norm2``: (alpha, weight, bias) float32.  ``prev`` float32 [slots, >= w]
+    holds a request's last n at ``ctx.state_slots`` and is left advanced.  ``row_map``: only these
+    rows (no shift, no ``resid_out``)."""
+    a = _stream_args(resid, terms, row)
+    a.alpha1, a.w1, a.b1 = (t.data_ptr() for t in norm1)
+    a.out1, a.ldo1 = out1.data_ptr(), out1.stride(0)
+    if out2 is not None:
+        a.alpha2, a.w2, a.b2 = (t.data_ptr() for t in norm2)
+        a.out2, a.ldo2 = out2.data_ptr(), out2.stride(0)
+    if resid_out is not None:
+        a.resid_out, a.ldx = resid_out.data_ptr(), resid_out.stride(0)
+    if shift is not None:
+        a.shift, a.prev, a.prev_stride, a.num_slots = shift.data_ptr(), prev.data_ptr(), prev.stride(0), prev.shape[0]
+        a.cu_q, a.seq_of_token = ctx.cu_q.data_ptr(), ctx.seq_of_token.data_ptr()
+        a.state_slots = ctx.state_slots.data_ptr()
+    a.row_map, a.rows = _p(row_map), (resid.shape[0] if row_map is None else row_map.numel())
+    fn = getattr(L.core(), "slb_dyt_parallel_" + _suffix(out1.dtype))
+    L.check(fn(_ct.byref(a), _stream()), "dyt_parallel")
+
+
+def stream_rows(resid: torch.Tensor, terms, row: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """out = resid (+ pending ``terms`` + ``row``) in ``out``'s type ([T, w], any row stride)."""
+    a = _stream_args(resid, terms, row)
+    a.out1, a.ldo1, a.rows = out.data_ptr(), out.stride(0), resid.shape[0]
+    fn = getattr(L.core(), "slb_stream_rows_" + _suffix(out.dtype))
+    L.check(fn(_ct.byref(a), _stream()), "stream_rows")
+
+
+# ------------------------------------------------- a token and the one before it
+def embed_bigram(ctx, table: torch.Tensor, pairs: torch.Tensor, buckets: int, mul_prev: int, mul_cur: int,
+                 state: torch.Tensor, out: torch.Tensor, copy: Optional[torch.Tensor] = None) -> None:
+    """out[t] = table[id] + pairs[(previous id * mul_prev + id * mul_cur) mod buckets] (row ``buckets`` for a
+    sequence's first token) as float32; ``copy`` [T, w] (a view): the same in the table's type.
+    ``state`` [slots, 1]: the id of a request's last token plus one, as an integer."""
+    fn = getattr(L.core(), "slb_embed_bigram_" + _suffix(table.dtype))
+    L.check(fn(ctx.token_ids.data_ptr(), ctx.cu_q.data_ptr(), ctx.seq_of_token.data_ptr(), ctx.state_slots.data_ptr(),
+               state.data_ptr(), state.stride(0), state.shape[0], table.data_ptr(), table.shape[0], pairs.data_ptr(),
+               int(buckets), int(mul_prev), int(mul_cur), out.data_ptr(), _p(copy),
+               copy.stride(0) if copy is not None else 0, out.shape[0], table.shape[1], _stream()), "embed_bigram")
+
+
+def token_mix(ctx, x: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, out: torch.Tensor) -> None:
+    """out[i] = x + (x_prev - x) * mu[i] for the vectors ``mu`` float32 [n, w]; out [n, T, w].  ``prev`` float32
+    [slots, >= w]: the last row of a request, left advanced."""
+    fn = getattr(L.core(), "slb_token_mix_" + _suffix(x.dtype))
+    L.check(fn(x.data_ptr(), x.stride(0), mu.data_ptr(), mu.shape[0], prev.data_ptr(), prev.stride(0), prev.shape[0],
+               ctx.cu_q.data_ptr(), ctx.seq_of_token.data_ptr(), ctx.state_slots.data_ptr(), out.data_ptr(),
+               x.shape[1], x.shape[0], _stream()), "token_mix")
+
+
+def tanh_linear(low: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """out = tanh(low) . w^T (+ bias), float32 results: the second product of a bottleneck."""
+    fn = getattr(L.core(), "slb_gemm_simt_tanh_" + _suffix(low.dtype))
+    L.check(fn(low.data_ptr(), low.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _p(bias),
+               low.shape[0], w.shape[0], w.shape[1], _stream()), "tanh_linear")
+
+
+# ------------------------------------------------------------------ delta rule
+class _DeltaRuleArgs(_ct.Structure):
+    _fields_ = [
+        ("proj", _ct.c_void_p), ("ld", _ct.c_int),
+        ("r_off", _ct.c_int), ("k_off", _ct.c_int), ("v_off", _ct.c_int), ("a_off", _ct.c_int),
+        ("H", _ct.c_int), ("D", _ct.c_int), ("Dv", _ct.c_int),
+        ("a_bias", _ct.c_void_p),
+        ("gate_z", _ct.c_void_p), ("ld_gate", _ct.c_int), ("decay_coef", _ct.c_float), ("unit_eps", _ct.c_float),
+        ("cu_q", _ct.c_void_p), ("state_slots", _ct.c_void_p),
+        ("state", _ct.c_void_p), ("num_slots", _ct.c_int), ("state_stride", _ct.c_longlong),
+        ("out", _ct.c_void_p), ("ldo", _ct.c_int),
+        ("out_t", _ct.c_void_p), ("ldt", _ct.c_int), ("g_off", _ct.c_int), ("norm_w", _ct.c_void_p),
+        ("norm_eps", _ct.c_float),
+    ]
+
+
+class _DeltaChunkArgs(_ct.Structure):
+    _fields_ = [("a", _DeltaRuleArgs), ("tile_seq", _ct.c_void_p), ("tile_row0", _ct.c_void_p),
+                ("num_tiles", _ct.c_int), ("work", _ct.c_void_p)]
+
+
+# Steps with portions of prompts in bfloat16 take the chunked kernels from this many tokens a request on
+# (shorter portions, single tokens and float32: the token-by-token kernel).
+delta_rule_chunked = True
+force_delta_chunks = False       # (tests: the chunked kernels also for float32 rows)
+delta_rule_chunk_min_tokens = 16
+
+
+def delta_rule(ctx, proj: torch.Tensor, state: torch.Tensor, out: torch.Tensor, *, r_off: int, k_off: int, v_off: int,
+               a_off: int, g_off: int, num_heads: int, head_dim: int, value_dim: int, a_bias: torch.Tensor,
+               gate_z: torch.Tensor, decay_coef: float, unit_eps: float, norm_w: torch.Tensor, norm_eps: float) -> None:
+    """The recurrence of ``DeltaRuleSpec`` over the tokens of every request of the step, in order, then the
+    head norm times ``norm_w`` times sigmoid(gate) into ``out`` [T, H * Dv]; r, k, v, a and the gate
+    are columns of ``proj``; ``gate_z`` float32 [T, H * D]; ``state`` float32 [slots, >= H * D * Dv] is left
+    advanced."""
+    a = _DeltaRuleArgs()
+    a.proj, a.ld = proj.data_ptr(), proj.stride(0)
+    a.r_off, a.k_off, a.v_off, a.a_off = r_off, k_off, v_off, a_off
+    a.H, a.D, a.Dv = num_heads, head_dim, value_dim
+    a.a_bias = a_bias.data_ptr()
+    a.gate_z, a.ld_gate, a.decay_coef, a.unit_eps = gate_z.data_ptr(), gate_z.stride(0), float(decay_coef), float(unit_eps)
+    a.cu_q, a.state_slots = ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr()
+    a.state, a.num_slots, a.state_stride = state.data_ptr(), state.shape[0], state.stride(0)
+    lib, suffix = L.core(), _suffix(proj.dtype)
+    chunked = (not ctx.decode_only and decay_coef <= 2.0
+               and ctx.num_tokens >= delta_rule_chunk_min_tokens * ctx.num_seqs
+               and (force_delta_chunks or (delta_rule_chunked and proj.dtype == _BF16)))
+    if not chunked and lib.slb_delta_rule_fuses(head_dim, value_dim):
+        a.out_t, a.ldt, a.g_off = out.data_ptr(), out.stride(0), g_off
+        a.norm_w, a.norm_eps = norm_w.data_ptr(), float(norm_eps)
+        L.check(getattr(lib, "slb_delta_rule_" + suffix)(_ct.byref(a), ctx.num_seqs, _stream()), "delta_rule")
+        return
+    o = torch.empty((proj.shape[0], num_heads * value_dim), dtype=_F32, device=proj.device)
+    a.out, a.ldo = o.data_ptr(), o.stride(0)
+    if chunked:
+        tile_seq, tile_row0, n = ctx.attention_tiles(1, lib.slb_delta_chunk_tokens())
+        work = torch.empty((max(n, 1), num_heads, lib.slb_delta_chunk_work_floats(head_dim)), dtype=_F32,
+                           device=proj.device)
+        c = _DeltaChunkArgs()
+        c.a = a
+        c.tile_seq, c.tile_row0, c.num_tiles, c.work = tile_seq.data_ptr(), tile_row0.data_ptr(), n, work.data_ptr()
+        L.check(getattr(lib, "slb_delta_chunk_" + suffix)(_ct.byref(c), ctx.num_seqs, _stream()), "delta_rule (chunks)")
+        global launch_count
+        launch_count += 1
+    else:
+        L.check(getattr(lib, "slb_delta_rule_" + suffix)(_ct.byref(a), ctx.num_seqs, _stream()), "delta_rule")
+    group_norm_gate(o, num_heads, value_dim, out, eps=norm_eps, weight=norm_w,
+                    gate=proj[:, g_off:g_off + num_heads * value_dim], gate_activation="sigmoid")
+
+
+# --------------------------------------------------- gated linear recurrence (a number a channel)
+class _GatedRecArgs(_ct.Structure):
+    _fields_ = [
+        ("u", _ct.c_void_p), ("ldu", _ct.c_int),
+        ("z", _ct.c_void_p), ("z_block", _ct.c_longlong), ("z_token", _ct.c_longlong),
+        ("r_bias", _ct.c_void_p), ("i_bias", _ct.c_void_p), ("rate", _ct.c_void_p),
+        ("y", _ct.c_void_p), ("ldy", _ct.c_int), ("y_bias", _ct.c_void_p),
+        ("state", _ct.c_void_p), ("state_stride", _ct.c_longlong), ("num_slots", _ct.c_int),
+        ("cu_q", _ct.c_void_p), ("state_slots", _ct.c_void_p),
+        ("width", _ct.c_int), ("n", _ct.c_int),
+        ("out", _ct.c_void_p), ("ldo", _ct.c_int),
+    ]
+
+
+def gated_recurrence(ctx, u: torch.Tensor, z: torch.Tensor, y: torch.Tensor, state: torch.Tensor, out: torch.Tensor, *,
+                     r_bias: torch.Tensor, i_bias: torch.Tensor, rate: torch.Tensor, y_bias: torch.Tensor) -> None:
+    """S_t = a S_{t-1} + sqrt(1 - a^2) i u with log a = rate * r per channel, out = S * gelu_tanh(y + y_bias)
+    over the tokens of every request, in order; ``z`` float32 [blocks, T, 2 n]: the logits of r, then
+    of i; ``state`` float32 [slots, >= width], left advanced."""
+    g = _GatedRecArgs()
+    g.u, g.ldu = u.data_ptr(), u.stride(0)
+    g.z, g.z_block, g.z_token = z.data_ptr(), z.stride(0), z.stride(1)
+    g.r_bias, g.i_bias, g.rate = r_bias.data_ptr(), i_bias.data_ptr(), rate.data_ptr()
+    g.y, g.ldy, g.y_bias = y.data_ptr(), y.stride(0), y_bias.data_ptr()
+    g.state, g.state_stride, g.num_slots = state.data_ptr(), state.stride(0), state.shape[0]
+    g.cu_q, g.state_slots = ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr()
+    g.width, g.n = out.shape[1], z.shape[2] // 2
+    g.out, g.ldo = out.data_ptr(), out.stride(0)
+    fn = getattr(L.core(), "slb_gated_recurrence_" + _suffix(out.dtype))
+    L.check(fn(_ct.byref(g), ctx.num_seqs, _stream()), "gated_recurrence")

@@ -69,10 +69,34 @@ _CORE_SIGNATURES = {
     "slb_sigmoid_gate_bf16": [P, I, P, I, P, I, I, I, I, P],
     "slb_attention_kv_tile_rows": [],
     "slb_attention_kv_status": [I],
-    "slb_attention_kv_f32": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, P],
-    "slb_attention_kv_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, P],
+    "slb_attention_kv_f32": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, I, P, P],
+    "slb_attention_kv_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, I, P, P],
     "slb_gemm_simt_batched_f32": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
     "slb_gemm_simt_batched_bf16": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
+    "slb_gemm_simt_batched_bf16_f32out": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
+    "slb_gemm_simt_tanh_f32": [P, I, P, I, P, I, P, I, I, I, P],
+    "slb_gemm_simt_tanh_bf16": [P, I, P, I, P, I, P, I, I, I, P],
+    "slb_dyt_parallel_f32": [P, P],
+    "slb_dyt_parallel_bf16": [P, P],
+    "slb_stream_rows_f32": [P, P],
+    "slb_stream_rows_bf16": [P, P],
+    "slb_short_conv_f32": [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, LL, P, P, P],
+    "slb_short_conv_bf16": [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, LL, P, P, P],
+    "slb_token_mix_max": [],
+    "slb_embed_bigram_f32": [P, P, P, P, P, LL, I, P, I, P, LL, LL, LL, P, P, I, I, I, P],
+    "slb_embed_bigram_bf16": [P, P, P, P, P, LL, I, P, I, P, LL, LL, LL, P, P, I, I, I, P],
+    "slb_token_mix_f32": [P, I, P, I, P, LL, I, P, P, P, P, I, I, P],
+    "slb_token_mix_bf16": [P, I, P, I, P, LL, I, P, P, P, P, I, I, P],
+    "slb_delta_rule_max_dim": [],
+    "slb_delta_rule_fuses": [I, I],
+    "slb_delta_rule_f32": [P, I, P],
+    "slb_delta_rule_bf16": [P, I, P],
+    "slb_delta_chunk_tokens": [],
+    "slb_delta_chunk_work_floats": [I],
+    "slb_delta_chunk_f32": [P, I, P],
+    "slb_delta_chunk_bf16": [P, I, P],
+    "slb_gated_recurrence_f32": [P, I, P],
+    "slb_gated_recurrence_bf16": [P, I, P],
     "slb_moe_tile_rows": [],
     "slb_moe_route": [P, I, I, I, I, I, I, F, I, P, P, P],
     "slb_moe_route_scored": [P, I, I, I, I, I, I, F, I, I, P, I, F, P, P, P],
@@ -268,7 +292,7 @@ _ATTN_KV_SIGNATURES = {
     "slb_attention_kv_mma_status": [I],
     "slb_attention_kv_mma_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, I, P, P, I, P],
     "slb_attention_kv_mma_capped_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, I, P, P, I,
-                                         F, P, P],
+                                         F, P, I, P, P],
     "slb_attention_kv_mma_max_splits": [],
     "slb_attention_kv_mma_resident": [I, I],
     "slb_attention_kv_mma_maps_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, I, P, P, I, P],
@@ -278,7 +302,8 @@ _ATTN_KV_SIGNATURES = {
     "slb_attention_kv_tc_status": [I],
     "slb_attention_kv_tc_where": [P],
     "slb_attention_kv_tc_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, P],
-    "slb_attention_kv_tc_capped_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, F, P, P],
+    "slb_attention_kv_tc_capped_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, F, P, I, P,
+                                        P],
     "slb_attention_kv_tc_maps_bf16": [P, I, P, P, P, I, P, I, P, P, P, P, I, I, I, I, I, I, F, I, P],
 }
 

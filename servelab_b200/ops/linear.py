@@ -217,3 +217,18 @@ def batched_head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> 
 
 
 use_vendor_batched = True
+
+
+def block_diagonal_logits(u: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """z[b, t] = w[b] . u[t, part b] for w [blocks, m, n] and u [T, blocks * n]: float32 [blocks, T, m].
+    bfloat16 with rows of whole 16-byte pieces: the vendor's batched product; otherwise this package's
+    CUDA-core kernel."""
+    blocks, m, n = w.shape
+    T = u.shape[0]
+    if u.dtype == torch.bfloat16 and n % 8 == 0 and m % 8 == 0 and u.stride(0) % 8 == 0 and T > 0:
+        z = torch.bmm(u.unflatten(1, (blocks, n)).transpose(0, 1), w.transpose(1, 2), out_dtype=torch.float32)
+        _mark("library gemm")
+        return z
+    z = torch.empty((blocks, T, m), dtype=torch.float32, device=u.device)
+    K.gemm_simt_batched(u.unflatten(1, (blocks, n)), w, z.transpose(0, 1))
+    return z

@@ -72,6 +72,16 @@ class LayerCache:
     state: Optional[torch.Tensor] = None
     page_size: int = 0
 
+    def with_state_slice(self, start: int, floats: int) -> "LayerCache":
+        """The same cache with ``floats`` floats of every record from ``start`` on as its state (None for
+        0 floats): what a part of a composed mixer or block sees.  The rows of the slice are the
+        whole record's length apart."""
+        state = None
+        if floats:
+            flat = self.state if self.state.dim() == 2 else self.state.view(self.state.shape[0], -1)
+            state = flat[:, start:start + floats]
+        return LayerCache(group=self.group, k=self.k, v=self.v, state=state, page_size=self.page_size)
+
 
 class Part:
     # True iff forward() only launches kernels on device buffers of the step

@@ -9,10 +9,11 @@ happens inside the next norm kernel.
 
 from __future__ import annotations
 
+from ..cache.manager import FixedStateRequest, paged_part, record_floats
 from ..ops.kernels import plain_unless
 from .base import Block
 from ..weights.source import BIAS, MIXING, TensorDecl
-from .norm import HyperPending, PostNormed
+from .norm import HyperPending, PendingUpdate, PostNormed
 from .registry import FEED_FORWARDS, MIXERS, NORMS, build_part, part_class, register_block
 
 
@@ -252,6 +253,75 @@ class HyperConnectionsBlock(Block):
         read, mix, out_w = self.hyper[1]
         x = self.ff_norm.read_streams(ctx, streams, pending, read)
         return streams, HyperPending(self.feed_forward.forward(ctx, x), mix, out_w)
+
+
+@register_block("parallel_norm")
+class ParallelNormBlock(Block):
+    """x += mixer(shift(norm1(x))) + ff(norm2(x)): both sublayers read the same stream, each behind a
+    norm of its own.  ``token_shift``: the mixer's input h becomes h + (h' - h) * shift with the
+    previous token's h' (before this; zeros for a sequence's first); a request's last h is part of its
+    state record, in front of the mixer's own.  Both results travel as one ``PendingUpdate`` to the
+    kernel that prepares the next reader's inputs.  ``feed_forward`` None: the mixer alone."""
+    accepts_pending_update = True
+
+    @staticmethod
+    def _members(spec, prefix):
+        return PreNormBlock._members(spec, prefix)
+
+    def __init__(self, spec, prefix, env):
+        super().__init__(spec, prefix, env)
+        self._parts = [build_part(t, part, name, env) for t, part, name in self._members(spec, prefix)]
+        self.mixer_norm, self.mixer = self._parts[:2]
+        self.ff_norm, self.feed_forward = self._parts[2:] if len(self._parts) > 2 else (None, None)
+        for norm in (self.mixer_norm, self.ff_norm):
+            if norm is not None and not hasattr(norm, "side_by_side"):
+                raise ValueError(f"parallel_norm: the norm {norm.spec.kind!r} cannot prepare two sublayers' inputs")
+        self.graph_safe = all(getattr(p, "graph_safe", False) for p in self._parts)
+        mixer_state = record_floats(part_class(MIXERS, spec.mixer).cache_request(spec.mixer))
+        self.padded_steps_safe = not mixer_state or getattr(self.mixer, "padded_steps_safe", False)
+        self.shift_floats, self.mixer_floats = self._shift_floats(spec), mixer_state
+
+    @staticmethod
+    def _shift_floats(spec) -> int:
+        return -(-spec.mixer_norm.dim // 4) * 4 if spec.token_shift else 0
+
+    @classmethod
+    def declare(cls, spec, prefix):
+        out = []
+        for table, part, name in cls._members(spec, prefix):
+            out += part_class(table, part).declare(part, name)
+        if spec.token_shift:
+            out.append(TensorDecl(f"{prefix}.{spec.shift_name}", (spec.mixer_norm.dim,), BIAS))
+        return out
+
+    @classmethod
+    def cache_request(cls, spec):
+        request = part_class(MIXERS, spec.mixer).cache_request(spec.mixer)
+        if not spec.token_shift:
+            return request
+        pages = paged_part(request)
+        record = FixedStateRequest((cls._shift_floats(spec) + record_floats(request),))
+        return record if pages is None else (pages, record)
+
+    def load(self, store):
+        for p in self._parts:
+            p.load(store)
+        self.shift = store.get(f"{self.prefix}.{self.spec.shift_name}") if self.spec.token_shift else None
+
+    def forward(self, ctx, resid, delta, cache, owns_cache):
+        prev = None
+        mixer_cache = cache
+        if self.shift is not None:
+            if not owns_cache:
+                raise NotImplementedError("parallel_norm: a token shift in a run that reads another run's cache")
+            prev = cache.with_state_slice(0, self.shift_floats).state
+            mixer_cache = cache.with_state_slice(self.shift_floats, self.mixer_floats)
+        resid, h, f = type(self.mixer_norm).side_by_side(ctx, resid, delta, self.mixer_norm, self.ff_norm,
+                                                         self.shift, prev)
+        terms = [self.mixer.forward(ctx, h, mixer_cache, owns_cache)]
+        if self.feed_forward is not None:
+            terms.append(self.feed_forward.forward(ctx, f))
+        return resid, PendingUpdate(terms)
 
 
 def K_plain(value):

@@ -4,6 +4,11 @@ for every token and key channel, alpha_t = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau) 
 W_a1 is part of the first product; the one with W_a2 returns float32, and the sigmoid, its
 logarithm and the power are formed in float32 inside the recurrence's kernel).
 
+With ``token_mix`` every projection reads a mix of its own of the token's input and the previous
+token's (one kernel forms them), so the projections are products of their own; the previous input is
+part of the request's record, in front of the state.  ``decay_gate_kind`` "exp_exp", ``decay_gate_tanh``
+and ``bonus``: the decay and the current token's part as ``DecayAttentionSpec`` describes them.
+
 Per step, with h the mixer's input [T, hidden]:
 
   1. one product for q | k | v | gate (their matrices are concatenated at load);
@@ -44,6 +49,11 @@ class DecayAttention(Mixer):
         self.gated = s.decay_gate_rank is not None
         # (the kernels for learned decays skip requests without tokens and tiles of padding)
         self.padded_steps_safe = self.gated
+        if s.decay_gate_kind not in K.DECAY_GATE_KINDS:
+            raise ValueError(f"decay_attention: decay_gate_kind {s.decay_gate_kind!r} "
+                             f"({', '.join(K.DECAY_GATE_KINDS)})")
+        if not self.gated and (s.bonus or s.token_mix or s.decay_gate_tanh or s.decay_gate_kind != "sigmoid_root"):
+            raise ValueError("decay_attention: a bonus, mixed inputs and the forms of a decay need learned decays")
         if self.gated and (s.decay or not s.decay_gate_tau > 0):
             raise ValueError("decay_attention: learned decays take no fixed ``decay`` and a positive tau")
         if not self.gated and len(s.decay) != s.num_heads:
@@ -75,7 +85,7 @@ class DecayAttention(Mixer):
     @classmethod
     def _names(cls, spec, prefix):
         return {n: f"{prefix}.{getattr(spec, n + '_name')}"
-                for n in ("q", "k", "v", "gate", "o", "out_norm", "decay_down", "decay_up", "decay_bias")}
+                for n in ("q", "k", "v", "gate", "o", "out_norm", "decay_down", "decay_up", "decay_bias", "bonus")}
 
     @classmethod
     def declare(cls, spec, prefix):
@@ -90,17 +100,33 @@ class DecayAttention(Mixer):
             r = spec.decay_gate_rank            # (-1: the checkpoint's tensor decides)
             out += [TensorDecl(n["decay_down"], (r, h), MATRIX), TensorDecl(n["decay_up"], (qs, r), MATRIX),
                     TensorDecl(n["decay_bias"], (qs,), BIAS)]
+        if spec.bonus:
+            out.append(TensorDecl(n["bonus"], (spec.num_heads, spec.head_dim), BIAS))
+        if spec.token_mix:
+            out += [TensorDecl(f"{prefix}.{name}", (h,), BIAS) for name in spec.token_mix_names]
         return out
 
     @classmethod
+    def _mix_floats(cls, spec) -> int:
+        """Floats of the record that hold the previous token's input (a multiple of 4)."""
+        return -(-spec.hidden_size // 4) * 4 if spec.token_mix else 0
+
+    @classmethod
     def cache_request(cls, spec):
+        if spec.token_mix:
+            return FixedStateRequest((cls._mix_floats(spec) + spec.num_heads * spec.head_dim * spec.value_dim,))
         return FixedStateRequest((spec.num_heads, spec.head_dim, spec.value_dim))
 
     def load(self, store):
         n = self._names(self.spec, self.prefix)
         s = self.spec
         names = [n["q"], n["k"], n["v"], n["gate"]] + ([n["decay_down"]] if self.gated else [])
-        self.w_in = pad_rows(store.cat(names))
+        if s.token_mix:
+            self.w_parts = [store.get(name) for name in names]
+            self.mu = torch.stack([store.get(f"{self.prefix}.{name}") for name in s.token_mix_names]).contiguous()
+        else:
+            self.w_in = pad_rows(store.cat(names))
+        self.bonus = store.get(n["bonus"]).reshape(-1).contiguous() if s.bonus else None
         self.w_o = store.get(n["o"])
         self.norm_w = store.get(n["out_norm"]) if s.out_norm_weight else None
         if self.norm_w is not None and s.out_norm_per_head:
@@ -110,28 +136,52 @@ class DecayAttention(Mixer):
             self.w_a2 = store.get(n["decay_up"])
             self.a2_bias = store.get(n["decay_bias"]).to(torch.float32).contiguous()
 
+    def _mixed_projections(self, ctx, x, cache):
+        """(q | k | v | gate [T, ...], the decay's bottleneck [T, rank], the state's slice of the record)"""
+        s, T = self.spec, x.shape[0]
+        floats = self._mix_floats(s)
+        prev = cache.with_state_slice(0, floats).state
+        state = cache.with_state_slice(floats, s.num_heads * s.head_dim * s.value_dim).state
+        mixed = torch.empty((len(s.token_mix_names), T, s.hidden_size), dtype=x.dtype, device=x.device)
+        K.token_mix(ctx, x, self.mu, prev, mixed)
+        proj = torch.empty((T, 2 * self.q_size + 2 * self.v_size), dtype=x.dtype, device=x.device)
+        at = 0
+        for i, w in enumerate(self.w_parts[:4]):
+            proj[:, at:at + w.shape[0]] = K.plain_unless(None, linear(mixed[i], w))
+            at += w.shape[0]
+        low = K.plain_unless(None, linear(mixed[4], self.w_parts[4]))
+        return proj, low, state
+
     def forward(self, ctx, x, cache, owns_cache):
         s = self.spec
         T = x.shape[0]
-        proj = K.plain_unless(None, linear(x, self.w_in))              # [T, q | k | v | gate]
+        low = None
+        if s.token_mix:
+            proj, low, state = self._mixed_projections(ctx, x, cache)
+        else:
+            proj = K.plain_unless(None, linear(x, self.w_in))          # [T, q | k | v | gate]
+            state = cache.state if cache.state.dim() == 2 else cache.state.view(cache.state.shape[0], -1)
         o = torch.empty((T, self.v_size), dtype=torch.float32, device=x.device)
         gate_z = None
         if self.gated:
-            low = proj[:, 2 * self.q_size + 2 * self.v_size:2 * self.q_size + 2 * self.v_size + self.rank]
-            if self.rank < 64:
+            if low is None:
+                low = proj[:, 2 * self.q_size + 2 * self.v_size:2 * self.q_size + 2 * self.v_size + self.rank]
+            if s.decay_gate_tanh:
+                gate_z = torch.empty((T, self.q_size), dtype=torch.float32, device=x.device)
+                K.tanh_linear(low, self.w_a2, None, gate_z)
+            elif self.rank < 64:
                 # a bottleneck this narrow: the CUDA-core product (float32 sums in k order)
                 gate_z = torch.empty((T, self.q_size), dtype=torch.float32, device=x.device)
                 K.gemm_simt(low, self.w_a2, gate_z)
             else:
                 gate_z = linear(low if low.data_ptr() % 16 == 0 else low.contiguous(), self.w_a2,
                                 out_dtype=torch.float32)
-        state = cache.state if cache.state.dim() == 2 else cache.state.view(cache.state.shape[0], -1)
         K.decay_attention(proj, ctx, state, self.decay, o, q_off=0, k_off=self.q_size,
                           v_off=2 * self.q_size, num_heads=s.num_heads, head_dim=s.head_dim,
                           value_dim=s.value_dim, activation=s.qkv_activation, freq=self.freq,
                           rot_dims=self.rot_dims, key_scale=self.key_scale, query_scale=self.query_scale,
                           gate_z=gate_z, gate_bias=self.a2_bias if self.gated else None,
-                          gate_tau=s.decay_gate_tau)
+                          gate_tau=s.decay_gate_tau, gate_kind=s.decay_gate_kind, bonus=self.bonus)
         gate = proj[:, 2 * self.q_size + self.v_size:2 * self.q_size + 2 * self.v_size]
         out = torch.empty((T, self.v_size), dtype=x.dtype, device=x.device)
         groups, size = (s.num_heads, s.value_dim) if s.out_norm == "head" else (1, self.v_size)

@@ -75,6 +75,33 @@ class HyperPending:
                         "it in (a norm with read_streams)")
 
 
+class PendingUpdate:
+    """Updates of the stream that have not been added yet: up to two results ``terms`` [T, w] (the
+    two sublayers of a block that run side by side) and one vector ``row`` [w] for every token.  The next
+    norm adds them on the way (``accepts_pending_update``)."""
+
+    accept_flag = "accepts_pending_update"
+
+    def __init__(self, terms, row=None):
+        self.terms = tuple(K.plain_unless(None, t) for t in terms)
+        self.row = row
+
+    def materialize(self) -> torch.Tensor:
+        total = self.row.to(torch.float32) if self.row is not None else None
+        for t in self.terms:
+            total = t.to(torch.float32) if total is None else total + t.to(torch.float32)
+        return total.to(self.terms[0].dtype) if self.terms else total
+
+
+def pending_parts(delta):
+    """(terms, row) of an update in any finished form."""
+    if delta is None:
+        return (), None
+    if isinstance(delta, PendingUpdate):
+        return delta.terms, delta.row
+    return (K.plain_unless(None, delta),), None
+
+
 fuse_product_norms = True     # Dynamic Tanh: a deferred product runs with the norms in its epilogue
 
 
@@ -104,6 +131,7 @@ class DynamicTanh(Norm):
     one kernel then norms the update, adds it and norms the sum."""
     graph_safe = True
     accepts_post_normed = True
+    accepts_pending_update = True     # (as the norm of selected rows, or ``side_by_side``)
     accepts_deferred_linear = True    # as the pending norm of a PostNormed value: the value may be a
                                       # product not launched yet, which then runs with both norms
                                       # and the add in its epilogue
@@ -121,8 +149,27 @@ class DynamicTanh(Norm):
         self.alpha = store.get(self.prefix + s.alpha_suffix).reshape(1)
         self.params = (self.alpha, self.weight, self.bias)
 
+    @staticmethod
+    def side_by_side(ctx, resid, delta, first: "DynamicTanh", second, shift=None, prev=None):
+        """The inputs of two sublayers that read the same stream: (stream with the pending update added,
+        first(x), second(x) or None).  ``shift`` [w]: the first is mixed with the previous token's,
+        whose last row per request is in ``prev``.  One launch; the stream moves to a new buffer if
+        anything was pending."""
+        terms, row = pending_parts(delta)
+        out = resid if not terms and row is None else torch.empty_like(resid)
+        a = torch.empty(resid.shape, dtype=first.env.dtype, device=resid.device)
+        b = None if second is None else torch.empty_like(a)
+        K.dyt_parallel(ctx, resid, terms, row, first.params, a, None if second is None else second.params, b,
+                       None if out is resid else out, shift, prev)
+        return out, a, b
+
     def forward(self, ctx, resid, delta, out_rows=None):
         post = None
+        if isinstance(delta, PendingUpdate) and out_rows is not None:
+            out = torch.empty((out_rows.numel(), self.spec.dim), dtype=self.env.dtype, device=resid.device)
+            K.dyt_parallel(ctx, resid, delta.terms, delta.row, self.params, out, row_map=out_rows)
+            return out
+        delta = delta.materialize() if isinstance(delta, PendingUpdate) else delta
         if isinstance(delta, PostNormed):
             if isinstance(delta.norm, DynamicTanh):
                 post, delta = delta.norm.params, delta.value

@@ -15,7 +15,8 @@ Per step, with h the mixer's input [T, hidden]:
      cache holds what the attention uses;
   3. attention of every query over its request's visible keys, softmax in float32 (scores
      soft-capped, a sink a head in the denominator: each optional), head h's row times
-     sigmoid(gate_h);
+     sigmoid(gate_h); or, with ``weight_fn`` "sigmoid", weights sigmoid(score + a number a head) that
+     are not normalized; visible keys: all earlier ones, a window, or the query's own chunk;
   4. the output projection (``out_dtype``: a mixer that norms the result asks for float32).
 
 The values of the source layer travel to the mixing layers through the step's scratch
@@ -61,6 +62,14 @@ class NormedAttention(Mixer):
             raise ValueError(f"normed_attention: 0..{K.CONV_MAX_TAPS} taps, got {spec.conv_taps}")
         if spec.softcap is not None and not spec.softcap > 0:
             raise ValueError("normed_attention: a soft cap must be positive")
+        if spec.weight_fn not in ("softmax", "sigmoid"):
+            raise ValueError(f"normed_attention: weight_fn {spec.weight_fn!r} ('softmax', 'sigmoid')")
+        if spec.weight_fn == "sigmoid" and (spec.softcap is not None or spec.sink or spec.head_gate):
+            raise ValueError("normed_attention: sigmoid weights go without a soft cap, sink or gate")
+        if spec.score_bias and spec.weight_fn != "sigmoid":
+            raise ValueError("normed_attention: a number a head on the scores needs sigmoid weights")
+        if spec.chunk is not None and (spec.window is not None or spec.chunk < 1):
+            raise ValueError("normed_attention: a chunk is at least 1 and goes without a window")
         self.position = build_part(POSITIONS, spec.position, f"{prefix}.rot", env)
         self.out_dtype = None                  # (set by a mixer that wraps this one)
         self.scale = spec.scale if spec.scale is not None else 1.0 / math.sqrt(spec.head_dim)
@@ -70,7 +79,8 @@ class NormedAttention(Mixer):
         A.check_kv_supported(spec.head_dim, spec.value_dim)
         A.prepare_kv_attention(spec.head_dim, spec.value_dim, env.dtype)
         if (spec.head_dim == spec.value_dim and env.dtype == torch.bfloat16 and spec.head_dim in (64, 128)
-                and spec.softcap is None and not spec.sink and torch.cuda.is_available()):
+                and spec.softcap is None and not spec.sink and spec.weight_fn == "softmax" and spec.chunk is None
+                and torch.cuda.is_available()):
             from ..ops import library
             library.attention(spec.head_dim)      # the kernels for equal sizes, built now
 
@@ -96,11 +106,14 @@ class NormedAttention(Mixer):
                     for x, rows in (("q", H * D), ("k", G * D), ("v", G * Dv))]
         if spec.sink:
             out.append(TensorDecl(f"{prefix}.{spec.sink_name}", (H,), BIAS))
+        if spec.score_bias:
+            out.append(TensorDecl(f"{prefix}.{spec.score_bias_name}", (H,), BIAS))
         return out
 
     @classmethod
     def cache_request(cls, spec):
-        pages = PagedKVRequest(spec.num_kv_heads, spec.head_dim, spec.window, value_dim=spec.value_dim)
+        pages = PagedKVRequest(spec.num_kv_heads, spec.head_dim, spec.window, value_dim=spec.value_dim,
+                               chunk=spec.chunk)
         if spec.conv_taps <= 1:
             return pages
         width = spec.num_heads * spec.head_dim + spec.num_kv_heads * (spec.head_dim + spec.value_dim)
@@ -118,6 +131,10 @@ class NormedAttention(Mixer):
         if s.conv_taps >= 1:
             # [taps, channels]: a tap's weights of neighbouring channels are neighbours
             self.taps = store.cat([n[x] + s.conv_suffix for x in ("q", "k", "v")]).t().contiguous()
+        self.sigmoid_bias = None
+        if s.weight_fn == "sigmoid":
+            self.sigmoid_bias = (store.get(f"{self.prefix}.{s.score_bias_name}") if s.score_bias
+                                 else torch.zeros(s.num_heads, dtype=torch.float32, device=self.env.device))
         self.sink = store.get(f"{self.prefix}.{s.sink_name}").to(torch.float32).contiguous() if s.sink else None
 
     def forward(self, ctx, x, cache, owns_cache):
@@ -147,6 +164,7 @@ class NormedAttention(Mixer):
         halves = pairs is None and self.position.rotary_table() is not None
         if halves:                                 # element i with element i + dims / 2
             freq, rot_dims = self.position.rotary_table()
+            mag = self.position.magnitude
         norm_dims = s.head_dim if s.qk_norm else 0
         unit_dims = s.head_dim if s.qk_unit_norm else 0
         K.head_prep(proj, ctx, table, cache.page_size,
@@ -162,7 +180,7 @@ class NormedAttention(Mixer):
         out = torch.empty((T, s.num_heads * s.value_dim), dtype=x.dtype, device=x.device)
         A.kv_attention(ctx, q, cache.k, cache.v, s.value_dim, out, table, s.num_heads, s.num_kv_heads,
                        s.head_dim, s.value_dim, cache.page_size, self.scale, s.window or 0, gate,
-                       s.softcap, self.sink)
+                       s.softcap, self.sink, s.chunk or 0, self.sigmoid_bias)
         if self.out_dtype is not None:
             return linear(out, self.w_o, out_dtype=self.out_dtype)
         return linear(out, self.w_o, consumer="norm")

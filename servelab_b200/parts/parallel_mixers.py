@@ -15,11 +15,9 @@ are the whole record's length apart, which the kernels that index state take as 
 
 from __future__ import annotations
 
-import math
-
 import torch
 
-from ..cache.manager import FixedStateRequest, paged_part, state_part
+from ..cache.manager import FixedStateRequest, paged_part, record_floats
 from ..ops import kernels as K
 from ..weights.source import NORM, TensorDecl
 from .base import LayerCache, Mixer
@@ -28,11 +26,7 @@ from .registry import MIXERS, build_part, part_class, register_mixer
 
 def _record_sizes(spec):
     """Floats of each branch's state record, rounded up to 4 (16-byte aligned slices)."""
-    sizes = []
-    for branch in (spec.left, spec.right):
-        st = state_part(part_class(MIXERS, branch).cache_request(branch))
-        sizes.append(0 if st is None else -(-math.prod(st.shape) // 4) * 4)
-    return sizes
+    return [record_floats(part_class(MIXERS, b).cache_request(b)) for b in (spec.left, spec.right)]
 
 
 @register_mixer("parallel_mixers")
@@ -76,9 +70,7 @@ class ParallelMixers(Mixer):
         self.w_left, self.w_right = (store.get(n) for n in self._norm_names(self.spec, self.prefix))
 
     def _branch_cache(self, cache: LayerCache, index: int) -> LayerCache:
-        start = sum(self.sizes[:index])
-        state = cache.state[:, start:start + self.sizes[index]] if self.sizes[index] else None
-        return LayerCache(group=cache.group, k=cache.k, v=cache.v, state=state, page_size=cache.page_size)
+        return cache.with_state_slice(sum(self.sizes[:index]), self.sizes[index])
 
     def forward(self, ctx, x, cache, owns_cache):
         a = K.plain_unless(None, self.left.forward(ctx, x, self._branch_cache(cache, 0), owns_cache))

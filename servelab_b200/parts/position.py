@@ -29,6 +29,19 @@ def stretch_long_wavelengths(f: torch.Tensor, factor: float, low: float, high: f
                        torch.where(wavelength > original / low, f / factor, blended))
 
 
+def interpolate_by_ramp(f: torch.Tensor, dims: int, theta: float, factor: float, original: float, fast: float,
+                        slow: float):
+    """(frequencies, factor on cos and sin) of the YaRN scaling of ``f`` (float64 [dims / 2]): f and
+    f / factor blended by a ramp over the pairs, from the pair that turns ``fast`` times within
+    ``original`` positions to the one that turns ``slow`` times."""
+    def pair_that_turns(times: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * times)) / (2.0 * math.log(theta))
+    lo = max(math.floor(pair_that_turns(fast)), 0)
+    hi = min(math.ceil(pair_that_turns(slow)), dims - 1)
+    ramp = ((torch.arange(dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 @register_position("rotary")
 class RotaryEmbedding(PositionEncoding):
     graph_safe = True
@@ -39,7 +52,8 @@ class RotaryEmbedding(PositionEncoding):
         if rd % 2 or rd > spec.head_dim:
             raise ValueError(f"rotary_dim {rd} must be even and <= head_dim {spec.head_dim}")
         inv_freq = 1.0 / (spec.theta ** (torch.arange(0, rd, 2, dtype=torch.float32) / rd))
-        if spec.precise or spec.stretch_factor is not None:
+        self.magnitude = 1.0                   # on cos and sin
+        if spec.precise or spec.stretch_factor is not None or spec.yarn_factor is not None:
             f = float(spec.theta) ** (-2.0 * torch.arange(rd // 2, dtype=torch.float64) / rd)
             if spec.stretch_factor is not None:
                 if not (spec.stretch_factor > 0 and spec.stretch_high > spec.stretch_low >= 0
@@ -47,6 +61,9 @@ class RotaryEmbedding(PositionEncoding):
                     raise ValueError("rotary: a stretch needs factor > 0, high > low >= 0 and original > 0")
                 f = stretch_long_wavelengths(f, float(spec.stretch_factor), float(spec.stretch_low),
                                              float(spec.stretch_high), float(spec.stretch_original))
+            if spec.yarn_factor is not None:
+                f, self.magnitude = interpolate_by_ramp(f, rd, float(spec.theta), float(spec.yarn_factor),
+                                                        spec.yarn_original, spec.yarn_fast, spec.yarn_slow)
             inv_freq = f.to(torch.float32)
         self.rotary_dim = rd
         self.inv_freq = inv_freq.to(env.device)
@@ -72,15 +89,8 @@ class PairRotary(PositionEncoding):
         f = float(spec.theta) ** (-2.0 * i / d)
         self.magnitude = 1.0
         if spec.yarn_factor is not None:
-            factor = float(spec.yarn_factor)
-
-            def pair_that_turns(times: float) -> float:
-                return d * math.log(spec.yarn_original / (2.0 * math.pi * times)) / (2.0 * math.log(spec.theta))
-            lo = max(math.floor(pair_that_turns(spec.yarn_fast)), 0)
-            hi = min(math.ceil(pair_that_turns(spec.yarn_slow)), d - 1)
-            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-            f = f / factor * ramp + f * (1.0 - ramp)
-            self.magnitude = 0.1 * math.log(factor) + 1.0
+            f, self.magnitude = interpolate_by_ramp(f, d, float(spec.theta), float(spec.yarn_factor),
+                                                    spec.yarn_original, spec.yarn_fast, spec.yarn_slow)
         if spec.stretch_factor is not None:
             f = stretch_long_wavelengths(f, float(spec.stretch_factor), float(spec.stretch_low),
                                          float(spec.stretch_high), float(spec.stretch_original))
