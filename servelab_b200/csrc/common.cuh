@@ -25,6 +25,10 @@ template <typename T> __device__ __forceinline__ T from_float(float v);
 template <> __device__ __forceinline__ float from_float<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_float<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// e^x for x <= 0 as a decay that is applied token after token: near 1 it is rounded to the nearest
+// float from an accurate e^x - 1, so that the errors of many steps do not all lean to one side.
+__device__ __forceinline__ float decay_exp(float x) { return x > -1.0f ? 1.0f + expm1f(x) : expf(x); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -90,7 +90,7 @@ __global__ void __launch_bounds__(DA_EV * DA_PARTS, R <= 16 ? 4 : 2) decay_atten
                 if (gated) {
                     float z = a.gate_z[(size_t)(q0 + t0 + j) * a.ld_gate + h * D + d];
                     if (a.gate_bias != nullptr) z += a.gate_bias[h * D + d];
-                    av = expf(da_log_decay(z, a.gate_kind, a.gate_inv_tau));
+                    av = decay_exp(da_log_decay(z, a.gate_kind, a.gate_inv_tau));
                 }
             }
             qs[idx] = qv;

@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(256) gated_chunk_prep_kernel(const GatedChunkA
             run += Ls[j * LD + d];
             Ls[j * LD + d] = run;
         }
-        c.dtot[((size_t)tile * a.H + h) * D + d] = expf(run);
+        c.dtot[((size_t)tile * a.H + h) * D + d] = decay_exp(run);
     }
     __syncthreads();
     const size_t ldl = (size_t)a.H * D;

@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(DR_MAX_WARPS * 32, 1) delta_rule_kernel(const 
                 if (d < D) {
                     k = to_float(row[a.k_off + h * D + d]);
                     const float r = to_float(row[a.r_off + h * D + d]);
-                    w = expf(-a.decay_coef * dr_sigmoid(zr[d]));
+                    w = decay_exp(-a.decay_coef * dr_sigmoid(zr[d]));
                     u = k * inv;
                     au = dr_sigmoid(to_float(row[a.a_off + h * D + d]) + a.a_bias[h * D + d]) * u;
                     rw = r * w;
@@ -368,7 +368,7 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const DeltaChunkA
             gR[j * Dp + d] = rg; gK[j * Dp + d] = ke; gB[j * Dp + d] = be;
         }
     }
-    for (int d = tid; d < Dp; d += blockDim.x) gG[d] = expf(Ls[(DC_C - 1) * LD + d]);
+    for (int d = tid; d < Dp; d += blockDim.x) gG[d] = decay_exp(Ls[(DC_C - 1) * LD + d]);
     __syncthreads();
     // the four score matrices as one 64 x 64 product; thread (ty, tx): rows ty + 16 i, columns tx + 16 j
     {

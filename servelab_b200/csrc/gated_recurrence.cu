@@ -32,7 +32,7 @@ __device__ __forceinline__ float gr_gelu_tanh(float z) {
 }
 // a and sqrt(1 - a^2) from log a (1 - a^2 = -expm1(2 log a): no cancellation for a near 1)
 __device__ __forceinline__ void gr_decay(float log_a, float& a, float& gain) {
-    a = expf(log_a);
+    a = decay_exp(log_a);
     gain = sqrtf(-expm1f(2.0f * log_a));
 }
 
