@@ -401,6 +401,106 @@ def _sumolorn_rooflines(size, res, peaks) -> Dict[str, object]:
     return out
 
 
+# Vufadra: four layers -- gated recurrence, delta rule, a parallel layer (chunked sigmoid attention
+# beside a linear attention with learned decays, a bonus and mixed inputs), delta rule -- each with a
+# SiLU feed-forward on the same stream, and the bigram embedding (no loop, so that both models run four
+# layers).  Beside it the closest model the package has: Sumolorn with its parallel layer (windowed
+# attention beside a linear attention with learned decays) where Vufadra has a parallel layer or a delta
+# rule -- the linear branches have the sizes of Vufadra's recurrences -- and its attention in the place
+# of the gated recurrence, the same feed-forward.
+# width, heads, kv heads, head size, feed-forward, recurrent heads (of the head size), bottleneck
+VUFADRA_SIZES = {
+    "1b-like": (2048, 16, 4, 128, 5632, 16, 64),
+    "small-1024": (1024, 8, 2, 64, 2816, 16, 32),
+}
+
+
+def vufadra_config(width, heads, kv, dim, ff, rh, rank, layers=LAYERS) -> dict:
+    mlp = {"kind": "dense", "ff": ff}
+    left = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": WINDOW},
+            "rot": {"base": 500000.0, "dims": dim,
+                    "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    delta = ("general_delta", {"heads": rh, "dim": dim, "rank": rank})
+    kinds = [("rglru", {"width": width, "blocks": width // 128, "conv": 4}), delta,
+             ("parallel", {"left": left, "right": {"heads": rh, "dim": dim, "rank": rank}}), delta]
+    return {"architecture": "Vufadra", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65536, "mul_prev": 31337, "mul_cur": 271}},
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(layers)]}
+
+
+def sumolorn_like_vufadra(width, heads, kv, dim, ff, rh, rank, layers=LAYERS) -> dict:
+    mlp = {"kind": "dense", "ff": ff, "limit": 7.0}
+    attn = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+            "mask": {"size": WINDOW}, "rot": {"base": 500000.0, "dims": dim}}
+    left = {"conv": 4, "heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+            "mask": {"size": WINDOW}, "rot": {"base": 500000.0, "dims": dim}}
+    par = ("parallel", {"left": left, "right": {"heads": rh, "dim": dim, "vdim": dim, "tau": 8.0, "rank": rank}})
+    kinds = [("attention", attn), par, par, par]
+    return {"architecture": "Sumolorn", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(layers)]}
+
+
+def _vufadra_rooflines(size, res, peaks) -> Dict[str, object]:
+    """Microseconds a layer and achieved fractions of the measured peaks for the kernels of the Vufadra
+    layers beside their Sumolorn counterparts, from the eager profiles.  Attention, prefill: 2 (Dk + Dv)
+    flops per visible pair and head of the bf16 peak; decode: the cached rows 8 requests may see of
+    the copy bandwidth.  Recurrences with a matrix of state, prefill: their own arithmetic (4 T H D Dv
+    flops for a decay and an output, 8 for the delta rule: state read along the key, two updates and the
+    output) of the bf16 peak; decode: the state read and written once.  Elementwise kernels and the
+    recurrence with a number a channel: the bytes they must move."""
+    width, heads, kv, dim, ff, rh, rank = VUFADRA_SIZES[size]
+    vp, sp = (res[a]["prefill_kernels_us"] for a in ("vufadra", "sumolorn"))
+    out: Dict[str, object] = {}
+
+    def hbm(nbytes, us):
+        return round(nbytes / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 4)
+
+    def tf(flops, us):
+        return round(flops / (us * 1e-6) / 1e12 / peaks["bf16_tflops"], 4)
+
+    def row(name, table, key, layers, frac):
+        us = sum(table.get(k) or 0 for k in ((key,) if isinstance(key, str) else key))
+        if us:
+            out[name] = {"us": round(us / layers, 2), "frac": frac(us / layers)}
+    state = rh * dim * dim
+    chunk_pairs = sum(t % WINDOW + 1 for t in range(PROMPT))
+    win_pairs = sum(min(t + 1, WINDOW) for t in range(PROMPT))
+    tc = ("attention_kv_tc", "attention_kv_mma", "prefill_attention_tc", "prefill_attention", "attention_kv")
+    row("vufadra_chunk_attention_prefill", vp, tc, 1, lambda us: tf(chunk_pairs * heads * 4 * dim, us))
+    row("sumolorn_attention_prefill", sp, tc, LAYERS, lambda us: tf(win_pairs * heads * 4 * dim, us))
+    row("vufadra_delta_prefill", vp, ("delta_rule (chunks)", "delta_rule"), 2, lambda us: tf(8.0 * PROMPT * state, us))
+    lin = ("decay_attention (gated chunks)", "decay_attention")
+    row("vufadra_decay_prefill", vp, lin, 1, lambda us: tf(4.0 * PROMPT * state, us))
+    row("sumolorn_decay_prefill", sp, lin, 3, lambda us: tf(4.0 * PROMPT * state, us))
+    row("vufadra_gated_recurrence_prefill", vp, "gated_recurrence", 1, lambda us: hbm(PROMPT * width * 14, us))
+    row("vufadra_conv_prefill", vp, "short_conv", 1, lambda us: hbm(PROMPT * width * 4, us))
+    row("sumolorn_conv_prefill", sp, "short_conv", 3, lambda us: hbm(PROMPT * (heads + 2 * kv) * dim * 4, us))
+    row("vufadra_norms_prefill", vp, "dyt_parallel", LAYERS, lambda us: hbm(PROMPT * width * 16, us))
+    row("sumolorn_norm_prefill", sp, "add_rmsnorm", 2 * LAYERS, lambda us: hbm(PROMPT * width * 12, us))
+    row("vufadra_token_mix_prefill", vp, "token_mix", 1, lambda us: hbm(PROMPT * width * 12, us))
+    row("vufadra_bottleneck_prefill", vp, "tanh_linear", 3, lambda us: hbm(PROMPT * rh * dim * 4, us))
+    row("sumolorn_bottleneck_prefill", sp, "gemm_simt", 3, lambda us: hbm(PROMPT * rh * dim * 4, us))
+    row("vufadra_head_prep_prefill", vp, "head_prep", 1, lambda us: hbm(PROMPT * 4 * (heads + 2 * kv) * dim, us))
+    row("sumolorn_head_prep_prefill", sp, "head_prep", LAYERS, lambda us: hbm(PROMPT * 4 * (heads + 2 * kv) * dim, us))
+    row("vufadra_norm_gate_prefill", vp, "group_norm_gate", 3, lambda us: hbm(PROMPT * rh * dim * 8, us))
+    row("sumolorn_norm_gate_prefill", sp, "group_norm_gate", 3, lambda us: hbm(PROMPT * rh * dim * 8, us))
+    row("vufadra_branch_norms_prefill", vp, "norm_sum2", 1, lambda us: hbm(PROMPT * width * 10, us))
+    row("sumolorn_branch_norms_prefill", sp, "norm_sum2", 3, lambda us: hbm(PROMPT * width * 10, us))
+    row("vufadra_embedding_prefill", vp, "embed_bigram", 1, lambda us: hbm(PROMPT * width * 8, us))
+    row("sumolorn_embedding_prefill", sp, "embedding", 1, lambda us: hbm(PROMPT * width * 6, us))
+    for b in (8, 64):
+        vd, sd = (res[a][f"decode_b{b}_kernels_us"] for a in ("vufadra", "sumolorn"))
+        dec = ("attention_kv_mma", "attention_kv", "decode_attention")
+        # (a context of CONTEXT tokens sits at CONTEXT % WINDOW in its chunk)
+        seen_v, seen_s = (CONTEXT - 1) % WINDOW + 1, min(CONTEXT, WINDOW)
+        row(f"vufadra_chunk_attention_decode_b{b}", vd, dec, 1, lambda us: hbm(b * seen_v * kv * 4 * dim, us))
+        row(f"sumolorn_attention_decode_b{b}", sd, dec, LAYERS, lambda us: hbm(b * seen_s * kv * 4 * dim, us))
+        row(f"vufadra_delta_decode_b{b}", vd, "delta_rule", 2, lambda us: hbm(b * state * 8, us))
+        row(f"vufadra_decay_decode_b{b}", vd, "decay_attention", 1, lambda us: hbm(b * state * 8, us))
+        row(f"sumolorn_decay_decode_b{b}", sd, "decay_attention", 3, lambda us: hbm(b * state * 8, us))
+    return out
+
+
 def _measure(cfg: dict, note, graph_prefill: bool = False) -> Dict[str, object]:
     """``graph_prefill``: the prompt's step replays the graph captured for its padded sizes where the
     model allows it (the eager step of a small model is bound by the host's launches); the eager
@@ -530,6 +630,22 @@ def _kernel_rooflines(size, res: Dict[str, Dict[str, object]], peaks) -> Dict[st
 
 
 def run(peaks, note=lambda m: None, sizes=None, design: str = "dezelorn") -> Dict[str, object]:
+    if design == "vufadra":
+        result = {"compare": "vufadra vs sumolorn (attention, and parallel layers with a linear branch of the same "
+                             "sizes) at equal layer sizes", "layers": LAYERS, "prompt": PROMPT,
+                  "decode_context": CONTEXT, "window": WINDOW, "vocab": VOCAB, "dtype": "bf16",
+                  "data": "synthetic: random weights, token ids uniform over the vocabulary",
+                  "peaks": peaks.get("source"), "sizes": {}}
+        for size in (sizes or VUFADRA_SIZES):
+            dims = VUFADRA_SIZES[size]
+            res = {}
+            for arch, make in (("vufadra", vufadra_config), ("sumolorn", sumolorn_like_vufadra)):
+                note(f"{size}: {arch}")
+                res[arch] = _measure(make(*dims), note, graph_prefill=True)
+            res["kernels"] = _vufadra_rooflines(size, res, peaks)
+            res["dims"] = dict(zip(("width", "heads", "kv_heads", "head_dim", "ff", "recurrent_heads", "bottleneck"), dims))
+            result["sizes"][size] = res
+        return result
     if design == "sumolorn":
         result = {"compare": "sumolorn vs daferax (grouped-query and latent attention, dense feed-forward) at equal "
                              "layer sizes", "layers": LAYERS, "prompt": PROMPT, "decode_context": CONTEXT,
