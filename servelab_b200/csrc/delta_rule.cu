@@ -9,24 +9,8 @@
 // projected row per token.  Everything after the load is float32.
 //
 // Token by token (`delta_rule_kernel`): steps of single tokens, short portions, the 32-bit path.
-// Chunked (`delta_chunk_*`): longer portions.  Both can cut a request anywhere.
-#include "mma_util.cuh"
-
-struct DeltaRuleArgs {
-    const void* proj; int ld;
-    int r_off, k_off, v_off, a_off;
-    int H, D, Dv;
-    const float* a_bias;                     // [H * D]
-    const float* gate_z; int ld_gate; float decay_coef; float unit_eps;
-    const int* cu_q; const int* state_slots;
-    float* state; int num_slots; long long state_stride;
-    float* out; int ldo;                     // [T][H * Dv] float32 (not with out_t)
-    // with out_t: every head's result divided by its root mean square, times norm_w [H * Dv], times
-    // sigmoid of the gate columns of proj, in the compute type
-    void* out_t; int ldt; int g_off; const float* norm_w; float norm_eps;
-};
-
-__device__ __forceinline__ float dr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// Chunked (delta_rule_chunk.cu): longer portions.  Both can cut a request anywhere.
+#include "delta_rule.cuh"
 
 // ------------------------------------------------------------------ token by token
 // Row of S that element i (of R = 4 * groups) of part p holds: groups of four rows are dealt out to the
@@ -38,7 +22,6 @@ __device__ __forceinline__ float dr_sigmoid(float z) { return 1.0f / (1.0f + exp
 // A warp owns 4 CV value columns: lane = 8 * column group + part; a thread keeps R rows of CV columns
 // in registers.
 #define DR_TT 8
-#define DR_MAX_D 256
 #define DR_MAX_WARPS 16
 
 template <typename T, int R, int CV>
@@ -212,16 +195,6 @@ __global__ void __launch_bounds__(DR_MAX_WARPS * 32, 1) delta_rule_kernel(const 
     }
 }
 
-static int dr_check(const DeltaRuleArgs& a) {
-    if (a.H <= 0 || a.D <= 0 || a.Dv <= 0 || a.num_slots <= 0 || a.state == nullptr || a.gate_z == nullptr ||
-        a.ld_gate < a.H * a.D || a.a_bias == nullptr || a.state_stride < (long long)a.H * a.D * a.Dv ||
-        !(a.decay_coef >= 0.f) || (a.out == nullptr) == (a.out_t == nullptr) ||
-        (a.out_t != nullptr && a.norm_w == nullptr))
-        return SLB_ERR_BAD_ARG;
-    if (a.D > DR_MAX_D || a.H > 65535) return SLB_ERR_TOO_LARGE;
-    return 0;
-}
-
 // rows a thread holds and columns a thread for key size D, and the warps (of 4 CV columns) for Dv columns
 static void dr_shape(int D, int Dv, int& R, int& CV, int& warps) {
     R = D <= 32 ? 4 : D <= 64 ? 8 : D <= 128 ? 16 : 32;
@@ -255,379 +228,6 @@ static int launch_delta_rule(const DeltaRuleArgs& a, int num_seqs, cudaStream_t 
     return launch_delta_rule_rc<T, 32, 2>(a, num_seqs, warps, z, st);
 }
 
-// ------------------------------------------------------------------ in chunks
-// A chunk of C = 32 tokens with entering state S.  L_t: sum of log w up to and including token t
-// (per channel), G_t = e^(L_t).  With seen_t = u_t^T S_{t-1} and b_t = a_t u_t,
-//
-//     S_t    = G_t S + sum_{j <= t} (G_t / G_j) (k_j v_j^T - b_j seen_j^T)
-//     seen_t = (u_t G_{t-1})^T S + sum_{j < t} (N[t][j] v_j - M[t][j] seen_j),
-//              N[t][j] = sum_d u_t G_{t-1} k_j / G_j,   M[t][j] = sum_d u_t G_{t-1} b_j / G_j
-//     o_t    = (r_t G_t)^T S + sum_{j <= t} (P[t][j] v_j - Q[t][j] seen_j),
-//              P[t][j] = sum_d r_t G_t k_j / G_j,       Q[t][j] = sum_d r_t G_t b_j / G_j
-//
-// so with the unit lower triangle I + M solved for its right-hand sides once,
-//
-//     seen = X S + Y v,   X = (I + M)^-1 (u G_{t-1}),   Y = (I + M)^-1 N.
-//
-// The factors 1 / G_j are formed alone: a step's log decay is at least -coef, so over a chunk they stay
-// below e^(32 coef) (the launcher takes coef <= 2), and every product of two factors has the relative
-// error of its factors.  Two launches: `prep` per (chunk, head) leaves X, Y, P, Q, the decayed rows
-// r_t G_t, k_j G_C / G_j, b_j G_C / G_j and G_C in a work buffer; `scan` walks a request's chunks with 16
-// value columns of the state a block.  float32 on the CUDA cores throughout.
-#define DC_C 32
-#define DC_EV 16
-
-struct DeltaChunkArgs {
-    DeltaRuleArgs a;
-    const int* tile_seq; const int* tile_row0; int num_tiles;
-    float* work;                             // [num_tiles][H][dc_floats(D)]
-};
-
-// a (chunk, head)'s record: X, R, K, B as [C][Dp], then Y, P, Q as [C][C], then G_C [Dp]
-__host__ __device__ constexpr int dc_pad(int D) { return (D + 3) & ~3; }
-__host__ __device__ constexpr size_t dc_floats(int D) {
-    return (size_t)4 * DC_C * dc_pad(D) + 3 * DC_C * DC_C + dc_pad(D);
-}
-
-__device__ __forceinline__ bool dc_tile(const DeltaChunkArgs& c, int tile, int& t0, int& n) {
-    const int s = c.tile_seq[tile];
-    const int q0 = c.a.cu_q[s], row0 = c.tile_row0[tile];
-    n = min(DC_C, c.a.cu_q[s + 1] - q0 - row0);
-    t0 = q0 + row0;
-    return n > 0;
-}
-
-template <typename T>
-__global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const DeltaChunkArgs c) {
-    extern __shared__ __align__(16) float dc_smem[];
-    pdl_wait();
-    pdl_launch_dependents();
-    const DeltaRuleArgs& a = c.a;
-    const int tile = blockIdx.x, h = blockIdx.y;
-    int t0, n;
-    if (!dc_tile(c, tile, t0, n)) return;
-    const int D = a.D, Dp = dc_pad(D), LD = Dp + 4;
-    float* Ls = dc_smem;                         // [C][LD]: log decays, then their running sums
-    float* Rs = Ls + DC_C * LD;                  // r_t G_t          (rows 0..31 of the left operand)
-    float* Us = Rs + DC_C * LD;                  // u_t G_{t-1}      (rows 32..63)
-    float* Ks = Us + DC_C * LD;                  // k_j / G_j        (rows 0..31 of the right operand)
-    float* Bs = Ks + DC_C * LD;                  // a_j u_j / G_j    (rows 32..63)
-    float* Gm = Bs + DC_C * LD;                  // [64][68]: the products of the two operands
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const T* proj = reinterpret_cast<const T*>(a.proj);
-    for (int idx = tid; idx < DC_C * Dp; idx += blockDim.x) {
-        const int j = idx / Dp, d = idx - j * Dp;
-        float l = 0.f;
-        if (j < n && d < D) l = -a.decay_coef * dr_sigmoid(a.gate_z[(size_t)(t0 + j) * a.ld_gate + h * D + d]);
-        Ls[j * LD + d] = l;
-    }
-    __syncthreads();
-    for (int d = tid; d < Dp; d += blockDim.x) {
-        float run = 0.f;
-        for (int j = 0; j < DC_C; ++j) {
-            run += Ls[j * LD + d];
-            Ls[j * LD + d] = run;                // (beyond the chunk's tokens the sum stays what it is)
-        }
-    }
-    __syncthreads();
-    float* rec = c.work + ((size_t)tile * a.H + h) * dc_floats(D);
-    float* gX = rec, *gR = gX + DC_C * Dp, *gK = gR + DC_C * Dp, *gB = gK + DC_C * Dp;
-    float* gY = gB + DC_C * Dp, *gP = gY + DC_C * DC_C, *gQ = gP + DC_C * DC_C, *gG = gQ + DC_C * DC_C;
-    for (int j = warp; j < DC_C; j += 8) {
-        if (j >= n) {
-            for (int d = lane; d < Dp; d += 32) {
-                Rs[j * LD + d] = Us[j * LD + d] = Ks[j * LD + d] = Bs[j * LD + d] = 0.f;
-                gR[j * Dp + d] = gK[j * Dp + d] = gB[j * Dp + d] = 0.f;
-            }
-            continue;
-        }
-        const T* row = proj + (size_t)(t0 + j) * a.ld;
-        float ss = 0.f;
-        for (int d = lane; d < D; d += 32) {
-            const float k = to_float(row[a.k_off + h * D + d]);
-            ss = fmaf(k, k, ss);
-        }
-        ss = warp_sum(ss);
-        const float inv = 1.0f / sqrtf(ss + a.unit_eps);
-        for (int d = lane; d < Dp; d += 32) {
-            float rg = 0.f, ug = 0.f, kg = 0.f, bg = 0.f, ke = 0.f, be = 0.f;
-            if (d < D) {
-                const float L = Ls[j * LD + d], Lp = j > 0 ? Ls[(j - 1) * LD + d] : 0.f, Le = Ls[(DC_C - 1) * LD + d];
-                const float k = to_float(row[a.k_off + h * D + d]), r = to_float(row[a.r_off + h * D + d]);
-                const float u = k * inv;
-                const float b = dr_sigmoid(to_float(row[a.a_off + h * D + d]) + a.a_bias[h * D + d]) * u;
-                const float up = expf(-L), rest = expf(Le - L);
-                rg = r * expf(L);
-                ug = u * expf(Lp);
-                kg = k * up;
-                bg = b * up;
-                ke = k * rest;
-                be = b * rest;
-            }
-            Rs[j * LD + d] = rg; Us[j * LD + d] = ug; Ks[j * LD + d] = kg; Bs[j * LD + d] = bg;
-            gR[j * Dp + d] = rg; gK[j * Dp + d] = ke; gB[j * Dp + d] = be;
-        }
-    }
-    for (int d = tid; d < Dp; d += blockDim.x) gG[d] = decay_exp(Ls[(DC_C - 1) * LD + d]);
-    __syncthreads();
-    // the four score matrices as one 64 x 64 product; thread (ty, tx): rows ty + 16 i, columns tx + 16 j
-    {
-        const int tx = tid & 15, ty = tid >> 4;
-        float acc[4][4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-        const float* A0 = Rs + ty * LD;          // (Us follows Rs, Bs follows Ks: one 64-row operand each)
-        const float* B0 = Ks + tx * LD;
-        for (int d = 0; d < Dp; d += 4) {
-            float4 x[4], y[4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                x[i] = *reinterpret_cast<const float4*>(A0 + i * 16 * LD + d);
-                y[i] = *reinterpret_cast<const float4*>(B0 + i * 16 * LD + d);
-            }
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    acc[i][j] = fmaf(x[i].x, y[j].x, acc[i][j]);
-                    acc[i][j] = fmaf(x[i].y, y[j].y, acc[i][j]);
-                    acc[i][j] = fmaf(x[i].z, y[j].z, acc[i][j]);
-                    acc[i][j] = fmaf(x[i].w, y[j].w, acc[i][j]);
-                }
-        }
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int r = ty + 16 * i, q = tx + 16 * j;
-                const int t = r & 31, jj = q & 31;
-                const bool keep = r < 32 ? jj <= t : jj < t;
-                const float v = keep ? acc[i][j] : 0.f;
-                Gm[r * 68 + q] = v;
-                if (r < 32) (q < 32 ? gP : gQ)[t * DC_C + jj] = v;
-            }
-    }
-    __syncthreads();
-    // (I + M) z = rhs, a column a thread: the D columns of u G_{t-1} give X, the 32 of N give Y
-    for (int col = tid; col < Dp + DC_C; col += blockDim.x) {
-        float z[DC_C];
-        const bool isX = col < Dp;
-#pragma unroll
-        for (int t = 0; t < DC_C; ++t) {
-            float v = isX ? Us[t * LD + col] : Gm[(32 + t) * 68 + (col - Dp)];
-            const float* m = Gm + (32 + t) * 68 + 32;
-#pragma unroll
-            for (int j4 = 0; j4 < (t + 3) / 4; ++j4) {     // (M is zero from column t on)
-                const float4 m4 = *reinterpret_cast<const float4*>(m + 4 * j4);
-                v = fmaf(-m4.x, z[4 * j4], v);
-                if (4 * j4 + 1 < t) v = fmaf(-m4.y, z[4 * j4 + 1], v);
-                if (4 * j4 + 2 < t) v = fmaf(-m4.z, z[4 * j4 + 2], v);
-                if (4 * j4 + 3 < t) v = fmaf(-m4.w, z[4 * j4 + 3], v);
-            }
-            z[t] = v;
-            if (isX) gX[t * Dp + col] = v;
-            else gY[t * DC_C + col - Dp] = v;
-        }
-    }
-}
-
-// STAGES 2: the next chunk's record is fetched while this one is worked on.
-template <typename T, int STAGES>
-__global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkArgs c) {
-    extern __shared__ __align__(16) float dc_smem[];
-    __shared__ int first_s;
-    pdl_wait();
-    const DeltaRuleArgs& a = c.a;
-    const int s = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * DC_EV;
-    const int q0 = a.cu_q[s];
-    const int qlen = a.cu_q[s + 1] - q0;
-    if (qlen <= 0) return;
-    const int slot = a.state_slots[s];
-    if (slot < 0 || slot >= a.num_slots) return;
-    const int tid = threadIdx.x;
-    if (tid == 0) first_s = c.num_tiles;
-    __syncthreads();
-    for (int i = tid; i < c.num_tiles; i += blockDim.x)     // a request's chunks are neighbours in the list, in order
-        if (c.tile_seq[i] == s) { atomicMin(&first_s, i); break; }
-    __syncthreads();
-    const int first = first_s;
-    const int count = (qlen + DC_C - 1) / DC_C;
-    if (first + count > c.num_tiles) return;
-    const int D = a.D, Dv = a.Dv, Dp = dc_pad(D), LD = Dp + 4;
-    // a stage: X [C][LD], R [C][LD], K [C][Dp], B [C][Dp], Y, P, Q [C][C], G [Dp], V [C][EV]
-    const int XR = 2 * DC_C * LD, KB = 2 * DC_C * Dp, YPQ = 3 * DC_C * DC_C;
-    const int stage_floats = XR + KB + YPQ + Dp + DC_C * DC_EV;
-    float* Ss = dc_smem;                                    // [Dp][EV]
-    float* Sn = Ss + Dp * DC_EV;                            // [C][EV]: seen
-    float* stages = Sn + DC_C * DC_EV;
-    const T* proj = reinterpret_cast<const T*>(a.proj);
-    float* gS = a.state + (size_t)slot * a.state_stride + (size_t)h * D * Dv;
-    for (int idx = tid; idx < Dp * DC_EV; idx += blockDim.x) {
-        const int d = idx / DC_EV, e = e0 + idx % DC_EV;
-        Ss[idx] = d < D && e < Dv ? gS[(size_t)d * Dv + e] : 0.f;
-    }
-    const int dq = Dp / 4;
-    auto fetch = [&](int k) {
-        float* b = stages + (k % STAGES) * stage_floats;
-        const float* rec = c.work + ((size_t)(first + k) * a.H + h) * dc_floats(D);
-        for (int idx = tid; idx < 2 * DC_C * dq; idx += blockDim.x) {
-            const int r = idx / dq, d4 = idx - r * dq;
-            slb_mma::cp_async16(b + r * LD + d4 * 4, rec + r * Dp + d4 * 4, true);
-        }
-        const float* rest = rec + 2 * DC_C * Dp;
-        float* dst = b + XR;
-        const int quads = (KB + YPQ + Dp) / 4;
-        for (int idx = tid; idx < quads; idx += blockDim.x) slb_mma::cp_async16(dst + idx * 4, rest + idx * 4, true);
-        slb_mma::cp_async_commit();
-        float* vs = b + XR + KB + YPQ + Dp;
-        for (int idx = tid; idx < DC_C * DC_EV; idx += blockDim.x) {
-            const int j = idx / DC_EV, e = e0 + idx % DC_EV;
-            const int t = k * DC_C + j;
-            vs[idx] = t < qlen && e < Dv ? to_float(proj[(size_t)(q0 + t) * a.ld + a.v_off + h * Dv + e]) : 0.f;
-        }
-    };
-    if (STAGES == 2) fetch(0);
-    const int cq = (tid & 3) * 4, row = tid >> 2;
-    for (int k = 0; k < count; ++k) {
-        if (STAGES == 2) {
-            if (k + 1 < count) {
-                fetch(k + 1);
-                slb_mma::cp_async_wait<1>();
-            } else {
-                slb_mma::cp_async_wait<0>();
-            }
-        } else {
-            fetch(k);
-            slb_mma::cp_async_wait<0>();
-        }
-        __syncthreads();
-        const float* b = stages + (k % STAGES) * stage_floats;
-        const float* Kd = b + XR, *Bd = Kd + DC_C * Dp, *Ym = b + XR + KB, *Pm = Ym + DC_C * DC_C, *Qm = Pm + DC_C * DC_C;
-        const float* G = b + XR + KB + YPQ, *V = G + Dp;
-        // rows 0..31: X S (+ Y V = seen); rows 32..63: R S, the state's part of the outputs
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
-#define DC_ROW(xv, s4)                                                                           \
-        acc[0] = fmaf(xv, s4.x, acc[0]); acc[1] = fmaf(xv, s4.y, acc[1]);                          \
-        acc[2] = fmaf(xv, s4.z, acc[2]); acc[3] = fmaf(xv, s4.w, acc[3]);
-        const float* xr = b + row * LD;
-#pragma unroll 4
-        for (int d = 0; d < Dp; d += 4) {
-            const float4 x4 = *reinterpret_cast<const float4*>(xr + d);
-            const float4 s0 = *reinterpret_cast<const float4*>(Ss + d * DC_EV + cq);
-            const float4 s1 = *reinterpret_cast<const float4*>(Ss + (d + 1) * DC_EV + cq);
-            const float4 s2 = *reinterpret_cast<const float4*>(Ss + (d + 2) * DC_EV + cq);
-            const float4 s3 = *reinterpret_cast<const float4*>(Ss + (d + 3) * DC_EV + cq);
-            DC_ROW(x4.x, s0) DC_ROW(x4.y, s1) DC_ROW(x4.z, s2) DC_ROW(x4.w, s3)
-        }
-        {
-            // both halves add their product with V: Y for the seen rows, P for the outputs
-            const float* m = row < DC_C ? Ym + row * DC_C : Pm + (row - DC_C) * DC_C;
-#pragma unroll 2
-            for (int j = 0; j < DC_C; j += 4) {
-                const float4 m4 = *reinterpret_cast<const float4*>(m + j);
-                const float4 v0 = *reinterpret_cast<const float4*>(V + j * DC_EV + cq);
-                const float4 v1 = *reinterpret_cast<const float4*>(V + (j + 1) * DC_EV + cq);
-                const float4 v2 = *reinterpret_cast<const float4*>(V + (j + 2) * DC_EV + cq);
-                const float4 v3 = *reinterpret_cast<const float4*>(V + (j + 3) * DC_EV + cq);
-                DC_ROW(m4.x, v0) DC_ROW(m4.y, v1) DC_ROW(m4.z, v2) DC_ROW(m4.w, v3)
-            }
-        }
-        if (row < DC_C) *reinterpret_cast<float4*>(Sn + row * DC_EV + cq) = make_float4(acc[0], acc[1], acc[2], acc[3]);
-        __syncthreads();
-        if (row >= DC_C) {
-            const int t = row - DC_C;
-            const float* m = Qm + t * DC_C;
-#pragma unroll 2
-            for (int j = 0; j < DC_C; j += 4) {
-                const float4 m4 = *reinterpret_cast<const float4*>(m + j);
-                const float4 v0 = *reinterpret_cast<const float4*>(Sn + j * DC_EV + cq);
-                const float4 v1 = *reinterpret_cast<const float4*>(Sn + (j + 1) * DC_EV + cq);
-                const float4 v2 = *reinterpret_cast<const float4*>(Sn + (j + 2) * DC_EV + cq);
-                const float4 v3 = *reinterpret_cast<const float4*>(Sn + (j + 3) * DC_EV + cq);
-                DC_ROW(-m4.x, v0) DC_ROW(-m4.y, v1) DC_ROW(-m4.z, v2) DC_ROW(-m4.w, v3)
-            }
-            const int tt = k * DC_C + t;
-            if (tt < qlen) {
-                float* o = a.out + (size_t)(q0 + tt) * a.ldo + h * Dv + e0 + cq;
-                if ((Dv & 3) == 0 && (a.ldo & 3) == 0) {
-                    if (e0 + cq < Dv) *reinterpret_cast<float4*>(o) = make_float4(acc[0], acc[1], acc[2], acc[3]);
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 4; ++i)
-                        if (e0 + cq + i < Dv) o[i] = acc[i];
-                }
-            }
-        }
-#undef DC_ROW
-        // S <- G S + K^T V - B^T seen: a thread two neighbouring rows of four columns at a time
-        for (int d = row * 2; d < Dp; d += 128) {
-            float4 s0 = *reinterpret_cast<const float4*>(Ss + d * DC_EV + cq);
-            float4 s1 = *reinterpret_cast<const float4*>(Ss + (d + 1) * DC_EV + cq);
-            const float g0 = G[d], g1 = G[d + 1];
-            s0.x *= g0; s0.y *= g0; s0.z *= g0; s0.w *= g0;
-            s1.x *= g1; s1.y *= g1; s1.z *= g1; s1.w *= g1;
-#pragma unroll 4
-            for (int j = 0; j < DC_C; ++j) {
-                const float2 k2 = *reinterpret_cast<const float2*>(Kd + j * Dp + d);
-                const float2 b2 = *reinterpret_cast<const float2*>(Bd + j * Dp + d);
-                const float4 v = *reinterpret_cast<const float4*>(V + j * DC_EV + cq);
-                const float4 q = *reinterpret_cast<const float4*>(Sn + j * DC_EV + cq);
-                s0.x = fmaf(k2.x, v.x, fmaf(-b2.x, q.x, s0.x));
-                s0.y = fmaf(k2.x, v.y, fmaf(-b2.x, q.y, s0.y));
-                s0.z = fmaf(k2.x, v.z, fmaf(-b2.x, q.z, s0.z));
-                s0.w = fmaf(k2.x, v.w, fmaf(-b2.x, q.w, s0.w));
-                s1.x = fmaf(k2.y, v.x, fmaf(-b2.y, q.x, s1.x));
-                s1.y = fmaf(k2.y, v.y, fmaf(-b2.y, q.y, s1.y));
-                s1.z = fmaf(k2.y, v.z, fmaf(-b2.y, q.z, s1.z));
-                s1.w = fmaf(k2.y, v.w, fmaf(-b2.y, q.w, s1.w));
-            }
-            *reinterpret_cast<float4*>(Ss + d * DC_EV + cq) = s0;
-            *reinterpret_cast<float4*>(Ss + (d + 1) * DC_EV + cq) = s1;
-        }
-        __syncthreads();                                   // (the stage may be filled again, S is whole)
-    }
-    pdl_launch_dependents();
-    for (int idx = tid; idx < D * DC_EV; idx += blockDim.x) {
-        const int d = idx / DC_EV, e = e0 + idx % DC_EV;
-        if (e < Dv) gS[(size_t)d * Dv + e] = Ss[idx];
-    }
-}
-
-static size_t dc_scan_smem(int D, int stages) {
-    const size_t Dp = dc_pad(D);
-    const size_t stage = (size_t)2 * DC_C * (Dp + 4) + 2 * DC_C * Dp + 3 * DC_C * DC_C + Dp + DC_C * DC_EV;
-    return (Dp * DC_EV + DC_C * DC_EV + stages * stage) * sizeof(float);
-}
-
-template <typename T>
-static int launch_delta_chunk(const DeltaChunkArgs& c, int num_seqs, cudaStream_t st) {
-    if (num_seqs <= 0 || c.num_tiles <= 0) return 0;
-    const DeltaRuleArgs& a = c.a;
-    int rc = dr_check(a);
-    if (rc != 0) return rc;
-    if (a.out == nullptr || c.work == nullptr || c.tile_seq == nullptr || c.tile_row0 == nullptr ||
-        ((uintptr_t)c.work & 15) || ((uintptr_t)a.out & 15) || a.decay_coef > 2.0f)
-        return SLB_ERR_BAD_ARG;
-    if (num_seqs > 65535) return SLB_ERR_TOO_LARGE;
-    const int Dp = dc_pad(a.D), vz = (a.Dv + DC_EV - 1) / DC_EV;
-    const size_t smem1 = ((size_t)5 * DC_C * (Dp + 4) + 64 * 68) * sizeof(float);
-    static unsigned long long conf1 = 0, conf2 = 0, conf3 = 0;
-    rc = slb_configure(&conf1, delta_chunk_prep_kernel<T>, ((size_t)5 * DC_C * (DR_MAX_D + 4) + 64 * 68) * sizeof(float));
-    if (rc != 0) return rc;
-    rc = slb_launch(delta_chunk_prep_kernel<T>, dim3(c.num_tiles, a.H), dim3(256), smem1, st, c);
-    if (rc != 0) return rc;
-    if (a.D <= 128) {
-        rc = slb_configure(&conf2, delta_chunk_scan_kernel<T, 2>, dc_scan_smem(128, 2));
-        if (rc != 0) return rc;
-        return slb_launch(delta_chunk_scan_kernel<T, 2>, dim3(num_seqs, a.H, vz), dim3(256), dc_scan_smem(a.D, 2), st, c);
-    }
-    rc = slb_configure(&conf3, delta_chunk_scan_kernel<T, 1>, dc_scan_smem(DR_MAX_D, 1));
-    if (rc != 0) return rc;
-    return slb_launch(delta_chunk_scan_kernel<T, 1>, dim3(num_seqs, a.H, vz), dim3(256), dc_scan_smem(a.D, 1), st, c);
-}
-
 extern "C" {
 int slb_delta_rule_max_dim() { return DR_MAX_D; }
 // 1 if the token-by-token kernel's block holds every value column of a head (the fused norm and gate)
@@ -642,13 +242,5 @@ int slb_delta_rule_f32(const DeltaRuleArgs* a, int num_seqs, cudaStream_t st) {
 }
 int slb_delta_rule_bf16(const DeltaRuleArgs* a, int num_seqs, cudaStream_t st) {
     return launch_delta_rule<bf16>(*a, num_seqs, st);
-}
-int slb_delta_chunk_tokens() { return DC_C; }
-int slb_delta_chunk_work_floats(int D) { return (int)dc_floats(D); }
-int slb_delta_chunk_f32(const DeltaChunkArgs* c, int num_seqs, cudaStream_t st) {
-    return launch_delta_chunk<float>(*c, num_seqs, st);
-}
-int slb_delta_chunk_bf16(const DeltaChunkArgs* c, int num_seqs, cudaStream_t st) {
-    return launch_delta_chunk<bf16>(*c, num_seqs, st);
 }
 }

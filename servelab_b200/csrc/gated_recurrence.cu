@@ -7,9 +7,14 @@
 // come from block-diagonal products: block b of n channels has its logits at z + b * z_block +
 // token * z_token, n for r and then n for i.  Everything here is float32; S is zero for a new request.
 //
-// A block owns 16 channels of a request and takes its tokens 64 at a time: all threads form a and the
-// update of every (token, channel), 16 threads walk the tokens (one multiply-add each, in order, so the
-// result of a token does not depend on how the request was cut), all threads finish the outputs.
+// Token by token (float32 rows, steps of single tokens): a block owns 16 channels of a request and takes
+// its tokens 64 at a time: all threads form a and the update of every (token, channel), 16 threads walk
+// the tokens (one multiply-add each, in order, so the result of a token does not depend on how the
+// request was cut), all threads finish the outputs.
+//
+// In segments (bfloat16 rows of longer portions): 32 segments of 8 tokens at a time, a thread a (segment,
+// channel).  A segment is S -> A S + B; each thread forms its own pair, takes the segments before it
+// from shared memory, and walks its tokens once more from the state that enters.
 #include "common.cuh"
 
 #define GR_EC 16
@@ -101,8 +106,85 @@ __global__ void __launch_bounds__(256) gated_recurrence_kernel(const GatedRecArg
     if (tk == 0 && live) *sp = S;
 }
 
+#define GR_SEGS 32
+#define GR_SEG_TOKENS 8
+
 template <typename T>
-static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, cudaStream_t st) {
+__global__ void __launch_bounds__(GR_EC * GR_SEGS) gated_recurrence_segments_kernel(const GatedRecArgs g) {
+    __shared__ float2 pairs[2][GR_SEGS][GR_EC];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.x, c0 = blockIdx.y * GR_EC;
+    const int q0 = g.cu_q[s];
+    const int qlen = g.cu_q[s + 1] - q0;
+    if (qlen <= 0) return;
+    const int slot = g.state_slots[s];
+    if (slot < 0 || slot >= g.num_slots) return;
+    const int ch = threadIdx.x % GR_EC, seg = threadIdx.x / GR_EC;
+    const int c = c0 + ch;
+    const bool live = c < g.width;
+    const T* u = reinterpret_cast<const T*>(g.u);
+    const T* y = reinterpret_cast<const T*>(g.y);
+    T* out = reinterpret_cast<T*>(g.out);
+    float rb = 0.f, ib = 0.f, rate = 0.f, yb = 0.f, S = 0.f;
+    const float* z = g.z;
+    float* sp = g.state + (size_t)slot * g.state_stride + c;
+    if (live) {
+        rb = g.r_bias[c]; ib = g.i_bias[c]; rate = g.rate[c]; yb = g.y_bias[c];
+        const int b = c / g.n;
+        z += (size_t)b * g.z_block + (c - b * g.n);
+        S = *sp;
+    }
+    for (int t0 = 0, k = 0; t0 < qlen; t0 += GR_SEGS * GR_SEG_TOKENS, ++k) {
+        const int first = t0 + seg * GR_SEG_TOKENS;
+        float zr[GR_SEG_TOKENS], zi[GR_SEG_TOKENS], uv[GR_SEG_TOKENS], yv[GR_SEG_TOKENS];
+#pragma unroll
+        for (int i = 0; i < GR_SEG_TOKENS; ++i) {
+            zr[i] = zi[i] = uv[i] = yv[i] = 0.f;
+            if (live && first + i < qlen) {
+                const size_t t = q0 + first + i;
+                zr[i] = z[t * g.z_token];
+                zi[i] = z[t * g.z_token + g.n];
+                uv[i] = to_float(u[t * g.ldu + c]);
+                yv[i] = to_float(y[t * g.ldy + c]);
+            }
+        }
+        float A = 1.f, B = 0.f;                  // (zr becomes a, zi the update)
+#pragma unroll
+        for (int i = 0; i < GR_SEG_TOKENS; ++i) {
+            float a = 1.f, b = 0.f;
+            if (live && first + i < qlen) {
+                float gain;
+                gr_decay(rate * gr_sigmoid(zr[i] + rb), a, gain);
+                b = gain * gr_sigmoid(zi[i] + ib) * uv[i];
+            }
+            zr[i] = a;
+            zi[i] = b;
+            A *= a;
+            B = fmaf(a, B, b);
+        }
+        float2 (*row)[GR_EC] = pairs[k & 1];     // (two buffers: one barrier a round)
+        row[seg][ch] = make_float2(A, B);
+        __syncthreads();
+        float enter = S;
+#pragma unroll 8
+        for (int i = 0; i < GR_SEGS; ++i) {
+            if (i == seg) enter = S;
+            const float2 p = row[i][ch];
+            S = fmaf(p.x, S, p.y);
+        }
+#pragma unroll
+        for (int i = 0; i < GR_SEG_TOKENS; ++i) {
+            enter = fmaf(zr[i], enter, zi[i]);
+            if (live && first + i < qlen)
+                out[(size_t)(q0 + first + i) * g.ldo + c] = from_float<T>(enter * gr_gelu_tanh(yv[i] + yb));
+        }
+    }
+    if (seg == 0 && live) *sp = S;
+}
+
+template <typename T>
+static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, int segments, cudaStream_t st) {
     if (num_seqs <= 0) return 0;
     if (g.width <= 0 || g.n <= 0 || g.width % g.n || g.u == nullptr || g.z == nullptr || g.y == nullptr ||
         g.state == nullptr || g.state_stride < g.width || g.num_slots <= 0 || g.r_bias == nullptr ||
@@ -110,14 +192,16 @@ static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, cudaStre
         return SLB_ERR_BAD_ARG;
     const int gy = (g.width + GR_EC - 1) / GR_EC;
     if (gy > 65535) return SLB_ERR_TOO_LARGE;
+    if (segments)
+        return slb_launch(gated_recurrence_segments_kernel<T>, dim3(num_seqs, gy), dim3(GR_EC * GR_SEGS), 0, st, g);
     return slb_launch(gated_recurrence_kernel<T>, dim3(num_seqs, gy), dim3(256), 0, st, g);
 }
 
 extern "C" {
-int slb_gated_recurrence_f32(const GatedRecArgs* g, int num_seqs, cudaStream_t st) {
-    return launch_gated_recurrence<float>(*g, num_seqs, st);
+int slb_gated_recurrence_f32(const GatedRecArgs* g, int num_seqs, int segments, cudaStream_t st) {
+    return launch_gated_recurrence<float>(*g, num_seqs, segments, st);
 }
-int slb_gated_recurrence_bf16(const GatedRecArgs* g, int num_seqs, cudaStream_t st) {
-    return launch_gated_recurrence<bf16>(*g, num_seqs, st);
+int slb_gated_recurrence_bf16(const GatedRecArgs* g, int num_seqs, int segments, cudaStream_t st) {
+    return launch_gated_recurrence<bf16>(*g, num_seqs, segments, st);
 }
 }

@@ -1665,6 +1665,9 @@ class _GatedRecArgs(_ct.Structure):
     ]
 
 
+force_gated_recurrence_segments = False       # (tests: the segmented kernel also for float32 rows)
+
+
 def gated_recurrence(ctx, u: torch.Tensor, z: torch.Tensor, y: torch.Tensor, state: torch.Tensor, out: torch.Tensor, *,
                      r_bias: torch.Tensor, i_bias: torch.Tensor, rate: torch.Tensor, y_bias: torch.Tensor) -> None:
     """S_t = a S_{t-1} + sqrt(1 - a^2) i u with log a = rate * r per channel, out = S * gelu_tanh(y + y_bias)
@@ -1680,4 +1683,5 @@ def gated_recurrence(ctx, u: torch.Tensor, z: torch.Tensor, y: torch.Tensor, sta
     g.width, g.n = out.shape[1], z.shape[2] // 2
     g.out, g.ldo = out.data_ptr(), out.stride(0)
     fn = getattr(L.core(), "slb_gated_recurrence_" + _suffix(out.dtype))
-    L.check(fn(_ct.byref(g), ctx.num_seqs, _stream()), "gated_recurrence")
+    segments = not ctx.decode_only and (force_gated_recurrence_segments or out.dtype == _BF16)
+    L.check(fn(_ct.byref(g), ctx.num_seqs, int(segments), _stream()), "gated_recurrence")

@@ -95,8 +95,8 @@ _CORE_SIGNATURES = {
     "slb_delta_chunk_work_floats": [I],
     "slb_delta_chunk_f32": [P, I, P],
     "slb_delta_chunk_bf16": [P, I, P],
-    "slb_gated_recurrence_f32": [P, I, P],
-    "slb_gated_recurrence_bf16": [P, I, P],
+    "slb_gated_recurrence_f32": [P, I, I, P],
+    "slb_gated_recurrence_bf16": [P, I, I, P],
     "slb_moe_tile_rows": [],
     "slb_moe_route": [P, I, I, I, I, I, I, F, I, P, P, P],
     "slb_moe_route_scored": [P, I, I, I, I, I, I, F, I, I, P, I, F, P, P, P],

@@ -503,14 +503,18 @@ def test_recurrence_with_a_bonus_and_double_exponential_decays(dtype, shape, shi
 
 @pytest.mark.parametrize("dtype", BOTH)
 @pytest.mark.parametrize("shape", [(36, 3, 3), (30, 5, 1), (128, 1, 5), (96, 6, 2), (1040, 2, 4), (17, 1, 2)])
-def test_gated_recurrence_with_its_convolution(dtype, shape):
+@pytest.mark.parametrize("segments", [False, True])
+def test_gated_recurrence_with_its_convolution(dtype, shape, segments, monkeypatch):
     """Convolution with its biases (whose zeros before the start stay zeros), block-diagonal gates and the
-    recurrence: whole, in portions, token by token, decays near 1 and fast ones."""
+    recurrence: whole, in portions, token by token, decays near 1 and fast ones; with `segments` the
+    kernel that takes longer portions 256 tokens at a time."""
+    from servelab_b200.ops import kernels as K
     from servelab_b200.config.specs import GatedRecurrenceSpec
     from servelab_b200.parts import BuildEnv, LayerCache
     from servelab_b200.parts.gated_recurrence import GatedRecurrence
     width, blocks, taps = shape
-    hidden, n, m = 40, 150, 9
+    hidden, n, m = 40, 530 if segments else 150, 9
+    monkeypatch.setattr(K, "force_gated_recurrence_segments", segments)
     g = torch.Generator().manual_seed(width)
     spec = GatedRecurrenceSpec(hidden_size=hidden, width=width, blocks=blocks, conv_taps=taps)
     W = {}
@@ -539,7 +543,7 @@ def test_gated_recurrence_with_its_convolution(dtype, shape):
         _close(got, want, 1e-5 if dtype == torch.float32 else 2e-2, name)
         assert float(state[1].min()) == 3.0
         results.append(got)
-    if dtype == torch.float32:
+    if dtype == torch.float32 and not segments:
         assert torch.equal(results[0], results[1]) and torch.equal(results[0], results[2])
     keep = state.clone()
     mixer.forward(_padded_ctx([_entry(2, 0, (), 1)], 16, 2), xd[:16].contiguous(), LayerCache(state=state), True)
