@@ -20,8 +20,9 @@
 // in shared memory; `scan` walks a request's chunks with 16 value columns of the state a block, a
 // chunk's record fetched as one bulk copy while the one before is worked on.
 //
-// The products run on mma.sync with every float32 operand split into two TF32 numbers (mma_split);
-// everything else, the solve and the decays included, is float32.
+// The products run on mma.sync with every float32 operand split into two TF32 numbers (the
+// product of the two low parts is left out: it is below float32's own rounding);
+// bfloat16 values need one); everything else, the solve and the decays included, is float32.
 #include "delta_rule.cuh"
 #include "mma_util.cuh"
 
@@ -73,21 +74,31 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const DeltaChunkA
     {
         const T* row = reinterpret_cast<const T*>(a.proj) + (size_t)t0 * a.ld + h * D;
         const float* zrow = a.gate_z + (size_t)t0 * a.ld_gate + h * D;
-#pragma unroll 4
-        for (int idx = tid; idx < DC_C * Dp; idx += 256) {
-            const int j = idx / Dp, d = idx - j * Dp;
-            float l = 0.f, k = 0.f, r = 0.f, b = 0.f;
-            if (j < n && d < D) {
-                const T* p = row + (size_t)j * a.ld + d;
-                l = zrow[(size_t)j * a.ld_gate + d];
-                k = to_float(p[a.k_off]);
-                r = to_float(p[a.r_off]);
-                b = to_float(p[a.a_off]) + a.a_bias[h * D + d];
-                l = -a.decay_coef * dr_sigmoid(l);
-                b = dr_sigmoid(b);
+for (int d = lane; d < Dp; d += 32) {        // (a warp has the four rows from 4 warp)
+            const bool live = d < D;
+            const float ab = live ? a.a_bias[h * D + d] : 0.f;
+            float l[4], k[4], r[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int j = warp * 4 + i;
+                l[i] = k[i] = r[i] = b[i] = 0.f;
+                if (live && j < n) {
+                    const T* p = row + (size_t)j * a.ld + d;
+                    l[i] = zrow[(size_t)j * a.ld_gate + d];
+                    k[i] = to_float(p[a.k_off]);
+                    r[i] = to_float(p[a.r_off]);
+                    b[i] = to_float(p[a.a_off]);
+                }
             }
-            const int at = j * LX + d;
-            Ls[at] = l; Ks[at] = k; Rs[at] = r; Bs[at] = b;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int at = (warp * 4 + i) * LX + d;
+                const bool in = live && warp * 4 + i < n;
+                Ls[at] = in ? -a.decay_coef * dr_sigmoid(l[i]) : 0.f;
+                Ks[at] = k[i];
+                Rs[at] = r[i];
+                Bs[at] = in ? dr_sigmoid(b[i] + ab) : 0.f;
+            }
         }
     }
     __syncthreads();
@@ -102,23 +113,31 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const DeltaChunkA
     float* rec = c.work + ((size_t)tile * a.H + h) * dc_floats(D);
     float* gX = rec, *gR = gX + DC_C * LX, *gK = gR + DC_C * LX, *gB = gK + DC_C * LK;
     float* gY = gB + DC_C * LK, *gP = gY + DC_C * DC_LM, *gQ = gP + DC_C * DC_LM, *gG = gQ + DC_C * DC_LM;
-    for (int j = warp; j < DC_C; j += 8) {
-        float ss = 0.f;
-        for (int d = lane; d < Dp; d += 32) ss = fmaf(Ks[j * LX + d], Ks[j * LX + d], ss);
-        ss = warp_sum(ss);
-        const float inv = 1.0f / sqrtf(ss + a.unit_eps);
+    {
+        const int j0 = warp * 4;
+        float inv[4] = {};
+        for (int d = lane; d < Dp; d += 32)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) inv[i] = fmaf(Ks[(j0 + i) * LX + d], Ks[(j0 + i) * LX + d], inv[i]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) inv[i] = 1.0f / sqrtf(warp_sum(inv[i]) + a.unit_eps);
         for (int d = lane; d < Dp; d += 32) {
-            const int at = j * LX + d;
-            const float L = Ls[at], Lp = j > 0 ? Ls[at - LX] : 0.f, Le = Ls[(DC_C - 1) * LX + d];
-            const float k = Ks[at], u = k * inv, b = Bs[at] * u;
-            const float up = expf(-L), rest = expf(Le - L), rg = Rs[at] * expf(L);
-            Rs[at] = rg;
-            Us[at] = u * expf(Lp);
-            Ks[at] = k * up;
-            Bs[at] = b * up;
-            gR[at] = rg;
-            gK[j * LK + d] = k * rest;
-            gB[j * LK + d] = b * rest;
+            const float Le = Ls[(DC_C - 1) * LX + d];
+            float before = j0 > 0 ? expf(Ls[(j0 - 1) * LX + d]) : 1.0f;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int at = (j0 + i) * LX + d;
+                const float L = Ls[at], k = Ks[at], u = k * inv[i], b = Bs[at] * u;
+                const float now = expf(L), up = expf(-L), rest = expf(Le - L), rg = Rs[at] * now;
+                Rs[at] = rg;
+                Us[at] = u * before;
+                Ks[at] = k * up;
+                Bs[at] = b * up;
+                gR[at] = rg;
+                gK[(j0 + i) * LK + d] = k * rest;
+                gB[(j0 + i) * LK + d] = b * rest;
+                before = now;
+            }
         }
     }
     for (int d = tid; d < Dp; d += 256) gG[d] = decay_exp(Ls[(DC_C - 1) * LX + d]);
@@ -179,13 +198,13 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const DeltaChunkA
     }
 }
 
-// acc += A B over `steps` contraction steps of 8.  A's fragment starts at A (+ row8 for the row 8 below,
+// acc += A B over `steps` contraction steps of 8, the cross terms of the split in chains of their own (low).  A's fragment starts at A (+ row8 for the row 8 below,
 // + k4 for the contraction 4 further, + k8 a step); B is [column][contraction] with stride ldb, B already
-// at this lane's column and contraction, NT tiles of 8 columns.
-template <int NT>
-__device__ __forceinline__ void dc_product(float (&acc)[NT][4], float (&low)[NT][4], const float* A, int row8,
+// at this lane's column and contraction, NT tiles of 8 columns; EXACT: B's elements are TF32 numbers.
+template <int NT, bool EXACT>
+__device__ __forceinline__ void dc_product(float (&acc)[NT][4], float (&low)[2][NT][4], const float* A, int row8,
                                            int k4, int k8, const float* B, int ldb, int steps) {
-#pragma unroll 4
+#pragma unroll 8
     for (int s = 0; s < steps; ++s) {
         unsigned ah[4], al[4];
 #pragma unroll
@@ -195,27 +214,27 @@ __device__ __forceinline__ void dc_product(float (&acc)[NT][4], float (&low)[NT]
             unsigned bh[2], bl[2];
             slb_mma::split_tf32(B[q * 8 * ldb + s * 8], bh[0], bl[0]);
             slb_mma::split_tf32(B[q * 8 * ldb + s * 8 + 4], bh[1], bl[1]);
-            slb_mma::mma_tf32(low[q], al, bh);
+            slb_mma::mma_tf32(low[0][q], al, bh);
             slb_mma::mma_tf32(acc[q], ah, bh);
-            slb_mma::mma_tf32(low[q], ah, bl);
+            if (!EXACT) slb_mma::mma_tf32(low[1][q], ah, bl);
         }
     }
 }
 
 // S <- G S + K^T V + B^T (-seen) for the 16 rows from d0 and NT tiles of 8 value columns from n0
-template <int NT>
+template <int NT, bool EXACT>
 __device__ __forceinline__ void dc_update(float* Ss, int LX, const float* G, const float* Kd, const float* Bd, int LK,
                                           const float* Vt, const float* Nt, int d0, int n0, int g, int t) {
-    float acc[NT][4] = {}, low[NT][4] = {};
-    dc_product<NT>(acc, low, Kd + t * LK + d0 + g, 8, 4 * LK, 8 * LK, Vt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
-    dc_product<NT>(acc, low, Bd + t * LK + d0 + g, 8, 4 * LK, 8 * LK, Nt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
+    float acc[NT][4] = {}, low[2][NT][4] = {};
+    dc_product<NT, EXACT>(acc, low, Kd + t * LK + d0 + g, 8, 4 * LK, 8 * LK, Vt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
+    dc_product<NT, false>(acc, low, Bd + t * LK + d0 + g, 8, 4 * LK, 8 * LK, Nt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
     const float g0 = G[d0 + g], g1 = G[d0 + g + 8];
 #pragma unroll
     for (int q = 0; q < NT; ++q)
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             float* s = Ss + (n0 + q * 8 + 2 * t + (i & 1)) * LX + d0 + g + (i >> 1) * 8;
-            *s = fmaf(i >> 1 ? g1 : g0, *s, acc[q][i] + low[q][i]);
+            *s = fmaf(i >> 1 ? g1 : g0, *s, acc[q][i] + (low[0][q][i] + low[1][q][i]));
         }
 }
 
@@ -223,6 +242,7 @@ __device__ __forceinline__ void dc_update(float* Ss, int LX, const float* G, con
 template <typename T, int STAGES>
 __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkArgs c) {
     extern __shared__ __align__(16) float dc_smem[];
+    constexpr bool EXACT = sizeof(T) == 2;           // (a bfloat16 value is a TF32 number)
     __shared__ int first_s;
     __shared__ __align__(8) uint64_t bars[STAGES];
     pdl_wait();
@@ -293,17 +313,17 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
         const float* Kd = b + 2 * DC_C * LX, *Bd = Kd + DC_C * LK, *Ym = Bd + DC_C * LK, *Qm = Ym + 2 * DC_C * DC_LM;
         const float* G = Qm + DC_C * DC_LM, *Vt = Vts + (k & 1) * DC_EV * DC_LM;
         // rows 0..31: X S + Y V = seen; rows 32..63: R S + P V, the outputs without what was removed
-        float acc[1][4] = {}, low[1][4] = {};
-        dc_product<1>(acc, low, b + (m0 + g) * LX + t, 8 * LX, 4, 8, Ss + (n0 + g) * LX + t, LX, Dp / 8);
-        dc_product<1>(acc, low, Ym + (m0 + g) * DC_LM + t, 8 * DC_LM, 4, 8, Vt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
+        float acc[1][4] = {}, low[2][1][4] = {};
+        dc_product<1, false>(acc, low, b + (m0 + g) * LX + t, 8 * LX, 4, 8, Ss + (n0 + g) * LX + t, LX, Dp / 8);
+        dc_product<1, EXACT>(acc, low, Ym + (m0 + g) * DC_LM + t, 8 * DC_LM, 4, 8, Vt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
         if (m0 < DC_C) {
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-                Nt[(n0 + 2 * t + (i & 1)) * DC_LM + m0 + g + (i >> 1) * 8] = -(acc[0][i] + low[0][i]);
+                Nt[(n0 + 2 * t + (i & 1)) * DC_LM + m0 + g + (i >> 1) * 8] = -(acc[0][i] + (low[0][0][i] + low[1][0][i]));
         }
         __syncthreads();
         if (m0 >= DC_C) {
-            dc_product<1>(acc, low, Qm + (m0 - DC_C + g) * DC_LM + t, 8 * DC_LM, 4, 8, Nt + (n0 + g) * DC_LM + t, DC_LM,
+            dc_product<1, false>(acc, low, Qm + (m0 - DC_C + g) * DC_LM + t, 8 * DC_LM, 4, 8, Nt + (n0 + g) * DC_LM + t, DC_LM,
                           DC_C / 8);
             const int e = e0 + n0 + 2 * t;
 #pragma unroll
@@ -311,7 +331,7 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
                 const int tt = k * DC_C + m0 - DC_C + g + i * 4;
                 if (tt >= qlen || e >= Dv) continue;
                 float* o = a.out + (size_t)(q0 + tt) * a.ldo + h * Dv + e;
-                const float x = acc[0][i] + low[0][i], y = acc[0][i + 1] + low[0][i + 1];
+                const float x = acc[0][i] + (low[0][0][i] + low[1][0][i]), y = acc[0][i + 1] + (low[0][0][i + 1] + low[1][0][i + 1]);
                 if ((Dv & 1) == 0 && (a.ldo & 1) == 0) {
                     *reinterpret_cast<float2*>(o) = make_float2(x, y);
                 } else {
@@ -321,9 +341,9 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
             }
         }
         if (Dp > 64) {
-            for (int d0 = warp * 16; d0 < Dp; d0 += 128) dc_update<2>(Ss, LX, G, Kd, Bd, LK, Vt, Nt, d0, 0, g, t);
+            for (int d0 = warp * 16; d0 < Dp; d0 += 128) dc_update<2, EXACT>(Ss, LX, G, Kd, Bd, LK, Vt, Nt, d0, 0, g, t);
         } else if (m0 < Dp) {
-            dc_update<1>(Ss, LX, G, Kd, Bd, LK, Vt, Nt, m0, n0, g, t);
+            dc_update<1, EXACT>(Ss, LX, G, Kd, Bd, LK, Vt, Nt, m0, n0, g, t);
         }
         if (more) store_v(k + 1);
         if (STAGES == 1 && more) {

@@ -43,26 +43,11 @@ __device__ __forceinline__ void mma_tf32(float (&c)[4], const unsigned (&a)[4], 
         : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
         : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
-__device__ __forceinline__ unsigned to_tf32(float x) {
-    unsigned r;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
-    return r;
-}
+// (the unit reads the upper 19 bits of an operand: what the high part leaves has at most 13 significant
+// bits, of which it sees 11)
 __device__ __forceinline__ void split_tf32(float x, unsigned& hi, unsigned& lo) {
-    hi = to_tf32(x);
-    lo = to_tf32(x - __uint_as_float(hi));
-}
-// c += a b with both operands split (the product of the two low parts is below float32's own rounding);
-// `low` collects the cross terms on a chain of its own
-__device__ __forceinline__ void mma_split(float (&c)[4], float (&low)[4], const float (&a)[4], const float (&b)[2]) {
-    unsigned ah[4], al[4], bh[2], bl[2];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) split_tf32(a[i], ah[i], al[i]);
-#pragma unroll
-    for (int i = 0; i < 2; ++i) split_tf32(b[i], bh[i], bl[i]);
-    mma_tf32(low, al, bh);
-    mma_tf32(c, ah, bh);
-    mma_tf32(low, ah, bl);
+    hi = __float_as_uint(x) & 0xffffe000u;
+    lo = __float_as_uint(x - __uint_as_float(hi));
 }
 __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
