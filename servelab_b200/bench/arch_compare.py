@@ -467,7 +467,9 @@ def _vufadra_rooflines(size, res, peaks) -> Dict[str, object]:
     win_pairs = sum(min(t + 1, WINDOW) for t in range(PROMPT))
     tc = ("attention_kv_tc", "attention_kv_mma", "prefill_attention_tc", "prefill_attention", "attention_kv")
     row("vufadra_chunk_attention_prefill", vp, tc, 1, lambda us: tf(chunk_pairs * heads * 4 * dim, us))
-    row("sumolorn_attention_prefill", sp, tc, LAYERS, lambda us: tf(win_pairs * heads * 4 * dim, us))
+    # (Sumolorn's three left branches run on the kernel for equal sizes, which takes no modified scores)
+    row("sumolorn_capped_attention_prefill", sp, tc[:2], 1, lambda us: tf(win_pairs * heads * 4 * dim, us))
+    row("sumolorn_plain_attention_prefill", sp, tc[2:4], 3, lambda us: tf(win_pairs * heads * 4 * dim, us))
     row("vufadra_delta_prefill", vp, ("delta_rule (chunks)", "delta_rule"), 2, lambda us: tf(8.0 * PROMPT * state, us))
     lin = ("decay_attention (gated chunks)", "decay_attention")
     row("vufadra_decay_prefill", vp, lin, 1, lambda us: tf(4.0 * PROMPT * state, us))
@@ -494,17 +496,20 @@ def _vufadra_rooflines(size, res, peaks) -> Dict[str, object]:
         # (a context of CONTEXT tokens sits at CONTEXT % WINDOW in its chunk)
         seen_v, seen_s = (CONTEXT - 1) % WINDOW + 1, min(CONTEXT, WINDOW)
         row(f"vufadra_chunk_attention_decode_b{b}", vd, dec, 1, lambda us: hbm(b * seen_v * kv * 4 * dim, us))
-        row(f"sumolorn_attention_decode_b{b}", sd, dec, LAYERS, lambda us: hbm(b * seen_s * kv * 4 * dim, us))
+        row(f"sumolorn_capped_attention_decode_b{b}", sd, dec[:2], 1, lambda us: hbm(b * seen_s * kv * 4 * dim, us))
+        row(f"sumolorn_plain_attention_decode_b{b}", sd, dec[2:], 3, lambda us: hbm(b * seen_s * kv * 4 * dim, us))
         row(f"vufadra_delta_decode_b{b}", vd, "delta_rule", 2, lambda us: hbm(b * state * 8, us))
         row(f"vufadra_decay_decode_b{b}", vd, "decay_attention", 1, lambda us: hbm(b * state * 8, us))
         row(f"sumolorn_decay_decode_b{b}", sd, "decay_attention", 3, lambda us: hbm(b * state * 8, us))
     return out
 
 
-def _measure(cfg: dict, note, graph_prefill: bool = False) -> Dict[str, object]:
+def _measure(cfg: dict, note, graph_prefill: bool = False, queue_ahead: bool = False) -> Dict[str, object]:
     """``graph_prefill``: the prompt's step replays the graph captured for its padded sizes where the
     model allows it (the eager step of a small model is bound by the host's launches); the eager
-    time is reported beside it."""
+    time is reported beside it.  ``queue_ahead``: the steps whose kernels are timed one by one (eager, an
+    event on both sides of each launch) are queued behind a kernel that only waits, so that the device
+    never waits for the host between two events."""
     import torch
     from ..ops import kernels as K
     from ..ops.profile import StepProfile
@@ -544,7 +549,9 @@ def _measure(cfg: dict, note, graph_prefill: bool = False) -> Dict[str, object]:
     ms = out.get("prefill_graph_ms", ms) if out.get("prefill_graph_replays") else ms
     out["prefill_ms"] = round(ms, 3)
     out["prefill_tok_s"] = round(PROMPT / (ms * 1e-3), 1)
+    hold = (lambda: torch.cuda._sleep(20_000_000)) if queue_ahead else (lambda: None)
     with StepProfile() as prof:
+        hold()
         runner.step([entry])
     out["prefill_kernels_us"] = prof.summary(1)
     runner.cuda_graphs = saved
@@ -566,6 +573,7 @@ def _measure(cfg: dict, note, graph_prefill: bool = False) -> Dict[str, object]:
         runner.step(entries)
         with StepProfile() as prof:
             for _ in range(5):
+                hold()
                 runner.step(entries)
         out[f"decode_b{batch}_kernels_us"] = prof.summary(5)
         runner.cuda_graphs = saved
@@ -641,7 +649,7 @@ def run(peaks, note=lambda m: None, sizes=None, design: str = "dezelorn") -> Dic
             res = {}
             for arch, make in (("vufadra", vufadra_config), ("sumolorn", sumolorn_like_vufadra)):
                 note(f"{size}: {arch}")
-                res[arch] = _measure(make(*dims), note, graph_prefill=True)
+                res[arch] = _measure(make(*dims), note, graph_prefill=True, queue_ahead=True)
             res["kernels"] = _vufadra_rooflines(size, res, peaks)
             res["dims"] = dict(zip(("width", "heads", "kv_heads", "head_dim", "ff", "recurrent_heads", "bottleneck"), dims))
             result["sizes"][size] = res

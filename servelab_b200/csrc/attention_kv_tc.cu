@@ -431,14 +431,15 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
             float sm[4] = {0.f, 0.f, 0.f, 0.f};
             uint32_t packed[32];
             if (sig_bias != nullptr) {
-                // sigmoid(x) = 1 / (1 + 2^(-x log2 e)); a masked score (-inf) gives 2^inf and so 0
+                // sigmoid(x) = 1 / (1 + 2^(-x log2 e)); a masked score (-inf) gives 2^inf and so 0 (as every
+                // divisor above 2^126 does)
 #pragma unroll
                 for (int h = 0; h < 2; ++h)
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
                         const float e0 = fast_exp2(fmaf(__uint_as_float(raw[h][i]), -scale_log2, -bias2));
                         const float e1 = fast_exp2(fmaf(__uint_as_float(raw[h][i + 1]), -scale_log2, -bias2));
-                        packed[h * 16 + i / 2] = pack2(__frcp_rn(1.f + e0), __frcp_rn(1.f + e1));
+                        packed[h * 16 + i / 2] = pack2(__fdividef(1.f, 1.f + e0), __fdividef(1.f, 1.f + e1));
                     }
             } else {
             if (mt > m_ref + RESCALE_THRESHOLD || (m_ref == -INFINITY && mt != -INFINITY)) {

@@ -7,7 +7,9 @@
 // come from block-diagonal products: block b of n channels has its logits at z + b * z_block +
 // token * z_token, n for r and then n for i.  Everything here is float32; S is zero for a new request.
 //
-// Token by token (float32 rows, steps of single tokens): a block owns 16 channels of a request and takes
+// Steps of single tokens: a thread a (request, channel).
+//
+// Token by token (float32 rows): a block owns 16 channels of a request and takes
 // its tokens 64 at a time: all threads form a and the update of every (token, channel), 16 threads walk
 // the tokens (one multiply-add each, in order, so the result of a token does not depend on how the
 // request was cut), all threads finish the outputs.
@@ -106,6 +108,31 @@ __global__ void __launch_bounds__(256) gated_recurrence_kernel(const GatedRecArg
     if (tk == 0 && live) *sp = S;
 }
 
+template <typename T>
+__global__ void __launch_bounds__(128) gated_recurrence_step_kernel(const GatedRecArgs g) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.x, c = blockIdx.y * 128 + threadIdx.x;
+    const int q0 = g.cu_q[s], q1 = g.cu_q[s + 1];
+    const int slot = g.state_slots[s];
+    if (q1 <= q0 || slot < 0 || slot >= g.num_slots || c >= g.width) return;
+    const float rb = g.r_bias[c], ib = g.i_bias[c], rate = g.rate[c], yb = g.y_bias[c];
+    const int b = c / g.n;
+    const float* z = g.z + (size_t)b * g.z_block + (c - b * g.n);
+    float* sp = g.state + (size_t)slot * g.state_stride + c;
+    float S = *sp;
+    for (size_t t = q0; t < q1; ++t) {
+        const float r = gr_sigmoid(z[t * g.z_token] + rb);
+        const float in = gr_sigmoid(z[t * g.z_token + g.n] + ib);
+        float a, gain;
+        gr_decay(rate * r, a, gain);
+        S = fmaf(a, S, __fmul_rn(__fmul_rn(gain, in), to_float(reinterpret_cast<const T*>(g.u)[t * g.ldu + c])));
+        const float y = gr_gelu_tanh(to_float(reinterpret_cast<const T*>(g.y)[t * g.ldy + c]) + yb);
+        reinterpret_cast<T*>(g.out)[t * g.ldo + c] = from_float<T>(S * y);
+    }
+    *sp = S;
+}
+
 #define GR_SEGS 32
 #define GR_SEG_TOKENS 8
 
@@ -184,7 +211,7 @@ __global__ void __launch_bounds__(GR_EC * GR_SEGS) gated_recurrence_segments_ker
 }
 
 template <typename T>
-static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, int segments, cudaStream_t st) {
+static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, int form, cudaStream_t st) {
     if (num_seqs <= 0) return 0;
     if (g.width <= 0 || g.n <= 0 || g.width % g.n || g.u == nullptr || g.z == nullptr || g.y == nullptr ||
         g.state == nullptr || g.state_stride < g.width || g.num_slots <= 0 || g.r_bias == nullptr ||
@@ -192,16 +219,19 @@ static int launch_gated_recurrence(const GatedRecArgs& g, int num_seqs, int segm
         return SLB_ERR_BAD_ARG;
     const int gy = (g.width + GR_EC - 1) / GR_EC;
     if (gy > 65535) return SLB_ERR_TOO_LARGE;
-    if (segments)
+    if (form == 2)
+        return slb_launch(gated_recurrence_step_kernel<T>, dim3(num_seqs, (g.width + 127) / 128), dim3(128), 0, st, g);
+    if (form == 1)
         return slb_launch(gated_recurrence_segments_kernel<T>, dim3(num_seqs, gy), dim3(GR_EC * GR_SEGS), 0, st, g);
     return slb_launch(gated_recurrence_kernel<T>, dim3(num_seqs, gy), dim3(256), 0, st, g);
 }
 
 extern "C" {
-int slb_gated_recurrence_f32(const GatedRecArgs* g, int num_seqs, int segments, cudaStream_t st) {
-    return launch_gated_recurrence<float>(*g, num_seqs, segments, st);
+// form 0: token by token, 1: in segments, 2: single tokens
+int slb_gated_recurrence_f32(const GatedRecArgs* g, int num_seqs, int form, cudaStream_t st) {
+    return launch_gated_recurrence<float>(*g, num_seqs, form, st);
 }
-int slb_gated_recurrence_bf16(const GatedRecArgs* g, int num_seqs, int segments, cudaStream_t st) {
-    return launch_gated_recurrence<bf16>(*g, num_seqs, segments, st);
+int slb_gated_recurrence_bf16(const GatedRecArgs* g, int num_seqs, int form, cudaStream_t st) {
+    return launch_gated_recurrence<bf16>(*g, num_seqs, form, st);
 }
 }

@@ -120,10 +120,6 @@ int slb_gemm_simt_tanh_f32(const float* A, int lda, const float* W, int ldw, flo
                            const float* bias, int M, int N, int K, cudaStream_t st) {
     return launch_gemm<float, float, float, 1>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
 }
-int slb_gemm_simt_tanh_bf16(const bf16* A, int lda, const bf16* W, int ldw, float* C, int ldc,
-                            const float* bias, int M, int N, int K, cudaStream_t st) {
-    return launch_gemm<bf16, bf16, float, 1>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
-}
 int slb_gemm_simt_bf16_f32out(const bf16* A, int lda, const bf16* W, int ldw, float* C, int ldc,
                               const float* bias, int M, int N, int K, cudaStream_t st) {
     return launch_gemm<bf16, bf16, float>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);

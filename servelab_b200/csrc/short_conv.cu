@@ -96,16 +96,19 @@ __global__ void __launch_bounds__(256) qk_conv_cache_kernel(
     float* st = state != nullptr ? state + (size_t)state_slots[s] * state_stride + c : nullptr;
     float y[VEC];
 #pragma unroll
-    for (int v = 0; v < VEC; ++v) y[v] = out_bias != nullptr ? out_bias[c + v] : 0.f;
+    for (int v = 0; v < VEC; ++v) y[v] = 0.f;
+    if (out_bias != nullptr) load_vec<float, VEC>(out_bias + c, y);
+    float add[VEC];
+#pragma unroll
+    for (int v = 0; v < VEC; ++v) add[v] = 0.f;
+    if (in_bias != nullptr) load_vec<float, VEC>(in_bias + c, add);
     for (int i = 0; i < taps; ++i) {
         const int jj = j - hist + i;
         float u[VEC], w[VEC];
         if (jj >= 0) {
             load_vec<T, VEC>(proj + (size_t)(q0 + jj) * ldp + c, u);
-            if (in_bias != nullptr) {
 #pragma unroll
-                for (int v = 0; v < VEC; ++v) u[v] += in_bias[c + v];
-            }
+            for (int v = 0; v < VEC; ++v) u[v] += add[v];
         } else if (st != nullptr) {
             load_vec<float, VEC>(st + (size_t)(hist + jj) * C, u);
         } else {
@@ -152,10 +155,17 @@ __global__ void __launch_bounds__(256) conv_state_update_kernel(
     const int hist = taps - 1;
     float* st = state + (size_t)state_slots[s] * state_stride + c;
     const float add = in_bias != nullptr ? in_bias[c] : 0.f;
-    // ascending i: row i + n of the old record is read before any row >= i + 1 is written
-    for (int i = 0; i < hist; ++i) {
-        const int src = i + n - hist;              // index into the portion, or before it
-        st[(size_t)i * C] = src >= 0 ? to_float(proj[(size_t)(q0 + src) * ldp + c]) + add : st[(size_t)(i + n) * C];
+    // ascending i, four rows at a time: row i + n of the old record is read before it is written
+    for (int i0 = 0; i0 < hist; i0 += 4) {
+        float v[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int i = i0 + k, src = i + n - hist;      // index into the portion, or before it
+            v[k] = i >= hist ? 0.f : src >= 0 ? to_float(proj[(size_t)(q0 + src) * ldp + c]) + add : st[(size_t)(i + n) * C];
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+            if (i0 + k < hist) st[(size_t)(i0 + k) * C] = v[k];
     }
 }
 
@@ -181,7 +191,7 @@ static int launch_conv(const T* proj, int ldp, const float* taps_w, int taps, fl
     const bool vec = q_size % V == 0 && D % V == 0 && ldp % V == 0 && ldq % V == 0 && C % 4 == 0 &&
                      state_stride % 4 == 0 &&
                      (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)state |
-                       (uintptr_t)taps_w) & 15) == 0;
+                       (uintptr_t)taps_w | (uintptr_t)in_bias | (uintptr_t)out_bias) & 15) == 0;
     int rc;
     if (vec) {
         const int threads = C / V >= 256 ? 256 : 64;

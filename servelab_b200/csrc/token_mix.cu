@@ -13,7 +13,34 @@
 // alone.
 #include "common.cuh"
 
-template <typename T>
+// VEC (1 or 4) consecutive elements as floats, in one access
+template <typename T, int VEC>
+__device__ __forceinline__ void tm_load(const T* p, float (&v)[VEC]) {
+    if constexpr (VEC == 1) {
+        v[0] = to_float(p[0]);
+    } else if constexpr (sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+        v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+    } else {
+        const float4 u = *reinterpret_cast<const float4*>(p);
+        v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
+    }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void tm_store(T* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 1) {
+        p[0] = from_float<T>(v[0]);
+    } else if constexpr (sizeof(T) == 2) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+    } else {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+}
+
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) embed_bigram_kernel(
     const int* __restrict__ ids, const int* __restrict__ cu_q, const int* __restrict__ seq_of_token,
     const int* __restrict__ state_slots, int* __restrict__ state, long long state_stride, int num_slots,
@@ -42,10 +69,14 @@ __global__ void __launch_bounds__(256) embed_bigram_kernel(
     if (pr < 0) pr += buckets;
     const T* row = table + (size_t)(ok ? id : 0) * h;
     const T* prow = pairs + (size_t)pr * h;
-    for (int c = threadIdx.x; c < h; c += blockDim.x) {
-        const float x = ok ? to_float(row[c]) + to_float(prow[c]) : 0.f;
-        out[(size_t)t * h + c] = x;
-        if (copy != nullptr) copy[(size_t)t * ldc + c] = from_float<T>(x);
+    for (int c = threadIdx.x * VEC; c < h; c += blockDim.x * VEC) {
+        float x[VEC], y[VEC];
+        tm_load<T, VEC>(row + c, x);
+        tm_load<T, VEC>(prow + c, y);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[i] = ok ? x[i] + y[i] : 0.f;
+        tm_store<float, VEC>(out + (size_t)t * h + c, x);
+        if (copy != nullptr) tm_store<T, VEC>(copy + (size_t)t * ldc + c, x);
     }
 }
 
@@ -88,13 +119,7 @@ __global__ void __launch_bounds__(256) token_mix_kernel(
         float y[VEC];
 #pragma unroll
         for (int i = 0; i < VEC; ++i) y[i] = h[i] + (hp[i] - h[i]) * mv[i];
-        if constexpr (VEC == 4 && sizeof(T) == 2) {
-            __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
-            *reinterpret_cast<uint2*>(o) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
-        } else {
-#pragma unroll
-            for (int i = 0; i < VEC; ++i) o[i] = from_float<T>(y[i]);
-        }
+        tm_store<T, VEC>(o, y);
     }
 }
 
@@ -107,7 +132,10 @@ static int launch_embed_bigram(const int* ids, const int* cu_q, const int* seq_o
     if (h <= 0 || vocab <= 0 || buckets <= 0 || state == nullptr || state_stride < 1 || num_slots <= 0 ||
         pairs == nullptr || (copy != nullptr && ldc < h))
         return SLB_ERR_BAD_ARG;
-    return slb_launch(embed_bigram_kernel<T>, dim3(T_), dim3(h >= 1024 ? 256 : 128), 0, st, ids, cu_q, seq_of_token,
+    const bool vec = h % 4 == 0 && ldc % 4 == 0 &&
+                     (((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out | (uintptr_t)copy) & 15) == 0;
+    return slb_launch(vec ? embed_bigram_kernel<T, 4> : embed_bigram_kernel<T, 1>, dim3(T_), dim3(h >= 1024 ? 256 : 128),
+                      0, st, ids, cu_q, seq_of_token,
                       state_slots, state, state_stride, num_slots, table, vocab, pairs, buckets, mul_prev, mul_cur,
                       out, copy, ldc, h);
 }

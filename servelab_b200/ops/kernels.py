@@ -1576,7 +1576,7 @@ def token_mix(ctx, x: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, out: t
 
 def tanh_linear(low: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor) -> None:
     """out = tanh(low) . w^T (+ bias), float32 results: the second product of a bottleneck."""
-    fn = getattr(L.core(), "slb_gemm_simt_tanh_" + _suffix(low.dtype))
+    fn = L.core().slb_gemm_simt_tanh_f32 if low.dtype == _F32 else L.core().slb_tanh_linear_bf16
     L.check(fn(low.data_ptr(), low.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _p(bias),
                low.shape[0], w.shape[0], w.shape[1], _stream()), "tanh_linear")
 
@@ -1683,5 +1683,5 @@ def gated_recurrence(ctx, u: torch.Tensor, z: torch.Tensor, y: torch.Tensor, sta
     g.width, g.n = out.shape[1], z.shape[2] // 2
     g.out, g.ldo = out.data_ptr(), out.stride(0)
     fn = getattr(L.core(), "slb_gated_recurrence_" + _suffix(out.dtype))
-    segments = not ctx.decode_only and (force_gated_recurrence_segments or out.dtype == _BF16)
-    L.check(fn(_ct.byref(g), ctx.num_seqs, int(segments), _stream()), "gated_recurrence")
+    form = 2 if ctx.decode_only else int(force_gated_recurrence_segments or out.dtype == _BF16)
+    L.check(fn(_ct.byref(g), ctx.num_seqs, form, _stream()), "gated_recurrence")

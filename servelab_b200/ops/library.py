@@ -75,7 +75,7 @@ _CORE_SIGNATURES = {
     "slb_gemm_simt_batched_bf16": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
     "slb_gemm_simt_batched_bf16_f32out": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
     "slb_gemm_simt_tanh_f32": [P, I, P, I, P, I, P, I, I, I, P],
-    "slb_gemm_simt_tanh_bf16": [P, I, P, I, P, I, P, I, I, I, P],
+    "slb_tanh_linear_bf16": [P, I, P, I, P, I, P, I, I, I, P],
     "slb_dyt_parallel_f32": [P, P],
     "slb_dyt_parallel_bf16": [P, P],
     "slb_stream_rows_f32": [P, P],

@@ -206,10 +206,11 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
 def batched_head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     """out[:, b, :] = a[:, b, :] . w[b]^T per head b: a [M, B, K], w [B, N, K], out [M, B, N]
     (views; last dimension contiguous).  float32: this package's CUDA-core kernel (true 32-bit,
-    k-sequential sums); bfloat16: the vendor's batched product."""
+    k-sequential sums); bfloat16: the vendor's batched product (rows that are no whole 16-byte pieces:
+    the CUDA-core kernel)."""
     if a.shape[0] == 0:
         return
-    if a.dtype == torch.float32 or not use_vendor_batched:
+    if a.dtype == torch.float32 or not use_vendor_batched or a.shape[2] % 8 or w.shape[1] % 8:
         K.gemm_simt_batched(a, w, out)
         return
     torch.bmm(a.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))

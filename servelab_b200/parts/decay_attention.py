@@ -30,7 +30,7 @@ import torch
 
 from ..cache.manager import FixedStateRequest
 from ..ops import kernels as K
-from ..ops.linear import linear
+from ..ops.linear import batched_head_linear, linear
 from ..weights.source import BIAS, MATRIX, NORM, TensorDecl
 from .base import Mixer
 from .normed_attention import pad_rows
@@ -122,7 +122,10 @@ class DecayAttention(Mixer):
         s = self.spec
         names = [n["q"], n["k"], n["v"], n["gate"]] + ([n["decay_down"]] if self.gated else [])
         if s.token_mix:
-            self.w_parts = [store.get(name) for name in names]
+            parts = [store.get(name) for name in names]
+            # r, k, v and the gate as one batch where they have one size
+            self.w_four = torch.stack(parts[:4]) if self.q_size == self.v_size else None
+            self.w_parts = parts if self.w_four is None else [None] * 4 + parts[4:]
             self.mu = torch.stack([store.get(f"{self.prefix}.{name}") for name in s.token_mix_names]).contiguous()
         else:
             self.w_in = pad_rows(store.cat(names))
@@ -145,10 +148,13 @@ class DecayAttention(Mixer):
         mixed = torch.empty((len(s.token_mix_names), T, s.hidden_size), dtype=x.dtype, device=x.device)
         K.token_mix(ctx, x, self.mu, prev, mixed)
         proj = torch.empty((T, 2 * self.q_size + 2 * self.v_size), dtype=x.dtype, device=x.device)
-        at = 0
-        for i, w in enumerate(self.w_parts[:4]):
-            proj[:, at:at + w.shape[0]] = K.plain_unless(None, linear(mixed[i], w))
-            at += w.shape[0]
+        if self.w_four is not None:
+            batched_head_linear(mixed[:4].transpose(0, 1), self.w_four, proj.view(T, 4, self.q_size))
+        else:
+            at = 0
+            for i, w in enumerate(self.w_parts[:4]):
+                proj[:, at:at + w.shape[0]] = K.plain_unless(None, linear(mixed[i], w))
+                at += w.shape[0]
         low = K.plain_unless(None, linear(mixed[4], self.w_parts[4]))
         return proj, low, state
 
