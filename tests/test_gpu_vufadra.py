@@ -550,6 +550,27 @@ def test_gated_recurrence_with_its_convolution(dtype, shape, segments, monkeypat
     assert torch.equal(state[[0, 2]], keep[[0, 2]]) and not torch.equal(state[1], keep[1])
 
 
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("shape", [(1, 64, 8, 0), (9, 40, 24, 0), (70, 130, 64, 8), (65, 33, 13, 3), (600, 200, 72, 16),
+                                   (520, 131, 7, 1)])
+def test_second_product_of_a_bottleneck(dtype, shape):
+    """tanh kept to more than the operands' 8 bits; columns of a larger projection; sizes of no tile."""
+    from servelab_b200.ops import kernels as K
+    M, N, R, off = shape
+    g = torch.Generator().manual_seed(M)
+    proj = torch.randn(M, R + 2 * off + 8, generator=g).to(dtype)
+    w, bias = torch.randn(N, R, generator=g).to(dtype), torch.randn(N, generator=g)
+    want = torch.tanh(proj[:, off:off + R].double()) @ w.double().t() + bias.double()
+    pd, wd, bd = proj.to(DEV), w.to(DEV), bias.to(DEV)
+    big = torch.full((M, N + 3), 7.0, device=DEV)
+    K.tanh_linear(pd[:, off:off + R], wd, bd, big[:, :N])
+    _close(big[:, :N], want, 2e-5)
+    assert float(big[:, N:].min()) == 7.0
+    out = torch.empty(M, N, device=DEV)
+    K.tanh_linear(pd[:, off:off + R], wd, None, out)
+    _close(out, want - bias.double(), 2e-5)
+
+
 # ------------------------------------------------------------ whole models
 LENGTHS = [70, 45, 190, 33, 2, 1, 58]
 TOL = {"float32": 1e-4, "bfloat16": 4e-2}       # of the largest logit
