@@ -512,7 +512,7 @@ def _measure(cfg: dict, note, graph_prefill: bool = False, queue_ahead: bool = F
     never waits for the host between two events."""
     import torch
     from ..ops import kernels as K
-    from ..ops.profile import StepProfile
+    from ..ops.profile import StepProfile, mark
     from . import workloads as W
     pages = 64 * (-(-(CONTEXT + 64) // PAGE)) + PROMPT // PAGE + 8
     engine = W.make_engine(cfg, pages, 64, PROMPT, 4096, weights_seed=3, page_size=PAGE)
@@ -549,11 +549,18 @@ def _measure(cfg: dict, note, graph_prefill: bool = False, queue_ahead: bool = F
     ms = out.get("prefill_graph_ms", ms) if out.get("prefill_graph_replays") else ms
     out["prefill_ms"] = round(ms, 3)
     out["prefill_tok_s"] = round(PROMPT / (ms * 1e-3), 1)
-    hold = (lambda: torch.cuda._sleep(20_000_000)) if queue_ahead else (lambda: None)
+
+    def hold():
+        if queue_ahead:
+            torch.cuda._sleep(20_000_000)
+            mark("(hold)")
+
+    def kernels_us(prof, steps):
+        return {name: us for name, us in prof.summary(steps).items() if name != "(hold)"}
     with StepProfile() as prof:
         hold()
         runner.step([entry])
-    out["prefill_kernels_us"] = prof.summary(1)
+    out["prefill_kernels_us"] = kernels_us(prof, 1)
     runner.cuda_graphs = saved
     runner.cache.release("p")
 
@@ -575,7 +582,7 @@ def _measure(cfg: dict, note, graph_prefill: bool = False, queue_ahead: bool = F
             for _ in range(5):
                 hold()
                 runner.step(entries)
-        out[f"decode_b{batch}_kernels_us"] = prof.summary(5)
+        out[f"decode_b{batch}_kernels_us"] = kernels_us(prof, 5)
         runner.cuda_graphs = saved
         for rid in rids:
             runner.cache.release(rid)
