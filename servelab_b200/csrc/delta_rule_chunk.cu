@@ -198,9 +198,10 @@ for (int d = lane; d < Dp; d += 32) {        // (a warp has the four rows from 4
     }
 }
 
-// acc += A B over `steps` contraction steps of 8, the cross terms of the split in chains of their own (low).  A's fragment starts at A (+ row8 for the row 8 below,
-// + k4 for the contraction 4 further, + k8 a step); B is [column][contraction] with stride ldb, B already
-// at this lane's column and contraction, NT tiles of 8 columns; EXACT: B's elements are TF32 numbers.
+// acc += A B over `steps` contraction steps of 8, the cross terms of the split in chains of their own
+// (low).  A's fragment starts at A (+ row8 for the row 8 below, + k4 for the contraction 4 further, + k8 a
+// step); B is [column][contraction] with stride ldb, B already at this lane's column and contraction, NT
+// tiles of 8 columns; EXACT: B's elements are TF32 numbers.
 template <int NT, bool EXACT>
 __device__ __forceinline__ void dc_product(float (&acc)[NT][4], float (&low)[2][NT][4], const float* A, int row8,
                                            int k4, int k8, const float* B, int ldb, int steps) {
@@ -315,7 +316,8 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
         // rows 0..31: X S + Y V = seen; rows 32..63: R S + P V, the outputs without what was removed
         float acc[1][4] = {}, low[2][1][4] = {};
         dc_product<1, false>(acc, low, b + (m0 + g) * LX + t, 8 * LX, 4, 8, Ss + (n0 + g) * LX + t, LX, Dp / 8);
-        dc_product<1, EXACT>(acc, low, Ym + (m0 + g) * DC_LM + t, 8 * DC_LM, 4, 8, Vt + (n0 + g) * DC_LM + t, DC_LM, DC_C / 8);
+        dc_product<1, EXACT>(acc, low, Ym + (m0 + g) * DC_LM + t, 8 * DC_LM, 4, 8, Vt + (n0 + g) * DC_LM + t, DC_LM,
+                             DC_C / 8);
         if (m0 < DC_C) {
 #pragma unroll
             for (int i = 0; i < 4; ++i)
@@ -323,15 +325,16 @@ __global__ void __launch_bounds__(256) delta_chunk_scan_kernel(const DeltaChunkA
         }
         __syncthreads();
         if (m0 >= DC_C) {
-            dc_product<1, false>(acc, low, Qm + (m0 - DC_C + g) * DC_LM + t, 8 * DC_LM, 4, 8, Nt + (n0 + g) * DC_LM + t, DC_LM,
-                          DC_C / 8);
+            dc_product<1, false>(acc, low, Qm + (m0 - DC_C + g) * DC_LM + t, 8 * DC_LM, 4, 8, Nt + (n0 + g) * DC_LM + t,
+                                 DC_LM, DC_C / 8);
             const int e = e0 + n0 + 2 * t;
 #pragma unroll
             for (int i = 0; i < 4; i += 2) {
                 const int tt = k * DC_C + m0 - DC_C + g + i * 4;
                 if (tt >= qlen || e >= Dv) continue;
                 float* o = a.out + (size_t)(q0 + tt) * a.ldo + h * Dv + e;
-                const float x = acc[0][i] + (low[0][0][i] + low[1][0][i]), y = acc[0][i + 1] + (low[0][0][i + 1] + low[1][0][i + 1]);
+                const float x = acc[0][i] + (low[0][0][i] + low[1][0][i]);
+                const float y = acc[0][i + 1] + (low[0][0][i + 1] + low[1][0][i + 1]);
                 if ((Dv & 1) == 0 && (a.ldo & 1) == 0) {
                     *reinterpret_cast<float2*>(o) = make_float2(x, y);
                 } else {
