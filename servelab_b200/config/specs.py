@@ -86,6 +86,7 @@ class RMSNormSpec(PartSpec):
     eps: float = 1e-6
     weight_suffix: str = ".weight"         # the weight is <prefix><weight_suffix>
     unit_offset: bool = False              # the stored weight lies around zero: the factor is 1 + w
+    factor: float = 1.0                    # a constant on the result
 
 
 @dataclass(frozen=True)
@@ -211,7 +212,13 @@ class NormedAttentionSpec(PartSpec):
                      j // chunk == i // chunk (not together with a window);
     ``weight_fn``    "softmax", or "sigmoid": the weight of a visible key is sigmoid(score) and
                      the weights are not normalized (no soft cap, sink or gate with it);
-    ``score_bias``   (sigmoid) a learned number a head added to the scaled score.
+    ``score_bias``   (sigmoid) a learned number a head added to the scaled score;
+    ``qk_row_norm``  RMS norm over all query heads of a token together, and over all its key heads, with
+                     weights of the whole rows (not together with ``qk_norm``);
+    ``qkv_bias``, ``out_bias``  biases of the projections, <projection><bias_suffix>;
+    ``distance_slopes``  numbers a head: slope_h (i - j) is taken off the (capped) score of query i, key j;
+    ``sink_score``   a constant in place of the learned numbers of ``sink``: exp(sink_score) joins every
+                     head's denominator.
     """
     kind: str = "normed_attention"
     hidden_size: int = 0
@@ -245,6 +252,12 @@ class NormedAttentionSpec(PartSpec):
     weight_fn: str = "softmax"
     score_bias: bool = False
     score_bias_name: str = "pb"
+    qk_row_norm: bool = False
+    qkv_bias: bool = False
+    out_bias: bool = False
+    bias_suffix: str = ".b"
+    distance_slopes: Tuple[float, ...] = ()
+    sink_score: Optional[float] = None
 
 
 @dataclass(frozen=True)
@@ -412,6 +425,37 @@ class GatedRecurrenceSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class StateSpaceSpec(PartSpec):
+    """A selective state space (Mamba-2): one projection gives z | x | B | C | dt (``num_heads`` x
+    ``value_dim`` for z and x, ``groups`` x ``state_dim`` for B and C, ``num_heads`` for dt); x, B and C pass
+    a causal convolution per channel (``conv_taps``, bias) and SiLU; with d = softplus(dt + dt_bias), head h
+    and its group h // (``num_heads`` / ``groups``),
+
+        S_t = exp(-exp(A_log_h) d) S_{t-1} + d B_t x_t^T,    y_t = S_t^T C_t + D_h x_t,
+
+    S of ``state_dim`` x ``value_dim`` float32 a head, S = 0 before a sequence's first token.  The row y is
+    multiplied by silu(z), RMS-normed in ``norm_groups`` equal parts (``norm_eps``), multiplied by a weight
+    and projected.  Per-request state: S and the convolution's last ``conv_taps`` - 1 inputs."""
+    kind: str = "state_space"
+    hidden_size: int = 0
+    num_heads: int = 0
+    value_dim: int = 0
+    state_dim: int = 0
+    groups: int = 1
+    conv_taps: int = 1
+    norm_groups: int = 1
+    norm_eps: float = 1e-6
+    in_name: str = "in"
+    conv_name: str = "conv"
+    conv_bias_name: str = "conv.b"
+    dt_bias_name: str = "dt_bias"
+    decay_name: str = "A_log"
+    skip_name: str = "D"
+    norm_name: str = "norm"
+    o_name: str = "o"
+
+
+@dataclass(frozen=True)
 class DifferentialAttentionSpec(PartSpec):
     """Grouped-query softmax attention with two maps a head: every query head and every kv head
     carries two query / key vectors of ``head_dim`` elements ([head][map]), each map attends on
@@ -446,7 +490,9 @@ class ParallelMixersSpec(PartSpec):
     """Two mixers side by side that read the same input; each one's result is RMS-normed over the
     model width with a weight of its own (``eps``) and the mixer returns ``factor`` times their
     sum.  The branches' tensors live under ``<prefix>.<left_name>`` and ``<prefix>.<right_name>``,
-    the norm weights under ``<prefix>.<left_name><out_suffix>`` and the same for the right."""
+    the norm weights under ``<prefix>.<left_name><out_suffix>`` and the same for the right.
+    ``branch_norms`` False: no norms, the mixer returns ``left_factor`` times the left result plus
+    ``right_factor`` times the right (branches that split off their projections, see ``parts/base.py``)."""
     kind: str = "parallel_mixers"
     hidden_size: int = 0
     left: PartSpec = None
@@ -456,6 +502,9 @@ class ParallelMixersSpec(PartSpec):
     left_name: str = "left"
     right_name: str = "right"
     out_suffix: str = ".out"
+    branch_norms: bool = True
+    left_factor: float = 1.0
+    right_factor: float = 1.0
 
 
 # -------------------------------------------------------------- feed-forward
@@ -488,7 +537,9 @@ class RoutedExpertsSpec(PartSpec):
     ``score_fn`` "sigmoid": the scores are sigmoids of the logits.  ``correction_name``: a learned
     offset per expert that is added to the scores for the choice (experts and groups) and not for
     the weights.  ``group_best``: a group scores as the sum of its that many largest choice scores
-    (1: its best).  ``norm_eps``: added to the sum of the chosen scores with ``renormalize``."""
+    (1: its best).  ``norm_eps``: added to the sum of the chosen scores with ``renormalize``.
+    ``activation``, ``limit``, ``swish_alpha``: the experts' gated activation, as ``GatedMLPSpec`` has it.
+    ``weight_inputs``: a weight multiplies the expert's input instead of its output."""
     kind: str = "routed_experts"
     hidden_size: int = 0
     num_experts: int = 0
@@ -510,6 +561,10 @@ class RoutedExpertsSpec(PartSpec):
     down_name: str = "down"
     shared_name: str = "shared"
     weight_suffix: str = ""
+    activation: str = "silu"
+    limit: Optional[float] = None
+    swish_alpha: float = 1.702
+    weight_inputs: bool = False
 
 
 # --------------------------------------------------------------------- block

@@ -15,6 +15,9 @@
 // and a sink, one number a head whose exponential is added to the softmax's denominator once (it
 // has no key and no value and is neither scaled nor capped).
 //
+// A distance bias (`slopes`, one number a head): slope_h (i - j) is taken off the (capped) score of query
+// position i and key position j.  `out_scale`: a factor on the results.
+//
 // Instead of the softmax (`sig_bias`, one number a head): the weight of a visible key is
 // sigmoid(s + sig_bias_h) and the weights are not normalized.  Instead of the window (`chunk` > 0): a query
 // at position i sees the keys j <= i with j / chunk == i / chunk.
@@ -50,7 +53,7 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
     const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
     int H, int Hkv, int Dk, int Dv, int ps, int num_pages, float scale, int window,
     const T* __restrict__ gate, int ldg, float softcap, const float* __restrict__ sink, int chunk,
-    const float* __restrict__ sig_bias) {
+    const float* __restrict__ sig_bias, const float* __restrict__ slopes, float out_scale) {
     extern __shared__ float ak_smem[];
     pdl_wait();
     const int ldq_s = Dk + 1;
@@ -93,6 +96,7 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
     // the first key of this thread's row, and what its head adds to a score
     const int my_first = window > 0 ? my_pos - window + 1 : chunk > 0 && my_pos >= 0 ? my_pos - my_pos % chunk : 0;
     const float my_bias = sig_bias != nullptr && row_valid ? sig_bias[kvh * g + (row0 + r) % g] : 0.f;
+    const float my_slope = slopes != nullptr && row_valid ? slopes[kvh * g + (row0 + r) % g] : 0.f;
     const int kend = p_last + 1;
     const int nvc = (Dv + AK_DC - 1) / AK_DC;
 
@@ -146,6 +150,7 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
             const bool vis = row_valid && kp <= my_pos && kp >= my_first;
             float sv = sc[j] * scale;
             if (softcap > 0.f) sv = softcap * tanhf(sv / softcap);
+            sv = fmaf(my_slope, (float)(kp - my_pos), sv);
             sc[j] = vis ? sv : -INFINITY;
             tmax = fmaxf(tmax, sc[j]);
         }
@@ -209,6 +214,7 @@ __global__ void __launch_bounds__(AK_THREADS) attention_kv_kernel(
         if (sink != nullptr) l += (m == -INFINITY) ? 1.f : expf(sink[head] - m);
         float inv = l > 0.f ? 1.0f / l : 0.f;
         if (sig_bias != nullptr) inv = 1.0f;
+        inv *= out_scale;
         if (gate != nullptr) {
             const float z = to_float(gate[(size_t)(q0 + tl) * ldg + head]);
             inv *= 1.0f / (1.0f + expf(-z));
@@ -230,11 +236,12 @@ static int launch_attention_kv(const T* q, int ldq, const T* kc, int ldk, int ma
                                const int* ctx_len, const int* tile_seq, const int* tile_row0,
                                int num_tiles, int H, int Hkv, int Dk, int Dv, int ps, int num_pages,
                                float scale, int window, const T* gate, int ldg, float softcap,
-                               const float* sink, cudaStream_t st, int chunk = 0, const float* sig_bias = nullptr) {
+                               const float* sink, cudaStream_t st, int chunk = 0, const float* sig_bias = nullptr,
+                               const float* slopes = nullptr, float out_scale = 1.f) {
     if (num_tiles <= 0) return 0;
     if (chunk < 0 || (chunk > 0 && window > 0) || (sig_bias != nullptr && (sink != nullptr || maps != 1)))
         return SLB_ERR_BAD_ARG;
-    if (softcap < 0.f || (sink != nullptr && maps != 1)) return SLB_ERR_BAD_ARG;
+    if (softcap < 0.f || ((sink != nullptr || slopes != nullptr) && maps != 1)) return SLB_ERR_BAD_ARG;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dv <= 0 || ps <= 0 || max_pages <= 0 ||
         num_pages <= 0 || ldv < Dv || maps <= 0 || ldk < maps * Dk)
         return SLB_ERR_BAD_ARG;
@@ -247,7 +254,8 @@ static int launch_attention_kv(const T* q, int ldq, const T* kc, int ldk, int ma
     if (rc != 0) return rc;
     return slb_launch(attention_kv_kernel<T, TO>, dim3(num_tiles, Hkv * maps), dim3(AK_THREADS), smem, st, q, ldq,
                       kc, ldk, maps, vc, ldv, out, ldo, block_table, max_pages, cu_q, ctx_len, tile_seq, tile_row0,
-                      H, Hkv, Dk, Dv, ps, num_pages, scale, window, gate, ldg, softcap, sink, chunk, sig_bias);
+                      H, Hkv, Dk, Dv, ps, num_pages, scale, window, gate, ldg, softcap, sink, chunk, sig_bias, slopes,
+                      out_scale);
 }
 
 extern "C" {
@@ -257,20 +265,22 @@ int slb_attention_kv_f32(const float* q, int ldq, const float* kc, const float* 
                          const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                          int H, int Hkv, int Dk, int Dv, int ps, int num_pages, float scale, int window,
                          const float* gate, int ldg, float softcap, const float* sink, int chunk,
-                         const float* sig_bias, cudaStream_t st) {
+                         const float* sig_bias, const float* slopes, float out_scale, cudaStream_t st) {
     return launch_attention_kv<float, float>(q, ldq, kc, Dk, 1, vc, ldv, out, ldo, block_table, max_pages, cu_q,
                                       ctx_len, tile_seq, tile_row0, num_tiles, H, Hkv, Dk, Dv, ps,
-                                      num_pages, scale, window, gate, ldg, softcap, sink, st, chunk, sig_bias);
+                                      num_pages, scale, window, gate, ldg, softcap, sink, st, chunk, sig_bias, slopes,
+                                      out_scale);
 }
 int slb_attention_kv_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int ldv, bf16* out,
                           int ldo, const int* block_table, int max_pages, const int* cu_q,
                           const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                           int H, int Hkv, int Dk, int Dv, int ps, int num_pages, float scale, int window,
                          const bf16* gate, int ldg, float softcap, const float* sink, int chunk,
-                         const float* sig_bias, cudaStream_t st) {
+                         const float* sig_bias, const float* slopes, float out_scale, cudaStream_t st) {
     return launch_attention_kv<bf16, bf16>(q, ldq, kc, Dk, 1, vc, ldv, out, ldo, block_table, max_pages, cu_q,
                                      ctx_len, tile_seq, tile_row0, num_tiles, H, Hkv, Dk, Dv, ps,
-                                     num_pages, scale, window, gate, ldg, softcap, sink, st, chunk, sig_bias);
+                                     num_pages, scale, window, gate, ldg, softcap, sink, st, chunk, sig_bias, slopes,
+                                      out_scale);
 }
 // several maps a head (see the top of the file); the results are float32 in both forms
 int slb_attention_kv_maps_f32(const float* q, int ldq, const float* kc, int ldk, int maps, const float* vc, int ldv,

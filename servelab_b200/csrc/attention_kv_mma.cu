@@ -27,6 +27,9 @@
 // sig_bias_h), the weights are not normalized, and key splits simply add up.  Instead of the window
 // (`chunk` > 0): a query at position i sees the keys j <= i with j / chunk == i / chunk.
 //
+// A distance bias (`slopes`, one number a head): slope_h (i - j) is taken off the (capped) score of query
+// position i and key position j.  `out_scale`: a factor on the results.
+//
 // Several attention maps a head (`maps`; not with `tied`): every query head and every kv head
 // carries `maps` query / key vectors side by side ([head][map][DK]; a cached key row is
 // [map][DK]), each map is an attention of its own over the kv head's one set of values, and a
@@ -101,7 +104,8 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
     const int* __restrict__ tile_row0, int H, int Hkv, int ps, int num_pages, float scale_log2,
     int window, const bf16* __restrict__ gate, int ldg, int splits, float* __restrict__ part_o,
     float* __restrict__ part_ml, int maps, float* __restrict__ out_f32, int q_rows, int fold,
-    float softcap, float scale, const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias) {
+    float softcap, float scale, const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias,
+    const float* __restrict__ slopes, float out_scale) {
     // softcap > 0: a scaled score s becomes softcap tanh(s / softcap); sink: one number a head whose
     // exponential joins the softmax's denominator (added where the row is finished: here without
     // key splits, in the combine kernel with them)
@@ -181,6 +185,13 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
         if (r_hi < nrows) bias2[1] = sig_bias[kvh * g + (row0 + r_hi) % g] * 1.4426950408889634f;
     }
 
+    // (what follows multiplies by scale * log2 e: the slopes divided by scale)
+    float slope[2] = {0.f, 0.f};
+    if (slopes != nullptr) {
+        if (r_lo < nrows) slope[0] = slopes[kvh * g + (row0 + r_lo) % g] / scale;
+        if (r_hi < nrows) slope[1] = slopes[kvh * g + (row0 + r_hi) % g] / scale;
+    }
+
     float o[NO][4];
 #pragma unroll
     for (int n = 0; n < NO; ++n)
@@ -250,6 +261,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
                 for (int e = 0; e < 4; ++e) {
                     const int kp = k0 + j * 8 + tig * 2 + (e & 1);
                     const int pos = (e < 2) ? pos_lo : pos_hi;
+                    if (slopes != nullptr) sc[j][e] = fmaf(slope[e >> 1], (float)(kp - pos), sc[j][e]);
                     const bool vis = kp < kend && kp <= pos && kp >= ((e < 2) ? first_lo : first_hi);
                     if (!vis) sc[j][e] = -INFINITY;
                     mx[e >> 1] = fmaxf(mx[e >> 1], sc[j][e]);
@@ -361,6 +373,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
             l[h] += (m[h] == -INFINITY) ? 1.f : exp2f(sink[head] * 1.4426950408889634f - m[h]);
         float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
         if (sig_bias != nullptr) inv = 1.f;
+        inv *= out_scale;
         if (gate != nullptr) {
             const float z = __bfloat162float(gate[(size_t)(q0 + tl) * ldg + head]);
             inv *= 1.0f / (1.0f + __expf(-z));
@@ -389,7 +402,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
 __global__ void __launch_bounds__(128) attention_kv_combine_kernel(
     const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits, bf16* __restrict__ out,
     int ldo, int H, const bf16* __restrict__ gate, int ldg, float* __restrict__ out_f32,
-    const float* __restrict__ sink, int plain_sum) {
+    const float* __restrict__ sink, int plain_sum, float out_scale) {
     __shared__ float wgt[32];
     __shared__ float inv_s;
     pdl_wait();
@@ -409,6 +422,7 @@ __global__ void __launch_bounds__(128) attention_kv_combine_kernel(
             if (sink != nullptr) L += (M == -INFINITY) ? 1.f : exp2f(sink[head] * 1.4426950408889634f - M);
             float inv = L > 0.f ? 1.f / L : 0.f;
             if (plain_sum) inv = 1.f;                      // (weights that are not normalized)
+            inv *= out_scale;
             if (gate != nullptr) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[t * ldg + head])));
             inv_s = inv;
         }
@@ -467,7 +481,8 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
                                    int H, int Hkv, int maps, int ps, int num_pages, float scale, int window,
                                    const bf16* gate, int ldg, int splits, float* part_o, float* part_ml,
                                    int narrow, int fold, cudaStream_t st, float softcap = 0.f,
-                                   const float* sink = nullptr, int chunk = 0, const float* sig_bias = nullptr) {
+                                   const float* sink = nullptr, int chunk = 0, const float* sig_bias = nullptr,
+                                   const float* slopes = nullptr, float out_scale = 1.f) {
     // `fold` > 1: H counts (head, map) pairs, `maps` is 1, DK is fold times a map's key size.
     // `narrow`: every tile of the list holds at most 16 rows (a step of single tokens with at most
     // 16 query heads a kv head).
@@ -477,7 +492,7 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
     if (splits < 1 || splits > 32 || (splits > 1 && (part_o == nullptr || part_ml == nullptr || H / Hkv > BM)))
         return SLB_ERR_BAD_ARG;
     if (narrow && H / Hkv > 16) return SLB_ERR_BAD_ARG;
-    if (softcap < 0.f || (sink != nullptr && (maps != 1 || fold != 1))) return SLB_ERR_BAD_ARG;
+    if (softcap < 0.f || ((sink != nullptr || slopes != nullptr) && (maps != 1 || fold != 1))) return SLB_ERR_BAD_ARG;
     if (chunk < 0 || (chunk > 0 && window > 0) || (sig_bias != nullptr && (maps != 1 || fold != 1 || sink != nullptr)))
         return SLB_ERR_BAD_ARG;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || ps <= 0 || max_pages <= 0 || num_pages <= 0 || scale <= 0.f ||
@@ -498,12 +513,13 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
                              dim3(num_tiles * Hkv * maps, splits), dim3(NTHREADS), smem, st,
                              q, ldq, kc, tied ? kc : vc, tied, out, ldo, block_table, max_pages, cu_q, ctx_len,
                              tile_seq, tile_row0, H, Hkv, ps, num_pages, scale * 1.4426950408889634f, window,
-                             gate, ldg, splits, part_o, part_ml, maps, out_f32, q_rows, fold, softcap, scale, sink, chunk, sig_bias);
+                             gate, ldg, splits, part_o, part_ml, maps, out_f32, q_rows, fold, softcap, scale, sink, chunk,
+                             sig_bias, slopes, out_scale);
     if (e != 0 || splits == 1) return e;
     // (one tile a token: num_tiles is the number of tokens)
     return slb_launch(attention_kv_combine_kernel, dim3(num_tiles, H * maps), dim3(128), 0, st, (const float*)part_o,
                       (const float*)part_ml, splits, out, ldo, H * maps, gate, ldg, out_f32, sink,
-                      sig_bias != nullptr ? 1 : 0);
+                      sig_bias != nullptr ? 1 : 0, out_scale);
 }
 // `tied`: the values are the first DV elements of the key rows (vc is ignored).
 int slb_attention_kv_mma_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int tied, bf16* out,
@@ -518,17 +534,19 @@ int slb_attention_kv_mma_bf16(const bf16* q, int ldq, const bf16* kc, const bf16
 }
 // The same with a soft cap on the scaled scores (`softcap` > 0: s <- softcap tanh(s / softcap)) and a
 // sink a head (`sink` [H] float32 or null) in the softmax's denominator; with `chunk` > 0 instead of the
-// window and `sig_bias` ([H] float32 or null) instead of the softmax.
+// window and `sig_bias` ([H] float32 or null) instead of the softmax; with slopes of a distance bias
+// (`slopes` [H] float32 or null) and a factor on the results.
 int slb_attention_kv_mma_capped_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int tied, bf16* out,
                                      int ldo, const int* block_table, int max_pages, const int* cu_q,
                                      const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                                      int H, int Hkv, int ps, int num_pages, float scale, int window,
                                      const bf16* gate, int ldg, int splits, float* part_o, float* part_ml,
                                      int narrow, float softcap, const float* sink, int chunk,
-                                     const float* sig_bias, cudaStream_t st) {
+                                     const float* sig_bias, const float* slopes, float out_scale, cudaStream_t st) {
     return launch_attention_kv_mma(q, ldq, kc, vc, tied, out, nullptr, ldo, block_table, max_pages, cu_q, ctx_len,
                                    tile_seq, tile_row0, num_tiles, H, Hkv, 1, ps, num_pages, scale, window, gate,
-                                   ldg, splits, part_o, part_ml, narrow, 1, st, softcap, sink, chunk, sig_bias);
+                                   ldg, splits, part_o, part_ml, narrow, 1, st, softcap, sink, chunk, sig_bias,
+                                   slopes, out_scale);
 }
 // `maps` attention maps a head; float32 results [token][head][map][DV] with rows `ldo` floats apart
 int slb_attention_kv_mma_maps_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int maps, float* out,

@@ -11,7 +11,9 @@
 //   * optional epilogue: head h's row times sigmoid(gate[token][h]);
 //   * `sig_bias` (one number a head) instead of the softmax: a visible key's weight is
 //     sigmoid(score + sig_bias_h), not normalized, so the accumulator is never rescaled; `chunk` > 0
-//     instead of the window: a query at position i sees the keys j <= i with j / chunk == i / chunk.
+//     instead of the window: a query at position i sees the keys j <= i with j / chunk == i / chunk;
+//   * `slopes` (one number a head): slope_h (i - j) is taken off the (capped) score of query position i and
+//     key position j; `out_scale`: a factor on the results.
 //
 // Work unit: 128 query rows x one kv head (rho = local_token * g + head_in_group, whole tokens per
 // tile).  Per 64-key tile: loader warps bring the pages' rows by TMA (128-byte swizzle) into
@@ -183,7 +185,8 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
     const int* __restrict__ ctx_len, const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
     int H, int Hkv, int ps, int box_rows, float scale_log2, int window, int* __restrict__ status, int tied,
     const bf16* __restrict__ gate, int ldg, int maps, float* __restrict__ out32, int ldo32,
-    float cap_in, float cap_back, const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias) {
+    float cap_in, float cap_back, const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias,
+    const float* __restrict__ slopes, float inv_scale, float out_scale) {
     // cap_in > 0: a soft cap c on the scaled scores.  With s the raw score, cap_in = 2 log2(e) scale / c
     // and cap_back = c / scale, the raw score becomes cap_back tanh(s scale / c), so that what follows
     // (which multiplies by scale log2 e) sees the capped score; tanh(x) = 1 - 2 / (e^(2x) + 1).
@@ -386,6 +389,8 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
         const int all_first = window > 0 ? p_last - window + 1 : chunk > 0 ? p_last - p_last % chunk : 0;
         float m_ref = -INFINITY, l = 0.f;
         const float bias2 = sig_bias != nullptr && r < nrows ? sig_bias[kvh * g + r % g] * 1.4426950408889634f : 0.f;
+        // (raw scores are multiplied by scale * log2 e below: the slope divided by scale)
+        const float slope = slopes != nullptr && r < nrows ? slopes[kvh * g + r % g] * inv_scale : 0.f;
         bool ok = true;
         for (int j = 0; j < ntiles && ok; ++j) {
             if (!mbar_spin(&s_full[j & 1], (j >> 1) & 1)) { if (lane == 0) gave_up(status, 0x301, 2, j, ntiles); ok = false; break; }
@@ -404,6 +409,14 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
                     }
             }
             const int k0 = kbeg + j * BN;
+            if (slopes != nullptr) {
+                const float base = slope * (float)(k0 - pos);
+#pragma unroll
+                for (int h = 0; h < 2; ++h)
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        raw[h][i] = __float_as_uint(fmaf(slope, (float)(h * 32 + i), __uint_as_float(raw[h][i]) + base));
+            }
             // raw scores stay unscaled; masked ones become -inf.  A tile that every row of
             // the block sees completely needs no mask (rows of padding compute garbage that
             // is never stored).
@@ -488,6 +501,7 @@ __global__ void __launch_bounds__(THREADS, TMEM_COLS == 512 ? 1 : 2) attention_k
             l += (m_ref == -INFINITY) ? 1.f : exp2f(sink[kvh * g + hg] * 1.4426950408889634f - m_ref);
         float inv = l > 0.f ? 1.f / l : 0.f;
         if (sig_bias != nullptr) inv = 1.f;
+        inv *= out_scale;
         if (gate != nullptr && r < nrows)
             inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)(q0 + tok0 + tl) * ldg + kvh * g + hg])));
         bf16* dst = out + (size_t)(q0 + tok0 + tl) * ldo + (size_t)(kvh * g + hg) * DV;
@@ -544,9 +558,10 @@ static int launch_attention_kv_tc(const bf16* q, int ldq, const bf16* kc, const 
                                   const int* tile_seq, const int* tile_row0, int num_tiles, int H, int Hkv, int ps,
                                   int num_pages, float scale, int window, const bf16* gate, int ldg, int maps,
                                   float* out32, int ldo32, cudaStream_t st, float softcap = 0.f,
-                                  const float* sink = nullptr, int chunk = 0, const float* sig_bias = nullptr) {
+                                  const float* sink = nullptr, int chunk = 0, const float* sig_bias = nullptr,
+                                  const float* slopes = nullptr, float out_scale = 1.f) {
     if (num_tiles <= 0) return 0;
-    if (softcap < 0.f || (sink != nullptr && maps != 1)) return SLB_ERR_BAD_ARG;
+    if (softcap < 0.f || ((sink != nullptr || slopes != nullptr) && maps != 1)) return SLB_ERR_BAD_ARG;
     if (chunk < 0 || (chunk > 0 && window > 0) || (sig_bias != nullptr && (maps != 1 || sink != nullptr)))
         return SLB_ERR_BAD_ARG;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || max_pages <= 0 || num_pages <= 0 || !(scale > 0.f) || maps < 1 ||
@@ -584,7 +599,7 @@ static int launch_attention_kv_tc(const bf16* q, int ldq, const bf16* kc, const 
                       map_k, map_v, out, ldo, block_table, max_pages, cu_q, ctx_len, tile_seq, tile_row0, H, Hkv,
                       ps, box_rows, scale * 1.4426950408889634f, window, status, tied, gate, ldg, maps, out32, ldo32,
                       softcap > 0.f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.f,
-                      softcap > 0.f ? softcap / scale : 0.f, sink, chunk, sig_bias);
+                      softcap > 0.f ? softcap / scale : 0.f, sink, chunk, sig_bias, slopes, 1.0f / scale, out_scale);
 }
 
 extern "C" {
@@ -600,16 +615,17 @@ int slb_attention_kv_tc_bf16(const bf16* q, int ldq, const bf16* kc, const bf16*
 }
 // The same with a soft cap on the scaled scores (`softcap` > 0: s <- softcap tanh(s / softcap)) and a
 // sink a head (`sink` [H] float32 or null) in the softmax's denominator; with `chunk` > 0 instead of the
-// window and `sig_bias` ([H] float32 or null) instead of the softmax.
+// window and `sig_bias` ([H] float32 or null) instead of the softmax; with slopes of a distance bias
+// (`slopes` [H] float32 or null) and a factor on the results.
 int slb_attention_kv_tc_capped_bf16(const bf16* q, int ldq, const bf16* kc, const bf16* vc, int tied, bf16* out,
                                     int ldo, const int* block_table, int max_pages, const int* cu_q,
                                     const int* ctx_len, const int* tile_seq, const int* tile_row0, int num_tiles,
                                     int H, int Hkv, int ps, int num_pages, float scale, int window, const bf16* gate,
                                     int ldg, float softcap, const float* sink, int chunk, const float* sig_bias,
-                                    cudaStream_t st) {
+                                    const float* slopes, float out_scale, cudaStream_t st) {
     return launch_attention_kv_tc(q, ldq, kc, vc, tied, out, ldo, block_table, max_pages, cu_q, ctx_len, tile_seq,
                                   tile_row0, num_tiles, H, Hkv, ps, num_pages, scale, window, gate, ldg, 1, nullptr,
-                                  0, st, softcap, sink, chunk, sig_bias);
+                                  0, st, softcap, sink, chunk, sig_bias, slopes, out_scale);
 }
 // `maps` attention maps a head: q [T][H][maps][DK], k_cache [num_pages][Hkv][ps][maps * DK], one set
 // of values a kv head, float32 results per map out32 [T][H][maps][DV].
@@ -652,7 +668,8 @@ int slb_attention_kv_tc_bf16(const bf16*, int, const bf16*, const bf16*, int, bf
 }
 int slb_attention_kv_tc_capped_bf16(const bf16*, int, const bf16*, const bf16*, int, bf16*, int, const int*, int,
                                     const int*, const int*, const int*, const int*, int, int, int, int, int, float,
-                                    int, const bf16*, int, float, const float*, int, const float*, cudaStream_t) {
+                                    int, const bf16*, int, float, const float*, int, const float*, const float*, float,
+                                    cudaStream_t) {
     return SLB_ERR_BAD_ARG;
 }
 int slb_attention_kv_tc_maps_bf16(const bf16*, int, const bf16*, const bf16*, float*, int, const int*, int, const int*,

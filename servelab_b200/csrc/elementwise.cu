@@ -7,7 +7,7 @@
 // Reference analogues: F.embedding (servelab/parallel/tp_model.py:123), RMSNorm
 // (servelab/attention/triton/paged_attention.py:76-91: one program per row,
 // float32 x*rsqrt(mean(x^2)+eps)*w), silu(gate)*up (tp_model.py:67-68).
-#include "common.cuh"
+#include "gated_act.cuh"
 
 // Vector helpers: 4 consecutive elements as float4 (float32: one 16-byte access,
 // bfloat16: one 8-byte access).  Callers guarantee the alignment.
@@ -315,6 +315,100 @@ __global__ void add_rmsnorm_parts_cluster_kernel(float* __restrict__ resid,
     if (threadIdx.x == 0) slb_trace_event(tr, 6, SLB_TR_END);
 }
 
+// ---- a sublayer's result that passes a norm of its own before it is added ----
+// One block per output row r, src = row_map ? row_map[r] : r:
+//   v = resid[src] + rmsnorm(delta[src]; post_eps) * post_w
+//   if no row_map: resid[src] = v
+//   out[r] = rmsnorm(v; eps) * weight
+// The update comes as a tensor or as K-split partial sums (with a bias), as above.  REGS: h % 4 == 0 and the
+// row fits NORM_NV vectors a thread, so update and stream stay in registers between the two norms.
+template <typename TD, typename TO, bool REGS>
+__global__ void post_add_rmsnorm_kernel(float* __restrict__ resid, const TD* __restrict__ delta,
+                                        const float* __restrict__ parts, int nparts, size_t part_stride,
+                                        const float* __restrict__ pbias, const float* __restrict__ post_w,
+                                        float post_eps, const float* __restrict__ weight, TO* __restrict__ out,
+                                        const int* __restrict__ row_map, int h, float eps) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    const int r = blockIdx.x;
+    if constexpr (REGS) {
+        float4 pv[NORM_NV], wv[NORM_NV];                   // (the weights are written by no kernel)
+#pragma unroll
+        for (int j = 0; j < NORM_NV; ++j) {
+            const int i = (threadIdx.x + j * blockDim.x) * 4;
+            pv[j] = i < h ? load4(post_w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            wv[j] = i < h ? load4(weight + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        pdl_wait();
+        const int src = row_map ? row_map[r] : r;
+        float* x = resid + (size_t)src * h;
+        const TD* d = delta ? delta + (size_t)src * h : nullptr;
+        const float* pp = nparts > 0 ? parts + (size_t)src * h : nullptr;
+        float4 xv[NORM_NV], dv[NORM_NV];
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < NORM_NV; ++j) {
+            const int i = (threadIdx.x + j * blockDim.x) * 4;
+            xv[j] = i < h ? load4(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            dv[j] = i < h ? delta4(d, pp, nparts, part_stride, pbias, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < NORM_NV; ++j) {
+            ss += dv[j].x * dv[j].x;
+            ss += dv[j].y * dv[j].y;
+            ss += dv[j].z * dv[j].z;
+            ss += dv[j].w * dv[j].w;
+        }
+        const float pr = 1.0f / sqrtf(block_sum(ss, scratch) / (float)h + post_eps);
+        ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < NORM_NV; ++j) {
+            const int i = (threadIdx.x + j * blockDim.x) * 4;
+            xv[j].x += dv[j].x * pr * pv[j].x; xv[j].y += dv[j].y * pr * pv[j].y;
+            xv[j].z += dv[j].z * pr * pv[j].z; xv[j].w += dv[j].w * pr * pv[j].w;
+            if (row_map == nullptr && i < h) store4(x + i, xv[j]);
+            ss += xv[j].x * xv[j].x;
+            ss += xv[j].y * xv[j].y;
+            ss += xv[j].z * xv[j].z;
+            ss += xv[j].w * xv[j].w;
+        }
+        const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)h + eps);
+        TO* o = out + (size_t)r * h;
+#pragma unroll
+        for (int j = 0; j < NORM_NV; ++j) {
+            const int i = (threadIdx.x + j * blockDim.x) * 4;
+            if (i < h)
+                store4(o + i, make_float4(xv[j].x * rstd * wv[j].x, xv[j].y * rstd * wv[j].y,
+                                          xv[j].z * rstd * wv[j].z, xv[j].w * rstd * wv[j].w));
+        }
+    } else {
+        pdl_wait();
+        const int src = row_map ? row_map[r] : r;
+        float* x = resid + (size_t)src * h;
+        const TD* d = delta ? delta + (size_t)src * h : nullptr;
+        const float* pp = nparts > 0 ? parts + (size_t)src * h : nullptr;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < h; i += blockDim.x) {
+            const float v = delta1(d, pp, nparts, part_stride, pbias, i);
+            ss += v * v;
+        }
+        const float pr = 1.0f / sqrtf(block_sum(ss, scratch) / (float)h + post_eps);
+        ss = 0.f;
+        for (int i = threadIdx.x; i < h; i += blockDim.x) {
+            const float v = x[i] + delta1(d, pp, nparts, part_stride, pbias, i) * pr * post_w[i];
+            if (row_map == nullptr) x[i] = v;
+            ss += v * v;
+        }
+        const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)h + eps);
+        TO* o = out + (size_t)r * h;
+        for (int i = threadIdx.x; i < h; i += blockDim.x) {
+            float v = x[i];
+            if (row_map != nullptr) v += delta1(d, pp, nparts, part_stride, pbias, i) * pr * post_w[i];
+            o[i] = from_float<TO>(v * rstd * weight[i]);
+        }
+    }
+}
+
 // out[t, i] = silu(gate_i) * up_i, silu(z) = z / (1 + exp(-z)), in float32.  Layout of a
 // row of gu: block == 0: all gates, then all ups (gate_i at i, up_i at inter + i);
 // block > 0: gates and ups alternate in runs of `block` (gate_i at (i / block) * 2 * block +
@@ -322,40 +416,18 @@ __global__ void add_rmsnorm_parts_cluster_kernel(float* __restrict__ resid,
 // weights delivers them.
 // V elements per thread and step: 8 (bfloat16 with inter, block, ld_gu and ld_out multiples
 // of 8: 16-byte accesses), 4 (multiples of 4) or 1.
-__device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + expf(-g)) * u; }
-// For results that are rounded to bfloat16: the hardware exponential and reciprocal (errors of
-// a few 1e-7 relative, a thousand times below the rounding), a third of the instructions
-// (42.4 against 47.8 us for 2,048 tokens of the 7B shape).
-__device__ __forceinline__ float silu_mul_fast(float g, float u) {
-    return g * __frcp_rn(1.0f + __expf(-g)) * u;
-}
-
-// the tanh form of GELU: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
-__device__ __forceinline__ float gelu_tanh_mul(float g, float u) {
-    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-}
-// the clamped form: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1)
-__device__ __forceinline__ float swish_clamped_mul(float g, float u, float limit, float alpha) {
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
-}
-template <int ACT> __device__ __forceinline__ float act_mul(float g, float u, float p0, float p1) {
-    return ACT == 2 ? swish_clamped_mul(g, u, p0, p1) : ACT == 1 ? gelu_tanh_mul(g, u) : silu_mul(g, u);
-}
-template <int ACT> __device__ __forceinline__ float act_mul_fast(float g, float u, float p0, float p1) {
-    return ACT == 2 ? swish_clamped_mul(g, u, p0, p1) : ACT == 1 ? gelu_tanh_mul(g, u) : silu_mul_fast(g, u);
-}
-
-// ACT 0: SiLU; 1: GELU (tanh form); 2: the clamped form with p0 = limit, p1 = alpha
+// ACT 0: SiLU; 1: GELU (tanh form); 2: the clamped form with p0 = limit, p1 = alpha.  `row_scale` (or null): a
+// factor a row on gate and up before the activation.
 template <typename T, int V, int ACT>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter,
-                              int ld_gu, int ld_out, int block, float p0, float p1) {
+                              int ld_gu, int ld_out, int block, float p0, float p1,
+                              const float* __restrict__ row_scale) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.y;
     const T* row = gu + (size_t)t * ld_gu;
     T* o = out + (size_t)t * ld_out;
+    const float rs = row_scale != nullptr ? row_scale[t] : 1.f;
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (i >= inter) return;
     const int gi = block > 0 ? (i / block) * 2 * block + i % block : i;     // where gate_i sits
@@ -371,15 +443,17 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const float2 g = __bfloat1622float2(g2[e]), u = __bfloat1622float2(u2[e]);
-            r2[e] = __floats2bfloat162_rn(act_mul_fast<ACT>(g.x, u.x, p0, p1), act_mul_fast<ACT>(g.y, u.y, p0, p1));
+            r2[e] = __floats2bfloat162_rn(act_mul_fast<ACT>(g.x * rs, u.x * rs, p0, p1),
+                                          act_mul_fast<ACT>(g.y * rs, u.y * rs, p0, p1));
         }
         *reinterpret_cast<uint4*>(o + i) = res;
     } else if constexpr (V == 4) {
         const float4 g = load4(row + gi), u = load4(row + ui);
-        store4(o + i, make_float4(act_mul<ACT>(g.x, u.x, p0, p1), act_mul<ACT>(g.y, u.y, p0, p1),
-                                  act_mul<ACT>(g.z, u.z, p0, p1), act_mul<ACT>(g.w, u.w, p0, p1)));
+        store4(o + i, make_float4(act_mul<ACT>(g.x * rs, u.x * rs, p0, p1), act_mul<ACT>(g.y * rs, u.y * rs, p0, p1),
+                                  act_mul<ACT>(g.z * rs, u.z * rs, p0, p1),
+                                  act_mul<ACT>(g.w * rs, u.w * rs, p0, p1)));
     } else {
-        o[i] = from_float<T>(act_mul<ACT>(to_float(row[gi]), to_float(row[ui]), p0, p1));
+        o[i] = from_float<T>(act_mul<ACT>(to_float(row[gi]) * rs, to_float(row[ui]) * rs, p0, p1));
     }
 }
 
@@ -419,22 +493,37 @@ static int launch_add_rmsnorm(float* resid, const TD* delta, const float* parts,
 #undef SLB_NORM_LAUNCH
 }
 
+template <typename TD, typename TO>
+static int launch_post_add_rmsnorm(float* resid, const TD* delta, const float* parts, int nparts, long long part_stride,
+                                   const float* pbias, const float* post_w, float post_eps, const float* weight,
+                                   TO* out, const int* row_map, int rows, int h, float eps, cudaStream_t st) {
+    if (rows <= 0) return 0;
+    if (h <= 0 || nparts < 0 || (nparts > 0) == (delta != nullptr) || (nparts > 0 && parts == nullptr))
+        return SLB_ERR_BAD_ARG;
+    const int threads = norm_threads(h);
+    if (h % 4 == 0 && part_stride % 4 == 0 && h <= threads * 4 * NORM_NV)
+        return slb_launch(post_add_rmsnorm_kernel<TD, TO, true>, dim3(rows), dim3(threads), 0, st, resid, delta, parts,
+                          nparts, (size_t)part_stride, pbias, post_w, post_eps, weight, out, row_map, h, eps);
+    return slb_launch(post_add_rmsnorm_kernel<TD, TO, false>, dim3(rows), dim3(threads), 0, st, resid, delta, parts,
+                      nparts, (size_t)part_stride, pbias, post_w, post_eps, weight, out, row_map, h, eps);
+}
+
 template <typename T, int ACT>
 static int launch_swiglu(const T* gu, T* out, int T_, int inter, int ld_gu, int ld_out, int block,
-                         cudaStream_t st, float p0 = 0.f, float p1 = 0.f) {
+                         cudaStream_t st, float p0 = 0.f, float p1 = 0.f, const float* row_scale = nullptr) {
     if (T_ <= 0) return 0;
     if (inter <= 0 || T_ > 65535 || block < 0 || (block > 0 && inter % block)) return SLB_ERR_BAD_ARG;
     if constexpr (sizeof(T) == 2) {
         if (inter % 8 == 0 && block % 8 == 0 && ld_gu % 8 == 0 && ld_out % 8 == 0 &&
             ((uintptr_t)gu | (uintptr_t)out) % 16 == 0)
             return slb_launch(swiglu_kernel<T, 8, ACT>, dim3((inter / 8 + 255) / 256, T_), dim3(256), 0, st,
-                              gu, out, inter, ld_gu, ld_out, block, p0, p1);
+                              gu, out, inter, ld_gu, ld_out, block, p0, p1, row_scale);
     }
     if (inter % 4 == 0 && block % 4 == 0 && ld_gu % 4 == 0 && ld_out % 4 == 0)
         return slb_launch(swiglu_kernel<T, 4, ACT>, dim3((inter / 4 + 255) / 256, T_), dim3(256), 0, st,
-                          gu, out, inter, ld_gu, ld_out, block, p0, p1);
+                          gu, out, inter, ld_gu, ld_out, block, p0, p1, row_scale);
     return slb_launch(swiglu_kernel<T, 1, ACT>, dim3((inter + 255) / 256, T_), dim3(256), 0, st, gu,
-                      out, inter, ld_gu, ld_out, block, p0, p1);
+                      out, inter, ld_gu, ld_out, block, p0, p1, row_scale);
 }
 
 SLB_DEFINE_PDL_SWITCH
@@ -500,6 +589,21 @@ int slb_add_rmsnorm_parts_bf16(float* resid, const float* parts, int nparts, lon
                                           out, row_map, rows, h, eps, st);
 }
 
+// resid += rmsnorm(update) * post_w, then the norm of the sum; the update is `delta` or, with nparts > 0, partial
+// sums [nparts][rows_total][h] (+ bias)
+int slb_post_add_rmsnorm_f32(float* resid, const float* delta, const float* parts, int nparts, long long part_stride,
+                             const float* pbias, const float* post_w, float post_eps, const float* weight, float* out,
+                             const int* row_map, int rows, int h, float eps, cudaStream_t st) {
+    return launch_post_add_rmsnorm<float, float>(resid, delta, parts, nparts, part_stride, pbias, post_w, post_eps,
+                                                 weight, out, row_map, rows, h, eps, st);
+}
+int slb_post_add_rmsnorm_bf16(float* resid, const bf16* delta, const float* parts, int nparts, long long part_stride,
+                              const float* pbias, const float* post_w, float post_eps, const float* weight, bf16* out,
+                              const int* row_map, int rows, int h, float eps, cudaStream_t st) {
+    return launch_post_add_rmsnorm<bf16, bf16>(resid, delta, parts, nparts, part_stride, pbias, post_w, post_eps,
+                                               weight, out, row_map, rows, h, eps, st);
+}
+
 // block: 0, or the run length in which gates and ups alternate in a row of gu
 int slb_swiglu_f32(const float* gu, float* out, int T, int inter, int ld_gu, int ld_out, int block,
                    cudaStream_t st) {
@@ -509,29 +613,23 @@ int slb_swiglu_bf16(const bf16* gu, bf16* out, int T, int inter, int ld_gu, int 
                     cudaStream_t st) {
     return launch_swiglu<bf16, 0>(gu, out, T, inter, ld_gu, ld_out, block, st);
 }
-// the same with the activation as an argument: 0 SiLU, 1 GELU (tanh form)
+// the same with the activation as an argument: 0 SiLU, 1 GELU (tanh form), 2 the clamped form (g = min(gate, limit),
+// u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1)); `row_scale` [T] or null: a factor a row on gate and up
 int slb_gated_act_f32(const float* gu, float* out, int T, int inter, int ld_gu, int ld_out, int block, int act,
-                      cudaStream_t st) {
-    if (act == 0) return launch_swiglu<float, 0>(gu, out, T, inter, ld_gu, ld_out, block, st);
-    if (act == 1) return launch_swiglu<float, 1>(gu, out, T, inter, ld_gu, ld_out, block, st);
+                      float limit, float alpha, const float* row_scale, cudaStream_t st) {
+    if (act == 0) return launch_swiglu<float, 0>(gu, out, T, inter, ld_gu, ld_out, block, st, 0.f, 0.f, row_scale);
+    if (act == 1) return launch_swiglu<float, 1>(gu, out, T, inter, ld_gu, ld_out, block, st, 0.f, 0.f, row_scale);
+    if (act == 2 && limit > 0.f)
+        return launch_swiglu<float, 2>(gu, out, T, inter, ld_gu, ld_out, block, st, limit, alpha, row_scale);
     return SLB_ERR_BAD_ARG;
 }
 int slb_gated_act_bf16(const bf16* gu, bf16* out, int T, int inter, int ld_gu, int ld_out, int block, int act,
-                       cudaStream_t st) {
-    if (act == 0) return launch_swiglu<bf16, 0>(gu, out, T, inter, ld_gu, ld_out, block, st);
-    if (act == 1) return launch_swiglu<bf16, 1>(gu, out, T, inter, ld_gu, ld_out, block, st);
+                       float limit, float alpha, const float* row_scale, cudaStream_t st) {
+    if (act == 0) return launch_swiglu<bf16, 0>(gu, out, T, inter, ld_gu, ld_out, block, st, 0.f, 0.f, row_scale);
+    if (act == 1) return launch_swiglu<bf16, 1>(gu, out, T, inter, ld_gu, ld_out, block, st, 0.f, 0.f, row_scale);
+    if (act == 2 && limit > 0.f)
+        return launch_swiglu<bf16, 2>(gu, out, T, inter, ld_gu, ld_out, block, st, limit, alpha, row_scale);
     return SLB_ERR_BAD_ARG;
-}
-// the clamped form: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1)
-int slb_gated_act_clamped_f32(const float* gu, float* out, int T, int inter, int ld_gu, int ld_out, int block,
-                              float limit, float alpha, cudaStream_t st) {
-    if (!(limit > 0.f)) return SLB_ERR_BAD_ARG;
-    return launch_swiglu<float, 2>(gu, out, T, inter, ld_gu, ld_out, block, st, limit, alpha);
-}
-int slb_gated_act_clamped_bf16(const bf16* gu, bf16* out, int T, int inter, int ld_gu, int ld_out, int block,
-                               float limit, float alpha, cudaStream_t st) {
-    if (!(limit > 0.f)) return SLB_ERR_BAD_ARG;
-    return launch_swiglu<bf16, 2>(gu, out, T, inter, ld_gu, ld_out, block, st, limit, alpha);
 }
 
 }  // extern "C"

@@ -1,6 +1,9 @@
 // What happens to the projected queries, keys and values of a step between the product and the
 // attention, for mixers that norm heads and rotate neighbouring pairs:
 //
+//   optional biases on the projected queries, keys and values (rows of H * Dq, G * Dk, G * Dv);
+//   optional RMS norm of ALL query heads of a token together, and of all key heads (`row_norm`), with a
+//   weight for every element of the row;
 //   per query head and per key head (a "vector" of D elements of the product's row):
 //     * RMS norm over its first `norm_dims` elements with a weight shared by the heads
 //       (x / sqrt(mean(x^2) + eps) * w; 0: no norm);
@@ -42,7 +45,20 @@ struct HeadPrepArgs {
     void* q_out; int ldq; void* k_cache; void* v_cache;
     int q_head_stride, q_skip;
     int rot_half, q_unit_dims, k_unit_dims;
+    const float* q_bias; const float* k_bias; const float* v_bias;     // or null
+    int row_norm;                  // the norm weights q_norm_w, k_norm_w then have H * Dq and G * Dk elements
 };
+
+// sum of squares of n elements (+ bias) of a row over the block; the order depends on n alone
+template <typename T>
+__device__ __forceinline__ float row_square_sum(const T* row, const float* bias, int n, float* scratch) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += HP_WARPS * 32) {
+        const float v = to_float(row[i]) + (bias != nullptr ? bias[i] : 0.f);
+        ss += v * v;
+    }
+    return block_sum(ss, scratch);
+}
 
 template <typename T>
 __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrepArgs a) {
@@ -63,6 +79,12 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
         cs_tab[i] = cs * a.rot_mag;
         sn_tab[i] = sn * a.rot_mag;
     }
+    __shared__ float scratch[33];
+    float q_rstd = 1.f, k_rstd = 1.f;
+    if (a.row_norm) {
+        q_rstd = 1.0f / sqrtf(row_square_sum(row + a.q_off, a.q_bias, a.H * a.Dq, scratch) / (float)(a.H * a.Dq) + a.eps);
+        k_rstd = 1.0f / sqrtf(row_square_sum(row + a.k_off, a.k_bias, a.G * a.Dk, scratch) / (float)(a.G * a.Dk) + a.eps);
+    }
     __syncthreads();
     // where this token's key and value go
     long long slot = -1;
@@ -82,6 +104,8 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
         T* dst = nullptr;
         int D, norm_dims = 0, rot_off = 0, unit_dims = 0;
         const float* nw = nullptr;
+        const float* bias = nullptr;                   // of this vector
+        float rstd = 1.f;
         bool rotate = a.rot_dims > 0;
         int vhead = -1, skip = 0;
         if (u < a.H) {
@@ -89,21 +113,26 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
             src = row + a.q_off + (size_t)u * D;
             dst = reinterpret_cast<T*>(a.q_out) + (size_t)t * a.ldq + (size_t)u * a.q_head_stride;
             skip = a.q_skip;
+            if (a.q_bias != nullptr) bias = a.q_bias + (size_t)u * D;
+            if (a.row_norm) { rstd = q_rstd; nw += (size_t)u * D; }
         } else if (u < a.H + a.G) {
             const int g = u - a.H;
             D = a.Dk; norm_dims = a.k_norm_dims; nw = a.k_norm_w; rot_off = a.k_rot_off; unit_dims = a.k_unit_dims;
             src = row + a.k_off + (size_t)g * D;
+            if (a.k_bias != nullptr) bias = a.k_bias + (size_t)g * D;
+            if (a.row_norm) { rstd = k_rstd; nw += (size_t)g * D; }
             if (a.k_cache != nullptr && slot >= 0)
                 dst = reinterpret_cast<T*>(a.k_cache) + (size_t)(slot + (long long)g * a.page_size) * D;
         } else {
             vhead = u - a.H - a.G;
             D = a.Dv; rotate = false;
             src = row + a.v_off + (size_t)vhead * D;
+            if (a.v_bias != nullptr) bias = a.v_bias + (size_t)vhead * D;
             if (a.v_cache != nullptr && slot >= 0)
                 dst = reinterpret_cast<T*>(a.v_cache) + (size_t)(slot + (long long)vhead * a.page_size) * D;
         }
         __syncwarp();
-        for (int i = lane; i < D; i += 32) buf[i] = to_float(src[i]);
+        for (int i = lane; i < D; i += 32) buf[i] = to_float(src[i]) + (bias != nullptr ? bias[i] : 0.f);
         __syncwarp();
         if (vhead >= 0) {
             if (a.v_keep != nullptr) {
@@ -116,7 +145,9 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
                 for (int i = lane; i < D; i += 32) buf[i] = (1.0f - lam) * buf[i] + lam * to_float(vf[i]);
             }
         } else {
-            if (norm_dims > 0) {
+            if (a.row_norm) {
+                for (int i = lane; i < D; i += 32) buf[i] = buf[i] * rstd * nw[i];
+            } else if (norm_dims > 0) {
                 float ss = 0.f;
                 for (int i = lane; i < norm_dims; i += 32) ss += buf[i] * buf[i];
                 ss = warp_sum(ss);
@@ -174,6 +205,7 @@ static int launch_head_prep(const HeadPrepArgs& a, int num_tokens, cudaStream_t 
     if (a.rot_dims > 0 && (a.freq == nullptr || (a.H > 0 && a.q_rot_off + a.rot_dims > a.Dq) ||
                            (a.G > 0 && a.k_rot_off + a.rot_dims > a.Dk)))
         return SLB_ERR_BAD_ARG;
+    if (a.row_norm && (a.q_norm_w == nullptr || a.k_norm_w == nullptr || a.H <= 0 || a.G <= 0)) return SLB_ERR_BAD_ARG;
     if (a.q_norm_dims > a.Dq || a.k_norm_dims > a.Dk || a.q_skip < 0 || a.q_skip > a.Dq) return SLB_ERR_BAD_ARG;
     if (a.q_unit_dims < 0 || a.q_unit_dims > a.Dq || a.k_unit_dims < 0 || a.k_unit_dims > a.Dk) return SLB_ERR_BAD_ARG;
     if ((a.k_cache != nullptr || a.v_cache != nullptr) && (a.block_table == nullptr || a.page_size <= 0))

@@ -143,6 +143,63 @@ __global__ void __launch_bounds__(128) group_norm_gate_kernel(
     }
 }
 
+// The gate before the norm: v = x * act(gate), every one of `groups` equal parts of a row divided by its own root
+// mean square, times a weight over the row and a factor.  A block a (token, part); x float32, float32 arithmetic;
+// up to GGN_NV elements a thread stay in registers, longer parts are formed again.
+#define GGN_THREADS 256
+#define GGN_NV 8
+__device__ __forceinline__ float gated_by(float x, float z, int gate_act) {
+    const float sg = 1.0f / (1.0f + expf(-z));
+    return x * (gate_act == 2 ? z * sg : sg);
+}
+template <typename T>
+__global__ void __launch_bounds__(GGN_THREADS) gate_group_norm_kernel(
+    const float* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, int gate_act, const float* __restrict__ w,
+    float eps, float factor, T* __restrict__ out, int ldo, int size) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t t = blockIdx.x;
+    const int c0 = blockIdx.y * size;
+    const float* xr = x + t * ldx + c0;
+    const T* gr = gate + t * ldg + c0;
+    T* o = out + t * ldo + c0;
+    float v[GGN_NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < GGN_NV; ++j) {
+        const int c = threadIdx.x + j * blockDim.x;
+        v[j] = c < size ? gated_by(xr[c], to_float(gr[c]), gate_act) : 0.f;
+        ss += v[j] * v[j];
+    }
+    for (int c = threadIdx.x + GGN_NV * blockDim.x; c < size; c += blockDim.x) {
+        const float u = gated_by(xr[c], to_float(gr[c]), gate_act);
+        ss += u * u;
+    }
+    const float rstd = factor / sqrtf(block_sum(ss, scratch) / (float)size + eps);
+#pragma unroll
+    for (int j = 0; j < GGN_NV; ++j) {
+        const int c = threadIdx.x + j * blockDim.x;
+        if (c < size) o[c] = from_float<T>(v[j] * rstd * (w != nullptr ? w[c0 + c] : 1.f));
+    }
+    for (int c = threadIdx.x + GGN_NV * blockDim.x; c < size; c += blockDim.x)
+        o[c] = from_float<T>(gated_by(xr[c], to_float(gr[c]), gate_act) * rstd * (w != nullptr ? w[c0 + c] : 1.f));
+}
+
+template <typename T>
+static int launch_gate_group_norm(const float* x, int ldx, const T* gate, int ldg, int gate_act, const float* w,
+                                  float eps, float factor, T* out, int ldo, int T_, int groups, int size,
+                                  cudaStream_t st) {
+    if (T_ <= 0) return 0;
+    if (groups <= 0 || groups > 65535 || size <= 0 || gate == nullptr || gate_act < 1 || gate_act > 2 ||
+        ldx < groups * size || ldg < groups * size || ldo < groups * size)
+        return SLB_ERR_BAD_ARG;
+    int threads = (size + 31) / 32 * 32;
+    threads = threads > GGN_THREADS ? GGN_THREADS : threads;
+    return slb_launch(gate_group_norm_kernel<T>, dim3(T_, groups), dim3(threads), 0, st, x, ldx, gate, ldg, gate_act, w,
+                      eps, factor, out, ldo, size);
+}
+
 template <typename T>
 static int launch_hyper_mix_norm(float* X, const T* y, int ldy, const float* M, const float* b, const float* a,
                                  const float* norm_w, float eps, T* out, int ldo, const int* row_map, int rows,
@@ -273,6 +330,14 @@ int slb_hyper_mix_norm_bf16(float* X, const bf16* y, int ldy, const float* M, co
                             const float* norm_w, float eps, bf16* out, int ldo, const int* row_map, int rows, int n,
                             int w, cudaStream_t st) {
     return launch_hyper_mix_norm<bf16>(X, y, ldy, M, b, a, norm_w, eps, out, ldo, row_map, rows, n, w, st);
+}
+int slb_gate_group_norm_f32(const float* x, int ldx, const float* gate, int ldg, int gate_act, const float* w, float eps,
+                            float factor, float* out, int ldo, int T, int groups, int size, cudaStream_t st) {
+    return launch_gate_group_norm<float>(x, ldx, gate, ldg, gate_act, w, eps, factor, out, ldo, T, groups, size, st);
+}
+int slb_gate_group_norm_bf16(const float* x, int ldx, const bf16* gate, int ldg, int gate_act, const float* w, float eps,
+                             float factor, bf16* out, int ldo, int T, int groups, int size, cudaStream_t st) {
+    return launch_gate_group_norm<bf16>(x, ldx, gate, ldg, gate_act, w, eps, factor, out, ldo, T, groups, size, st);
 }
 int slb_group_norm_gate_f32(const float* in, int ldi, int maps, const float* lam, const float* w, float eps,
                             float factor, const float* gate, int ldg, int gate_act, float* out, int ldo, int T,

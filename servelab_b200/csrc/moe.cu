@@ -12,13 +12,17 @@
 //   slb_moe_plan       (token, choice) pairs sorted by expert: counts, offsets, the list, and the
 //                      row tiles of the products (tile -> expert, first row), of a length that
 //                      depends only on the number of pairs and experts (a fixed grid).
-//   slb_moe_gate_up    act[pair] = silu(W_gate[e] x) * (W_up[e] x) for the pair's expert e;
+//   slb_moe_gate_up    act[pair] = silu(W_gate[e] x) * (W_up[e] x) for the pair's expert e, or another gated
+//                      activation; with `in_weights` the expert's input is the pair's weight times x
+//                      (a factor on both sums, since the products are linear);
 //   slb_moe_down       y[pair] = W_down[e] act[pair], float32;
-//   slb_moe_combine    out[t] = (shared[t]) + sum_k weight[t][k] * y[t * top + k], in the order k.
+//   slb_moe_combine    out[t] = (shared[t]) + sum_k weight[t][k] * y[t * top + k], in the order k (no
+//                      weights: the plain sum).
 //
 // Each output element of a product is a sum over k = 0..K-1 in that order (plain FFMA), and the
 // combine adds a token's experts in the order of its choice, so a token's result does not depend
 // on what else is in the batch.
+#include "gated_act.cuh"
 #include "mma_util.cuh"
 
 #define MOE_MAX_EXPERTS 1024
@@ -257,7 +261,7 @@ template <typename T, typename TC, int MODE>
 __global__ void __launch_bounds__(256) moe_product_kernel(
     const T* __restrict__ A, int lda, const T* __restrict__ W, long long w_expert_stride, int ldw,
     TC* __restrict__ C, int ldc, const int* __restrict__ plan, int E, int num_tiles, int P, int top,
-    int N, int K) {
+    int N, int K, int act, float limit, float alpha, const float* __restrict__ in_weights) {
     __shared__ __align__(16) float As[MOE_BK][MOE_BM + 4];
     __shared__ __align__(16) float Ws[MOE_BK][MOE_BN + 4];
     __shared__ __align__(16) float Us[MODE == 0 ? MOE_BK : 1][MOE_BN + 4];
@@ -323,6 +327,7 @@ __global__ void __launch_bounds__(256) moe_product_kernel(
     for (int i = 0; i < 4; ++i) {
         const int pr = rows[ty * 4 + i];
         if (pr < 0) continue;
+        const float iw = MODE == 0 && in_weights != nullptr ? in_weights[pr] : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gn = n0 + tx * 4 + j;
@@ -331,8 +336,8 @@ __global__ void __launch_bounds__(256) moe_product_kernel(
             if (MODE == 0) {
                 // the gate and the up value are rounded to the activations' type first, as two
                 // separate products would leave them
-                const float gte = to_float(from_float<T>(v)), up = to_float(from_float<T>(acu[i][j]));
-                v = gte / (1.0f + expf(-gte)) * up;
+                const float gte = to_float(from_float<T>(v * iw)), up = to_float(from_float<T>(acu[i][j] * iw));
+                v = act_mul_of(act, gte, up, limit, alpha);
             }
             C[(size_t)pr * ldc + gn] = from_float<TC>(v);
         }
@@ -354,7 +359,7 @@ template <int MODE>
 __global__ void __launch_bounds__(128) moe_product_mma_kernel(
     const bf16* __restrict__ A, int lda, const bf16* __restrict__ W, long long w_expert_stride, int ldw,
     void* __restrict__ Cv, int ldc, const int* __restrict__ plan, int E, int num_tiles, int top, int N,
-    int K) {
+    int K, int act, float limit, float alpha, const float* __restrict__ in_weights) {
     using namespace slb_mma;
     __shared__ __align__(16) bf16 As[2][MM_BM][MM_LD];
     __shared__ __align__(16) bf16 Ws[2][MM_BN][MM_LD];
@@ -442,17 +447,16 @@ __global__ void __launch_bounds__(128) moe_product_mma_kernel(
     for (int h = 0; h < 2; ++h) {
         const int pr = rows[warp * 16 + (lane >> 2) + 8 * h];
         if (pr < 0) continue;
+        const float iw = MODE == 0 && in_weights != nullptr ? in_weights[pr] : 1.f;
 #pragma unroll
         for (int j = 0; j < MM_BN / 8; ++j) {
             const int gn = n0 + j * 8 + tig * 2;
             if (gn >= N) continue;                        // (N is even: both columns exist or neither)
             float v0 = acc[j][2 * h], v1 = acc[j][2 * h + 1];
             if (MODE == 0) {
-                const float g0 = __bfloat162float(__float2bfloat16_rn(v0)), g1 = __bfloat162float(__float2bfloat16_rn(v1));
-                const float u0 = __bfloat162float(__float2bfloat16_rn(acu[j][2 * h]));
-                const float u1 = __bfloat162float(__float2bfloat16_rn(acu[j][2 * h + 1]));
-                v0 = g0 / (1.0f + expf(-g0)) * u0;
-                v1 = g1 / (1.0f + expf(-g1)) * u1;
+                auto rounded = [&](float x) { return __bfloat162float(__float2bfloat16_rn(x * iw)); };
+                v0 = act_mul_of(act, rounded(v0), rounded(acu[j][2 * h]), limit, alpha);
+                v1 = act_mul_of(act, rounded(v1), rounded(acu[j][2 * h + 1]), limit, alpha);
                 *reinterpret_cast<unsigned*>(reinterpret_cast<bf16*>(Cv) + (size_t)pr * ldc + gn) = pack_bf16(v0, v1);
             } else {
                 *reinterpret_cast<float2*>(reinterpret_cast<float*>(Cv) + (size_t)pr * ldc + gn) = make_float2(v0, v1);
@@ -471,7 +475,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(
     const int t = blockIdx.x;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < N; c += gridDim.y * blockDim.x) {
         float v = 0.f;
-        for (int k = 0; k < top; ++k) v += weights[(size_t)t * top + k] * to_float(y[((size_t)t * top + k) * ldy + c]);
+        for (int k = 0; k < top; ++k) v += (weights != nullptr ? weights[(size_t)t * top + k] : 1.f) * to_float(y[((size_t)t * top + k) * ldy + c]);
         if (shared != nullptr) v += to_float(shared[(size_t)t * lds + c]);
         out[(size_t)t * ldo + c] = from_float<T>(v);
     }
@@ -480,14 +484,15 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(
 static int moe_num_tiles(int P, int E) { return (P + MOE_BM - 1) / MOE_BM + E; }
 
 template <typename T>
-static int launch_moe_gate_up(const T* x, int ldx, const T* w_gu, int ldw, T* act, int lda,
-                              const int* plan, int E, int P, int top, int I, int K, cudaStream_t st) {
+static int launch_moe_gate_up(const T* x, int ldx, const T* w_gu, int ldw, T* out, int lda,
+                              const int* plan, int E, int P, int top, int I, int K, int act, float limit,
+                              float alpha, const float* in_weights, cudaStream_t st) {
     if (P <= 0) return 0;
-    if (E <= 0 || top <= 0 || I <= 0 || K <= 0) return SLB_ERR_BAD_ARG;
+    if (E <= 0 || top <= 0 || I <= 0 || K <= 0 || act < 0 || act > 2 || (act == 2 && !(limit > 0.f))) return SLB_ERR_BAD_ARG;
     const int nt = moe_num_tiles(P, E);
     if (nt > 65535) return SLB_ERR_TOO_LARGE;
     return slb_launch(moe_product_kernel<T, T, 0>, dim3((I + MOE_BN - 1) / MOE_BN, nt), dim3(256), 0, st, x,
-                      ldx, w_gu, (long long)2 * I * ldw, ldw, act, lda, plan, E, nt, P, top, I, K);
+                      ldx, w_gu, (long long)2 * I * ldw, ldw, out, lda, plan, E, nt, P, top, I, K, act, limit, alpha, in_weights);
 }
 
 template <typename T>
@@ -498,26 +503,28 @@ static int launch_moe_down(const T* act, int lda, const T* w_down, int ldw, floa
     const int nt = moe_num_tiles(P, E);
     if (nt > 65535) return SLB_ERR_TOO_LARGE;
     return slb_launch(moe_product_kernel<T, float, 1>, dim3((N + MOE_BN - 1) / MOE_BN, nt), dim3(256), 0, st,
-                      act, lda, w_down, (long long)N * ldw, ldw, y, ldy, plan, E, nt, P, top, N, I);
+                      act, lda, w_down, (long long)N * ldw, ldw, y, ldy, plan, E, nt, P, top, N, I, 0, 0.f, 0.f, (const float*)nullptr);
 }
 
 template <int MODE>
 static int launch_moe_mma(const bf16* A, int lda, const bf16* W, long long stride, int ldw, void* C, int ldc,
-                          const int* plan, int E, int P, int top, int N, int K, cudaStream_t st) {
+                          const int* plan, int E, int P, int top, int N, int K, cudaStream_t st, int act = 0,
+                          float limit = 0.f, float alpha = 0.f, const float* in_weights = nullptr) {
     if (P <= 0) return 0;
     if (E <= 0 || top <= 0 || N <= 0 || K <= 0 || K % 8 || lda % 8 || ldw % 8 || N % 2 || ldc % 2 ||
-        ((uintptr_t)A & 15) || ((uintptr_t)W & 15) || (stride % 8))
+        ((uintptr_t)A & 15) || ((uintptr_t)W & 15) || (stride % 8) || act < 0 || act > 2 || (act == 2 && !(limit > 0.f)))
         return SLB_ERR_BAD_ARG;
     const int nt = moe_num_tiles(P, E);
     if (nt > 65535) return SLB_ERR_TOO_LARGE;
     return slb_launch(moe_product_mma_kernel<MODE>, dim3((N + MM_BN - 1) / MM_BN, nt), dim3(128), 0, st, A, lda,
-                      W, stride, ldw, C, ldc, plan, E, nt, top, N, K);
+                      W, stride, ldw, C, ldc, plan, E, nt, top, N, K, act, limit, alpha, in_weights);
 }
 
 extern "C" {
-int slb_moe_gate_up_mma_bf16(const bf16* x, int ldx, const bf16* w_gu, int ldw, bf16* act, int lda,
-                             const int* plan, int E, int P, int top, int I, int K, cudaStream_t st) {
-    return launch_moe_mma<0>(x, ldx, w_gu, (long long)2 * I * ldw, ldw, act, lda, plan, E, P, top, I, K, st);
+int slb_moe_gate_up_mma_bf16(const bf16* x, int ldx, const bf16* w_gu, int ldw, bf16* out, int lda,
+                             const int* plan, int E, int P, int top, int I, int K, int act, float limit, float alpha,
+                             const float* in_weights, cudaStream_t st) {
+    return launch_moe_mma<0>(x, ldx, w_gu, (long long)2 * I * ldw, ldw, out, lda, plan, E, P, top, I, K, st, act, limit, alpha, in_weights);
 }
 int slb_moe_down_mma_bf16(const bf16* act, int lda, const bf16* w_down, int ldw, float* y, int ldy,
                           const int* plan, int E, int P, int top, int N, int I, cudaStream_t st) {
@@ -570,13 +577,15 @@ int slb_moe_plan(const int* ids, int P, int E, int* plan, cudaStream_t st) {
     if (E <= 0 || E > MOE_MAX_EXPERTS) return SLB_ERR_BAD_ARG;
     return slb_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, st, ids, P, E, moe_num_tiles(P, E), plan);
 }
-int slb_moe_gate_up_f32(const float* x, int ldx, const float* w_gu, int ldw, float* act, int lda,
-                        const int* plan, int E, int P, int top, int I, int K, cudaStream_t st) {
-    return launch_moe_gate_up<float>(x, ldx, w_gu, ldw, act, lda, plan, E, P, top, I, K, st);
+int slb_moe_gate_up_f32(const float* x, int ldx, const float* w_gu, int ldw, float* out, int lda,
+                        const int* plan, int E, int P, int top, int I, int K, int act, float limit, float alpha,
+                        const float* in_weights, cudaStream_t st) {
+    return launch_moe_gate_up<float>(x, ldx, w_gu, ldw, out, lda, plan, E, P, top, I, K, act, limit, alpha, in_weights, st);
 }
-int slb_moe_gate_up_bf16(const bf16* x, int ldx, const bf16* w_gu, int ldw, bf16* act, int lda,
-                         const int* plan, int E, int P, int top, int I, int K, cudaStream_t st) {
-    return launch_moe_gate_up<bf16>(x, ldx, w_gu, ldw, act, lda, plan, E, P, top, I, K, st);
+int slb_moe_gate_up_bf16(const bf16* x, int ldx, const bf16* w_gu, int ldw, bf16* out, int lda,
+                         const int* plan, int E, int P, int top, int I, int K, int act, float limit, float alpha,
+                         const float* in_weights, cudaStream_t st) {
+    return launch_moe_gate_up<bf16>(x, ldx, w_gu, ldw, out, lda, plan, E, P, top, I, K, act, limit, alpha, in_weights, st);
 }
 int slb_moe_down_f32(const float* act, int lda, const float* w_down, int ldw, float* y, int ldy,
                      const int* plan, int E, int P, int top, int N, int I, cudaStream_t st) {

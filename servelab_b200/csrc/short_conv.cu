@@ -22,7 +22,8 @@
 // With no key heads (Hkv = 0) every channel is a "query" channel: the kernel is then a plain
 // convolution of the first q_size columns into q_out, which a mixer runs on q | k | v before its
 // head kernel.  Two biases are optional: one on the projected rows (`in_bias`: what the record holds
-// then includes it, so the zeros before a sequence's start stay zeros) and one on the result.  The
+// then includes it, so the zeros before a sequence's start stay zeros) and one on the result, and so is SiLU on
+// the result (`act` 1).  The
 // records of two requests lie `state_stride` floats apart (a record may be part of
 // a larger one).
 #include "common.cuh"
@@ -81,7 +82,7 @@ __global__ void __launch_bounds__(256) qk_conv_cache_kernel(
     const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
     float temp_coef, int temp_every, T* __restrict__ q_out, int ldq, T* __restrict__ k_cache,
     int q_size, int Hkv, int D, int update_inline, long long state_stride,
-    const float* __restrict__ in_bias, const float* __restrict__ out_bias) {
+    const float* __restrict__ in_bias, const float* __restrict__ out_bias, int act) {
     const int C = q_size + Hkv * D;
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     pdl_launch_dependents();
@@ -121,6 +122,10 @@ __global__ void __launch_bounds__(256) qk_conv_cache_kernel(
         // a step of single tokens: row i - 1 of the new record is row i of (record, token); this
         // thread alone reads and writes these columns of the record, in this order
         if (update_inline && i >= 1 && st != nullptr) store_vec<float, VEC>(st + (size_t)(i - 1) * C, u);
+    }
+    if (act == 1) {
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) y[v] = y[v] / (1.0f + expf(-y[v]));
     }
     if (c < q_size) {
         if (temp_coef != 0.f) {
@@ -175,7 +180,8 @@ static int launch_conv(const T* proj, int ldp, const float* taps_w, int taps, fl
                        const int* positions, const int* block_table, int max_pages, int page_size,
                        int num_pages, float temp_coef, int temp_every, T* q_out, int ldq, T* k_cache,
                        int T_tokens, int S, int q_size, int Hkv, int D, int decode_only, long long state_stride,
-                       cudaStream_t st, const float* in_bias = nullptr, const float* out_bias = nullptr) {
+                       cudaStream_t st, const float* in_bias = nullptr, const float* out_bias = nullptr,
+                       int act = 0) {
     if (T_tokens <= 0) return 0;
     if (state_stride <= 0) state_stride = (long long)(taps - 1) * (q_size + Hkv * D);
     if (state_stride < (long long)(taps - 1) * (q_size + Hkv * D)) return SLB_ERR_BAD_ARG;
@@ -198,12 +204,12 @@ static int launch_conv(const T* proj, int ldp, const float* taps_w, int taps, fl
         rc = slb_launch(qk_conv_cache_kernel<T, V>, dim3((C / V + threads - 1) / threads, T_tokens), dim3(threads),
                         0, st, proj, ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions,
                         block_table, max_pages, page_size, num_pages, temp_coef, temp_every, q_out, ldq,
-                        k_cache, q_size, Hkv, D, inline_update, state_stride, in_bias, out_bias);
+                        k_cache, q_size, Hkv, D, inline_update, state_stride, in_bias, out_bias, act);
     } else {
         rc = slb_launch(qk_conv_cache_kernel<T, 1>, dim3((C + 255) / 256, T_tokens), dim3(256), 0, st, proj,
                         ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions, block_table,
                         max_pages, page_size, num_pages, temp_coef, temp_every, q_out, ldq, k_cache, q_size,
-                        Hkv, D, inline_update, state_stride, in_bias, out_bias);
+                        Hkv, D, inline_update, state_stride, in_bias, out_bias, act);
     }
     if (rc != 0 || taps == 1 || inline_update) return rc;
     return slb_launch(conv_state_update_kernel<T>, dim3((C + 255) / 256, S), dim3(256), 0, st, proj, ldp,
@@ -211,22 +217,22 @@ static int launch_conv(const T* proj, int ldp, const float* taps_w, int taps, fl
 }
 
 extern "C" {
-// the convolution alone of the first C columns of proj, with biases (null: none)
+// the convolution alone of the first C columns of proj, with biases (null: none) and an activation (0: none; 1: SiLU)
 int slb_short_conv_f32(const float* proj, int ldp, const float* taps_w, int taps, float* state,
                        const int* state_slots, const int* cu_q, const int* seq_of_token, const int* positions,
                        float* out, int ldo, int T_tokens, int S, int C, int decode_only, long long state_stride,
-                       const float* in_bias, const float* out_bias, cudaStream_t st) {
+                       const float* in_bias, const float* out_bias, int act, cudaStream_t st) {
     return launch_conv<float>(proj, ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions, nullptr, 0,
                               1, 0, 0.f, 1, out, ldo, nullptr, T_tokens, S, C, 0, 0, decode_only, state_stride, st,
-                              in_bias, out_bias);
+                              in_bias, out_bias, act);
 }
 int slb_short_conv_bf16(const bf16* proj, int ldp, const float* taps_w, int taps, float* state,
                         const int* state_slots, const int* cu_q, const int* seq_of_token, const int* positions,
                         bf16* out, int ldo, int T_tokens, int S, int C, int decode_only, long long state_stride,
-                        const float* in_bias, const float* out_bias, cudaStream_t st) {
+                        const float* in_bias, const float* out_bias, int act, cudaStream_t st) {
     return launch_conv<bf16>(proj, ldp, taps_w, taps, state, state_slots, cu_q, seq_of_token, positions, nullptr, 0,
                              1, 0, 0.f, 1, out, ldo, nullptr, T_tokens, S, C, 0, 0, decode_only, state_stride, st,
-                             in_bias, out_bias);
+                             in_bias, out_bias, act);
 }
 int slb_qk_conv_cache_f32(const float* proj, int ldp, const float* taps_w, int taps, float* state,
                           const int* state_slots, const int* cu_q, const int* seq_of_token,

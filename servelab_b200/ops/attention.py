@@ -126,7 +126,8 @@ def prepare_kv_attention(key_dim: int, value_dim: int, dtype: torch.dtype) -> No
 
 
 def kv_attention(ctx, q, k_cache, v_cache, v_row_stride, out, table, H, Hkv, Dk, Dv, page_size, scale,
-                 window, head_gate, softcap=None, sink=None, chunk=0, sigmoid_bias=None) -> None:
+                 window, head_gate, softcap=None, sink=None, chunk=0, sigmoid_bias=None, slopes=None,
+                 out_scale=1.0) -> None:
     """Attention with keys of ``Dk`` and values of ``Dv`` elements (value rows ``v_row_stride``
     apart in ``v_cache``, which may be the key cache: the values are then a prefix of the key
     rows), causal with an optional window, head h's row times sigmoid(head_gate[t, h]) if given.
@@ -135,10 +136,12 @@ def kv_attention(ctx, q, k_cache, v_cache, v_row_stride, out, table, H, Hkv, Dk,
     sizes, the mma.sync kernel and the plain kernel take both; the kernels for equal sizes of the
     other models take neither, so a mixer that has one does not reach them; nor do they take ``chunk``
     (a query sees the keys of its own run of ``chunk`` positions) or ``sigmoid_bias`` float32 [H] (weights
-    sigmoid(score + bias), not normalized).
+    sigmoid(score + bias), not normalized), ``slopes`` float32 [H] (slopes[h] (i - j) is taken off the capped
+    score) or ``out_scale`` (a factor on the results).
     float32, or sizes the tensor-core kernel does not take: the plain kernel."""
     tied = v_cache.data_ptr() == k_cache.data_ptr() and v_row_stride == Dk
     modified = bool(softcap) or sink is not None or bool(chunk) or sigmoid_bias is not None
+    modified = modified or slopes is not None or out_scale != 1.0
     if (Dk == Dv and not tied and not modified and v_row_stride == Dv and q.dtype == torch.bfloat16 and not force_generic
             and use_equal_size_kernels and K.has_fast_attention(Dk) and Dk in (64, 128)):
         # keys and values of one size the tcgen05 kernels take: the framework's attention for
@@ -152,13 +155,13 @@ def kv_attention(ctx, q, k_cache, v_cache, v_row_stride, out, table, H, Hkv, Dk,
         if (not ctx.decode_only and out.stride(0) % 8 == 0 and (use_kv_tc_capped or not modified)
                 and K.attention_kv_tc_takes(Dk, Dv, page_size, H // Hkv, tied)):
             K.attention_kv_tc(ctx, q, k_cache, v_cache, tied, out, table, H, Hkv, Dk, Dv, page_size, scale,
-                              window, head_gate, softcap or 0.0, sink, chunk, sigmoid_bias)
+                              window, head_gate, softcap or 0.0, sink, chunk, sigmoid_bias, slopes, out_scale)
             return
         K.attention_kv_mma(ctx, q, k_cache, v_cache, tied, out, table, H, Hkv, Dk, Dv, page_size, scale,
-                           window, head_gate, softcap or 0.0, sink, chunk, sigmoid_bias)
+                           window, head_gate, softcap or 0.0, sink, chunk, sigmoid_bias, slopes, out_scale)
         return
     K.attention_kv(ctx, q, k_cache, v_cache, v_row_stride, out, table, H, Hkv, Dk, Dv, page_size, scale,
-                   window, head_gate, softcap or 0.0, sink, chunk, sigmoid_bias)
+                   window, head_gate, softcap or 0.0, sink, chunk, sigmoid_bias, slopes, out_scale)
 
 
 # ------------------------------------------------- several attention maps a head

@@ -172,6 +172,24 @@ def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torc
                rows, out.shape[1], float(eps), _stream()), "add_rmsnorm")
 
 
+def post_add_rmsnorm(resid: torch.Tensor, update, post_weight: torch.Tensor, post_eps: float, weight: torch.Tensor,
+                     eps: float, out: torch.Tensor, row_map: Optional[torch.Tensor] = None) -> None:
+    """resid += rmsnorm(update) * post_weight (in place, float32; skipped when ``row_map`` selects rows);
+    out[r] = rmsnorm(of that sum's row src(r)) * weight.  ``update``: a tensor or a ``SplitSum``."""
+    parts = None
+    if isinstance(update, SplitSum):
+        if out.dtype == _BF16:
+            parts, update = update, None
+        else:
+            update = update.materialize()
+    S, M, N = parts.parts.shape if parts is not None else (0, 0, 0)
+    fn = getattr(L.core(), "slb_post_add_rmsnorm_" + _suffix(out.dtype))
+    L.check(fn(resid.data_ptr(), _p(update), _p(parts.parts if parts is not None else None), S, M * N,
+               _p(parts.bias if parts is not None else None), post_weight.data_ptr(), float(post_eps),
+               weight.data_ptr(), out.data_ptr(), _p(row_map), out.shape[0], out.shape[1], float(eps), _stream()),
+            "post_add_rmsnorm")
+
+
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> None:
     """out[t, i] = silu(gate_i) * up_i of row t of ``gate_up`` ([T, 2 I], I = out.shape[1]).
     ``block`` == 0: a row holds all gates, then all ups; ``block`` > 0: gates and ups
@@ -352,20 +370,20 @@ def qk_conv_cache(proj: torch.Tensor, taps_w: torch.Tensor, state: Optional[torc
 
 def short_conv(proj: torch.Tensor, taps_w: torch.Tensor, state: Optional[torch.Tensor], ctx,
                out: torch.Tensor, in_bias: Optional[torch.Tensor] = None,
-               out_bias: Optional[torch.Tensor] = None) -> None:
+               out_bias: Optional[torch.Tensor] = None, activation: Optional[str] = None) -> None:
     """The convolution alone: y_t = sum_i taps_w[i] u_(t - taps + 1 + i) on the first C = out.shape[1]
     columns of ``proj`` into ``out`` [T, C]; the rows before a portion come from ``state`` (float32
     [slots, >= (taps - 1) * C], a request's record at ``ctx.state_slots``; rows of the record may be
     ``state.stride(0)`` apart, so it can be a slice of a larger record), which is left holding the
     last taps - 1 projected rows.  ``in_bias`` / ``out_bias`` float32 [C]: added to the projected rows
-    (and so part of the record) / to the result."""
+    (and so part of the record) / to the result.  ``activation``: None or "silu" on the result."""
     fn = getattr(L.core(), "slb_short_conv_" + _suffix(proj.dtype))
     n = 1 if (taps_w.shape[0] == 1 or ctx.decode_only) else 2
     L.check(fn(proj.data_ptr(), proj.stride(0), taps_w.data_ptr(), taps_w.shape[0], _p(state),
                ctx.state_slots.data_ptr(), ctx.cu_q.data_ptr(), ctx.seq_of_token.data_ptr(),
                ctx.positions.data_ptr(), out.data_ptr(), out.stride(0), proj.shape[0], ctx.num_seqs, out.shape[1],
                1 if ctx.decode_only else 0, state.stride(0) if state is not None else 0, _p(in_bias), _p(out_bias),
-               _stream()), "short_conv")
+               {None: 0, "silu": 1}[activation], _stream()), "short_conv")
     global launch_count
     launch_count += n - 1
 
@@ -866,6 +884,7 @@ class _HeadPrepArgs(_ct.Structure):
         ("q_out", _ct.c_void_p), ("ldq", _ct.c_int), ("k_cache", _ct.c_void_p), ("v_cache", _ct.c_void_p),
         ("q_head_stride", _ct.c_int), ("q_skip", _ct.c_int),
         ("rot_half", _ct.c_int), ("q_unit_dims", _ct.c_int), ("k_unit_dims", _ct.c_int),
+        ("q_bias", _ct.c_void_p), ("k_bias", _ct.c_void_p), ("v_bias", _ct.c_void_p), ("row_norm", _ct.c_int),
     ]
 
 
@@ -875,7 +894,8 @@ def head_prep(proj: torch.Tensor, ctx, block_table: torch.Tensor, page_size: int
               v_off: int, v_dim: int, freq, rot_dims: int, rot_mag: float, eps: float,
               q_out: torch.Tensor, k_cache, v_cache, lam=None, v_first=None, v_keep=None,
               q_head_stride: Optional[int] = None, q_skip: int = 0, rot_half: bool = False,
-              q_unit_dims: int = 0, k_unit_dims: int = 0) -> None:
+              q_unit_dims: int = 0, k_unit_dims: int = 0, q_bias=None, k_bias=None, v_bias=None,
+              row_norm: bool = False) -> None:
     """One launch between a mixer's first product and its attention: RMS norm of the first
     ``*_norm_dims`` elements of every query / key head (weight shared by the heads; 0: none),
     rotation of ``rot_dims`` elements from ``*_rot_off`` on (neighbouring pairs, or with
@@ -884,7 +904,10 @@ def head_prep(proj: torch.Tensor, ctx, block_table: torch.Tensor, page_size: int
     by their root mean square (0: not), queries into ``q_out``, keys into the pages;
     (head h at ``q_out[t, h * q_head_stride:]``, without its first ``q_skip`` elements);
     values (``v_off`` < 0: none) mixed with ``v_first`` by ``lam`` (a float32 scalar on the
-    device) or copied to ``v_keep``, and into the pages.  A cache that is None is not written."""
+    device) or copied to ``v_keep``, and into the pages.  A cache that is None is not written.
+    ``q_bias``, ``k_bias``, ``v_bias`` float32: added to the projected rows first.  ``row_norm``: instead of
+    every head, all query heads of a token are RMS-normed together and so are all key heads, with
+    weights of ``num_heads * q_dim`` and ``num_kv_heads * k_dim`` elements."""
     a = _HeadPrepArgs()
     a.proj, a.ld = proj.data_ptr(), proj.stride(0)
     a.q_off, a.H, a.Dq, a.q_norm_dims, a.q_rot_off, a.q_norm_w = (q_off, num_heads, q_dim, q_norm_dims,
@@ -905,6 +928,7 @@ def head_prep(proj: torch.Tensor, ctx, block_table: torch.Tensor, page_size: int
     a.k_cache, a.v_cache = _p(k_cache), _p(v_cache)
     a.q_head_stride, a.q_skip = (q_dim if q_head_stride is None else q_head_stride), q_skip
     a.rot_half, a.q_unit_dims, a.k_unit_dims = int(bool(rot_half)), int(q_unit_dims), int(k_unit_dims)
+    a.q_bias, a.k_bias, a.v_bias, a.row_norm = _p(q_bias), _p(k_bias), _p(v_bias), int(bool(row_norm))
     fn = getattr(L.core(), "slb_head_prep_" + _suffix(proj.dtype))
     L.check(fn(_ct.byref(a), proj.shape[0], _stream()), "head_prep")
 
@@ -934,14 +958,16 @@ def attention_kv(ctx, q, k_cache, v_cache, v_row_stride: int, out, block_table, 
                  num_kv_heads: int, k_dim: int, v_dim: int, page_size: int, scale: float, window: int,
                  head_gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
                  sink: Optional[torch.Tensor] = None, chunk: int = 0,
-                 sigmoid_bias: Optional[torch.Tensor] = None) -> None:
+                 sigmoid_bias: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
+                 out_scale: float = 1.0) -> None:
     """The plain kernel: float32 arithmetic; keys of ``k_dim``, values of ``v_dim`` elements at
     ``v_cache`` with rows ``v_row_stride`` apart (the key cache itself for values that are a
     prefix of the keys); ``head_gate`` [T, >= H]: head h's row times sigmoid(head_gate[t, h]);
     ``softcap`` > 0: a scaled score s becomes softcap tanh(s / softcap); ``sink`` float32 [H]: its
     exponential joins the softmax's denominator; ``chunk`` > 0 (instead of ``window``): a query at i sees
     the keys j <= i with j // chunk == i // chunk; ``sigmoid_bias`` float32 [H] (instead of the
-    softmax): a visible key's weight is sigmoid(score + sigmoid_bias[h]), not normalized."""
+    softmax): a visible key's weight is sigmoid(score + sigmoid_bias[h]), not normalized; ``slopes`` float32
+    [H]: slopes[h] (i - j) is taken off the (capped) score; ``out_scale``: a factor on the results."""
     tile_seq, tile_row0, n = ctx.attention_tiles(num_heads // num_kv_heads, attention_kv_tile_rows())
     fn = getattr(L.core(), "slb_attention_kv_" + _suffix(q.dtype))
     L.check(fn(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), v_row_stride,
@@ -949,7 +975,8 @@ def attention_kv(ctx, q, k_cache, v_cache, v_row_stride: int, out, block_table, 
                ctx.cu_q.data_ptr(), ctx.ctx_len.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), n,
                num_heads, num_kv_heads, k_dim, v_dim, page_size, k_cache.shape[0], float(scale),
                int(window), _p(head_gate), head_gate.stride(0) if head_gate is not None else 0,
-               float(softcap), _p(sink), int(chunk), _p(sigmoid_bias), _stream()), "attention_kv")
+               float(softcap), _p(sink), int(chunk), _p(sigmoid_bias), _p(slopes), float(out_scale), _stream()),
+            "attention_kv")
 
 
 def attention_kv_splits(num_seqs: int, num_kv_heads: int, longest_context: int, window: int,
@@ -984,11 +1011,12 @@ def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num
                      num_kv_heads: int, k_dim: int, v_dim: int, page_size: int, scale: float, window: int,
                      head_gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
                      sink: Optional[torch.Tensor] = None, chunk: int = 0,
-                     sigmoid_bias: Optional[torch.Tensor] = None) -> None:
+                     sigmoid_bias: Optional[torch.Tensor] = None,
+                     slopes: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
     """The tensor-core kernel (bfloat16), for prompt portions and single tokens; in a step of
     single tokens the keys of a request are split over several blocks when the requests alone
-    would not fill the device.  ``softcap``, ``sink``, ``chunk`` and ``sigmoid_bias`` as in
-    ``attention_kv``."""
+    would not fill the device.  ``softcap``, ``sink``, ``chunk``, ``sigmoid_bias``, ``slopes`` and
+    ``out_scale`` as in ``attention_kv``."""
     lib = L.attention_kv(k_dim, v_dim)
     rows = lib.slb_attention_kv_mma_tile_rows()
     tile_seq, tile_row0, n = ctx.attention_tiles(num_heads // num_kv_heads, rows)
@@ -1011,9 +1039,10 @@ def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num
             page_size, k_cache.shape[0], float(scale), int(window), _p(head_gate),
             head_gate.stride(0) if head_gate is not None else 0, splits, _p(part_o), _p(part_ml),
             1 if ctx.decode_only and attention_kv_narrow and num_heads // num_kv_heads <= 16 else 0)
-    if softcap or sink is not None or chunk or sigmoid_bias is not None:
+    if (softcap or sink is not None or chunk or sigmoid_bias is not None or slopes is not None
+            or out_scale != 1.0):
         L.check(lib.slb_attention_kv_mma_capped_bf16(*args, float(softcap or 0.0), _p(sink), int(chunk),
-                                                     _p(sigmoid_bias), _stream()), "attention_kv_mma")
+                                                     _p(sigmoid_bias), _p(slopes), float(out_scale), _stream()), "attention_kv_mma")
         return
     L.check(lib.slb_attention_kv_mma_bf16(*args, _stream()), "attention_kv_mma")
 
@@ -1050,10 +1079,11 @@ def attention_kv_tc(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num_
                     num_kv_heads: int, k_dim: int, v_dim: int, page_size: int, scale: float, window: int,
                     head_gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
                     sink: Optional[torch.Tensor] = None, chunk: int = 0,
-                    sigmoid_bias: Optional[torch.Tensor] = None) -> None:
+                    sigmoid_bias: Optional[torch.Tensor] = None,
+                    slopes: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
     """The tcgen05 kernel (bfloat16; key and value sizes multiples of 64; steps with prompt
     portions): 128 flattened rows a block, accumulators in tensor memory.  ``softcap``, ``sink``,
-    ``chunk`` and ``sigmoid_bias`` as in ``attention_kv``."""
+    ``chunk``, ``sigmoid_bias``, ``slopes`` and ``out_scale`` as in ``attention_kv``."""
     lib = L.attention_kv(k_dim, v_dim)
     group = num_heads // num_kv_heads
     tile_seq, tile_row0, n = ctx.attention_tiles(group, lib.slb_attention_kv_tc_tile_rows(group))
@@ -1062,9 +1092,10 @@ def attention_kv_tc(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num_
             ctx.ctx_len.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), n, num_heads, num_kv_heads,
             page_size, k_cache.shape[0], float(scale), int(window), _p(head_gate),
             head_gate.stride(0) if head_gate is not None else 0)
-    if softcap or sink is not None or chunk or sigmoid_bias is not None:
+    if (softcap or sink is not None or chunk or sigmoid_bias is not None or slopes is not None
+            or out_scale != 1.0):
         L.check(lib.slb_attention_kv_tc_capped_bf16(*args, float(softcap or 0.0), _p(sink), int(chunk),
-                                                    _p(sigmoid_bias), _stream()), "attention_kv_tc")
+                                                    _p(sigmoid_bias), _p(slopes), float(out_scale), _stream()), "attention_kv_tc")
         return
     L.check(lib.slb_attention_kv_tc_bf16(*args, _stream()), "attention_kv_tc")
 
@@ -1148,9 +1179,14 @@ moe_tensor_cores = True        # bfloat16: the experts' products on mma.sync (of
 
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
-                w_down: torch.Tensor, shared: Optional[torch.Tensor]) -> torch.Tensor:
+                w_down: torch.Tensor, shared: Optional[torch.Tensor], activation: str = "silu",
+                limit: Optional[float] = None, alpha: float = 1.0, weight_inputs: bool = False) -> torch.Tensor:
     """sum_k weights[t, k] * down_e(silu(gate_e x_t) * up_e x_t) (+ shared[t]), e = ids[t, k];
-    ``w_gate_up`` [E, 2 I, h] (gate rows, then up rows), ``w_down`` [E, h, I]."""
+    ``w_gate_up`` [E, 2 I, h] (gate rows, then up rows), ``w_down`` [E, h, I].  ``activation``, ``limit``,
+    ``alpha`` as in ``gated_act``.  ``weight_inputs``: the expert's input is weights[t, k] x_t and its results
+    are added as they are."""
+    act_args = (GATED_ACTIVATIONS[activation], float(limit or 0.0), float(alpha))
+    out_weights = None if weight_inputs else weights
     T, top = ids.shape
     E, two_i, h = w_gate_up.shape
     inter = two_i // 2
@@ -1173,14 +1209,18 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         gu = torch._grouped_mm(xs, w_gate_up.transpose(1, 2), offs=ends)
         mark("library grouped gemm")
         act = torch.empty((P, inter), dtype=x.dtype, device=x.device)
-        swiglu(gu, act, 0)
+        if activation == "silu" and not weight_inputs:
+            swiglu(gu, act, 0)
+        else:
+            gated_act(gu, act, 0, activation, limit, alpha,
+                      weights.view(-1).index_select(0, order) if weight_inputs else None)
         ys = torch._grouped_mm(act, w_down.transpose(1, 2), offs=ends)
         mark("library grouped gemm")
         y = torch.empty_like(ys)
         y.index_copy_(0, order.long(), ys)
         out = torch.empty((T, n_out), dtype=x.dtype, device=x.device)
         L.check(lib.slb_moe_combine_bf16_rows(
-            y.data_ptr(), y.stride(0), weights.data_ptr(), _p(shared),
+            y.data_ptr(), y.stride(0), _p(out_weights), _p(shared),
             shared.stride(0) if shared is not None else 0, out.data_ptr(), out.stride(0), T, top, n_out,
             _stream()), "moe_combine")
         return out
@@ -1192,14 +1232,15 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     up_sfx = "mma_bf16" if mma else sfx
     L.check(getattr(lib, "slb_moe_gate_up_" + up_sfx)(
         x.data_ptr(), x.stride(0), w_gate_up.data_ptr(), w_gate_up.stride(1), act.data_ptr(), act.stride(0),
-        plan.data_ptr(), E, P, top, inter, h, _stream()), "moe_gate_up")
+        plan.data_ptr(), E, P, top, inter, h, *act_args, _p(weights if weight_inputs else None), _stream()),
+        "moe_gate_up")
     y = torch.empty((P, n_out), dtype=_F32, device=x.device)
     L.check(getattr(lib, "slb_moe_down_" + up_sfx)(
         act.data_ptr(), act.stride(0), w_down.data_ptr(), w_down.stride(1), y.data_ptr(), y.stride(0),
         plan.data_ptr(), E, P, top, n_out, inter, _stream()), "moe_down")
     out = torch.empty((T, n_out), dtype=x.dtype, device=x.device)
     L.check(getattr(lib, "slb_moe_combine_" + sfx)(
-        y.data_ptr(), y.stride(0), weights.data_ptr(), _p(shared),
+        y.data_ptr(), y.stride(0), _p(out_weights), _p(shared),
         shared.stride(0) if shared is not None else 0, out.data_ptr(), out.stride(0), T, top, n_out,
         _stream()), "moe_combine")
     return out
@@ -1227,18 +1268,16 @@ GATED_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "swish_clamped": 2}
 
 
 def gated_act(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation: str = "silu",
-              limit: Optional[float] = None, alpha: float = 1.0) -> None:
+              limit: Optional[float] = None, alpha: float = 1.0,
+              row_scale: Optional[torch.Tensor] = None) -> None:
     """out[t, i] = act(gate_i) * up_i (layout as ``swiglu``); ``activation`` "silu", "gelu_tanh"
     (0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))) or "swish_clamped": with g = min(gate, limit)
-    and u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1)."""
-    if activation == "swish_clamped":
-        fn = getattr(L.core(), "slb_gated_act_clamped_" + _suffix(out.dtype))
-        L.check(fn(gate_up.data_ptr(), out.data_ptr(), out.shape[0], out.shape[1], gate_up.stride(0),
-                   out.stride(0), int(block), float(limit), float(alpha), _stream()), "gated_act")
-        return
+    and u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1).  ``row_scale`` float32 [T]: a
+    factor a row on gate and up before the activation."""
     fn = getattr(L.core(), "slb_gated_act_" + _suffix(out.dtype))
     L.check(fn(gate_up.data_ptr(), out.data_ptr(), out.shape[0], out.shape[1], gate_up.stride(0),
-               out.stride(0), int(block), GATED_ACTIVATIONS[activation], _stream()), "gated_act")
+               out.stride(0), int(block), GATED_ACTIVATIONS[activation], float(limit or 0.0), float(alpha),
+               _p(row_scale), _stream()), "gated_act")
 
 
 # ------------------------------------------- several residual streams, embedding norm
@@ -1304,6 +1343,57 @@ def group_norm_gate(x: torch.Tensor, groups: int, size: int, out: torch.Tensor, 
     L.check(fn(x.data_ptr(), x.stride(0), maps, _p(lam), _p(weight), float(eps), float(factor), _p(gate),
                gate.stride(0) if gate is not None else 0, GATE_ACTIVATIONS[gate_activation if gate is not None else None],
                out.data_ptr(), out.stride(0), x.shape[0], groups, size, _stream()), "group_norm_gate")
+
+
+def gate_group_norm(x: torch.Tensor, gate: torch.Tensor, groups: int, out: torch.Tensor, *, eps: float,
+                    weight: Optional[torch.Tensor] = None, factor: float = 1.0, gate_activation: str = "silu") -> None:
+    """The gate before the norm: v = x * act(gate), each of ``groups`` equal parts of a row divided by its own
+    root mean square, times ``weight`` (float32, over the row) and ``factor``.  x float32 [T, n]; out [T, n]
+    may be columns of a wider row."""
+    fn = getattr(L.core(), "slb_gate_group_norm_" + _suffix(out.dtype))
+    L.check(fn(x.data_ptr(), x.stride(0), gate.data_ptr(), gate.stride(0), GATE_ACTIVATIONS[gate_activation],
+               _p(weight), float(eps), float(factor), out.data_ptr(), out.stride(0), x.shape[0], groups,
+               x.shape[1] // groups, _stream()), "gate_group_norm")
+
+
+# ----------------------------------------------------- selective state space
+class _StateSpaceArgs(_ct.Structure):
+    _fields_ = [
+        ("u", _ct.c_void_p), ("ld", _ct.c_int),
+        ("x_off", _ct.c_int), ("b_off", _ct.c_int), ("c_off", _ct.c_int),
+        ("H", _ct.c_int), ("P", _ct.c_int), ("N", _ct.c_int), ("G", _ct.c_int),
+        ("dt", _ct.c_void_p), ("ld_dt", _ct.c_int), ("dt_bias", _ct.c_void_p),
+        ("rate", _ct.c_void_p), ("skip", _ct.c_void_p),
+        ("cu_q", _ct.c_void_p), ("state_slots", _ct.c_void_p),
+        ("state", _ct.c_void_p), ("num_slots", _ct.c_int), ("state_stride", _ct.c_longlong),
+        ("out", _ct.c_void_p), ("ldo", _ct.c_int),
+    ]
+
+
+def state_space_max_state() -> int:
+    return L.core().slb_state_space_max_state()
+
+
+def state_space(ctx, u: torch.Tensor, dt: torch.Tensor, state: torch.Tensor, out: torch.Tensor, *, num_heads: int,
+                value_dim: int, state_dim: int, groups: int, dt_bias: torch.Tensor, rate: torch.Tensor,
+                skip: torch.Tensor) -> None:
+    """S_t = exp(-rate_h d_t) S_{t-1} + d_t B_t x_t^T, y_t = S_t^T C_t + skip_h x_t with d_t = softplus(dt + dt_bias),
+    over the tokens of every request of the step in order; ``u`` [T, x: H P | B: G N | C: G N] (head h reads
+    group h // (H / G)); ``dt`` float32 [T, >= H]; ``state`` float32 [slots, >= H N P] (may be a slice of a larger
+    record) is read at ``ctx.state_slots`` and left advanced; ``out`` float32 [T, H P]."""
+    if dt.dtype != _F32 or out.dtype != _F32 or state.dtype != _F32:
+        raise L.KernelError("state_space: step sizes, state and results are float32")
+    a = _StateSpaceArgs()
+    a.u, a.ld = u.data_ptr(), u.stride(0)
+    a.x_off, a.b_off, a.c_off = 0, num_heads * value_dim, num_heads * value_dim + groups * state_dim
+    a.H, a.P, a.N, a.G = num_heads, value_dim, state_dim, groups
+    a.dt, a.ld_dt, a.dt_bias = dt.data_ptr(), dt.stride(0), dt_bias.data_ptr()
+    a.rate, a.skip = rate.data_ptr(), skip.data_ptr()
+    a.cu_q, a.state_slots = ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr()
+    a.state, a.num_slots, a.state_stride = state.data_ptr(), state.shape[0], state.stride(0)
+    a.out, a.ldo = out.data_ptr(), out.stride(0)
+    fn = getattr(L.core(), "slb_state_space_" + _suffix(u.dtype))
+    L.check(fn(_ct.byref(a), ctx.num_seqs, _stream()), "state_space")
 
 
 # ----------------------------------------------- linear attention with a decay

@@ -69,8 +69,10 @@ _CORE_SIGNATURES = {
     "slb_sigmoid_gate_bf16": [P, I, P, I, P, I, I, I, I, P],
     "slb_attention_kv_tile_rows": [],
     "slb_attention_kv_status": [I],
-    "slb_attention_kv_f32": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, I, P, P],
-    "slb_attention_kv_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, I, P, P],
+    "slb_attention_kv_f32": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, I, P, P, F,
+                             P],
+    "slb_attention_kv_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, F, P, I, P, P, F,
+                              P],
     "slb_gemm_simt_batched_f32": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
     "slb_gemm_simt_batched_bf16": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
     "slb_gemm_simt_batched_bf16_f32out": [P, I, P, I, P, I, I, I, I, I, LL, LL, LL, P],
@@ -80,8 +82,8 @@ _CORE_SIGNATURES = {
     "slb_dyt_parallel_bf16": [P, P],
     "slb_stream_rows_f32": [P, P],
     "slb_stream_rows_bf16": [P, P],
-    "slb_short_conv_f32": [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, LL, P, P, P],
-    "slb_short_conv_bf16": [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, LL, P, P, P],
+    "slb_short_conv_f32": [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, LL, P, P, I, P],
+    "slb_short_conv_bf16": [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, LL, P, P, I, P],
     "slb_token_mix_max": [],
     "slb_embed_bigram_f32": [P, P, P, P, P, LL, I, P, I, P, LL, LL, LL, P, P, I, I, I, P],
     "slb_embed_bigram_bf16": [P, P, P, P, P, LL, I, P, I, P, LL, LL, LL, P, P, I, I, I, P],
@@ -100,10 +102,8 @@ _CORE_SIGNATURES = {
     "slb_moe_tile_rows": [],
     "slb_moe_route": [P, I, I, I, I, I, I, F, I, P, P, P],
     "slb_moe_route_scored": [P, I, I, I, I, I, I, F, I, I, P, I, F, P, P, P],
-    "slb_gated_act_f32": [P, P, I, I, I, I, I, I, P],
-    "slb_gated_act_bf16": [P, P, I, I, I, I, I, I, P],
-    "slb_gated_act_clamped_f32": [P, P, I, I, I, I, I, F, F, P],
-    "slb_gated_act_clamped_bf16": [P, P, I, I, I, I, I, F, F, P],
+    "slb_gated_act_f32": [P, P, I, I, I, I, I, I, F, F, P, P],
+    "slb_gated_act_bf16": [P, P, I, I, I, I, I, I, F, F, P, P],
     "slb_rms_norm_rows_f32": [P, I, P, F, P, I, I, I, P],
     "slb_rms_norm_rows_bf16": [P, I, P, F, P, I, I, I, P],
     "slb_norm_sum2_f32": [P, I, P, I, P, P, F, F, P, I, I, I, P],
@@ -111,11 +111,18 @@ _CORE_SIGNATURES = {
     "slb_attention_kv_maps_f32": [P, I, P, I, I, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
     "slb_attention_kv_maps_bf16": [P, I, P, I, I, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
     "slb_hyper_max_streams": [],
+    "slb_state_space_max_state": [],
     "slb_embed_norm_streams_f32": [P, P, P, F, P, I, I, I, I, P],
     "slb_embed_norm_streams_bf16": [P, P, P, F, P, I, I, I, I, P],
     "slb_hyper_mix_norm_f32": [P, P, I, P, P, P, P, F, P, I, P, I, I, I, P],
     "slb_hyper_mix_norm_bf16": [P, P, I, P, P, P, P, F, P, I, P, I, I, I, P],
+    "slb_gate_group_norm_f32": [P, I, P, I, I, P, F, F, P, I, I, I, I, P],
+    "slb_post_add_rmsnorm_f32": [P, P, P, I, LL, P, P, F, P, P, P, I, I, F, P],
+    "slb_state_space_f32": [P, I, P],
     "slb_group_norm_gate_f32": [P, I, I, P, P, F, F, P, I, I, P, I, I, I, I, P],
+    "slb_gate_group_norm_bf16": [P, I, P, I, I, P, F, F, P, I, I, I, I, P],
+    "slb_post_add_rmsnorm_bf16": [P, P, P, I, LL, P, P, F, P, P, P, I, I, F, P],
+    "slb_state_space_bf16": [P, I, P],
     "slb_group_norm_gate_bf16": [P, I, I, P, P, F, F, P, I, I, P, I, I, I, I, P],
     "slb_decay_attention_max_dim": [],
     "slb_decay_attention_f32": [P, I, P],
@@ -131,11 +138,11 @@ _CORE_SIGNATURES = {
     "slb_router_logits_bf16": [P, I, P, I, P, I, I, I, I, P],
     "slb_moe_plan_ints": [I, I],
     "slb_moe_plan": [P, I, I, P, P],
-    "slb_moe_gate_up_f32": [P, I, P, I, P, I, P, I, I, I, I, I, P],
-    "slb_moe_gate_up_bf16": [P, I, P, I, P, I, P, I, I, I, I, I, P],
+    "slb_moe_gate_up_f32": [P, I, P, I, P, I, P, I, I, I, I, I, I, F, F, P, P],
+    "slb_moe_gate_up_bf16": [P, I, P, I, P, I, P, I, I, I, I, I, I, F, F, P, P],
     "slb_moe_down_f32": [P, I, P, I, P, I, P, I, I, I, I, I, P],
     "slb_moe_down_bf16": [P, I, P, I, P, I, P, I, I, I, I, I, P],
-    "slb_moe_gate_up_mma_bf16": [P, I, P, I, P, I, P, I, I, I, I, I, P],
+    "slb_moe_gate_up_mma_bf16": [P, I, P, I, P, I, P, I, I, I, I, I, I, F, F, P, P],
     "slb_moe_down_mma_bf16": [P, I, P, I, P, I, P, I, I, I, I, I, P],
     "slb_moe_combine_f32": [P, I, P, P, I, P, I, I, I, I, P],
     "slb_moe_combine_bf16": [P, I, P, P, I, P, I, I, I, I, P],
@@ -292,7 +299,7 @@ _ATTN_KV_SIGNATURES = {
     "slb_attention_kv_mma_status": [I],
     "slb_attention_kv_mma_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, I, P, P, I, P],
     "slb_attention_kv_mma_capped_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, I, P, P, I,
-                                         F, P, I, P, P],
+                                         F, P, I, P, P, F, P],
     "slb_attention_kv_mma_max_splits": [],
     "slb_attention_kv_mma_resident": [I, I],
     "slb_attention_kv_mma_maps_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, I, P, P, I, P],
@@ -303,7 +310,7 @@ _ATTN_KV_SIGNATURES = {
     "slb_attention_kv_tc_where": [P],
     "slb_attention_kv_tc_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, P],
     "slb_attention_kv_tc_capped_bf16": [P, I, P, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, F, P, I, P,
-                                        P],
+                                        P, F, P],
     "slb_attention_kv_tc_maps_bf16": [P, I, P, P, P, I, P, I, P, P, P, P, I, I, I, I, I, I, F, I, P],
 }
 

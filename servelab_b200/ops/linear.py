@@ -166,8 +166,10 @@ def which_kernel(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None) ->
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
-           out_dtype: Optional[torch.dtype] = None, consumer: Optional[str] = None):
-    """``consumer`` ("rope" or "norm"): the caller hands the result to a kernel of that
+           out_dtype: Optional[torch.dtype] = None, consumer: Optional[str] = None,
+           bias_cast: Optional[torch.Tensor] = None):
+    """``bias_cast``: the bias in the compute type, which the library's product adds (None: converted
+    here, a launch).  ``consumer`` ("rope" or "norm"): the caller hands the result to a kernel of that
     kind, which accepts an unfinished form: a ``SplitSum`` (partial sums of a K-split
     product) or, for "norm", a ``DeferredLinear`` (the product not launched yet: the norm
     launches it with itself in the epilogue).  The caller may then get one instead of a
@@ -196,11 +198,23 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         if bias is not None:
             out += bias
     elif bias is not None:
-        out = torch.addmm(bias.to(x.dtype), x, w.t())
+        out = torch.addmm(bias.to(x.dtype) if bias_cast is None else bias_cast, x, w.t())
     else:
         out = torch.mm(x, w.t())
     _mark("library gemm")
     return out
+
+
+narrow_logits_max_tokens = 512     # from here on the library's product
+
+
+def narrow_logits(x: torch.Tensor, w: torch.Tensor, w_f32: torch.Tensor) -> torch.Tensor:
+    """float32 x W^T for a matrix of few rows: [T, >= rows].  ``w`` in the compute type with its rows padded to
+    a multiple of 8, ``w_f32`` float32 [rows, hidden].  Steps of few tokens: one launch of this package's
+    kernel for narrow matrices (a product of wide tiles would split K and reduce)."""
+    if x.dtype == torch.float32 or x.shape[0] >= narrow_logits_max_tokens:
+        return linear(x, w, out_dtype=torch.float32)
+    return K.router_logits(x, w_f32)
 
 
 def batched_head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:

@@ -2,7 +2,7 @@
 
 from . import (attention, block, conv_attention, decay_attention, delta_rule,  # noqa: F401
                differential_attention, feed_forward, gated_recurrence, latent_attention, norm, normed_attention, parallel_mixers, position,
-               routed_experts)                                                  # (registration)
+               routed_experts, state_space)                                     # (registration)
 from .base import (Block, BuildEnv, FeedForward, LayerCache, Mixer, Norm, Part,
                    PositionEncoding)
 from .registry import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, build_part, part_class,

@@ -36,6 +36,12 @@ update handed from one part to the next may be unfinished (``ops.kernels.SplitSu
 float32 partial sums of a K-split product, which the consuming kernel adds itself).  A part
 says that it takes the form with the class attribute ``accepts_split_sum``; a part that does
 not set it always gets plain tensors.
+
+A mixer with ``splits_projections = True`` lets a mixer around it merge its products with those of
+another: after ``load`` it holds ``w_in`` (the matrix of its first product, [a multiple of 8, hidden]),
+``w_o`` and ``o_bias`` (None: none) of its last one, and ``core(ctx, x, proj, cache, owns_cache, out,
+factor)`` turns the first product's rows ``proj`` (columns of a wider row) into ``factor`` times the rows
+that the last product reads, written to ``out`` [T, out_width] (columns of a wider row too).
 """
 
 from __future__ import annotations

@@ -23,6 +23,8 @@ class RMSNorm(Norm):
                                       # add and this norm in its epilogue; the result is ScaledRows
 
     accepts_hyper_pending = True      # ... or the update of a residual kept as several streams
+    accepts_post_normed = True        # ... or a result whose own norm is still to come: if that is an RMS
+                                      # norm too, both norms and the add are one launch
 
     @classmethod
     def declare(cls, spec, prefix):
@@ -33,6 +35,8 @@ class RMSNorm(Norm):
         self.weight = store.get(self.prefix + self.spec.weight_suffix)
         if self.spec.unit_offset:             # the stored weight lies around zero: the factor is 1 + w
             self.weight = (self.weight.to(torch.float32) + 1.0).contiguous()
+        if self.spec.factor != 1.0:
+            self.weight = (self.weight.to(torch.float32) * self.spec.factor).contiguous()
 
     def read_streams(self, ctx, streams, pending, read_weights, out_rows=None):
         """For a residual kept as streams [T, n, dim]: folds the pending update in (``HyperPending``
@@ -49,6 +53,15 @@ class RMSNorm(Norm):
     def forward(self, ctx, resid, delta, out_rows=None):
         if resid.dim() == 3:              # several streams: their sum is what a model's last norm reads
             return self.read_streams(ctx, resid, delta, None, out_rows)
+        if isinstance(delta, PostNormed):
+            if isinstance(delta.norm, RMSNorm):
+                value = delta.value.materialize() if isinstance(delta.value, K.DeferredLinear) else delta.value
+                rows = resid.shape[0] if out_rows is None else out_rows.numel()
+                out = torch.empty((rows, self.spec.dim), dtype=self.env.dtype, device=resid.device)
+                K.post_add_rmsnorm(resid, value, delta.norm.weight, delta.norm.spec.eps, self.weight, self.spec.eps,
+                                   out, out_rows)
+                return out
+            delta = delta.materialize()
         if isinstance(delta, K.DeferredLinear):
             if out_rows is None and self.env.dtype == torch.bfloat16:
                 return K.gemm_tc_resid_norm(delta.x, delta.w, delta.bias, resid, self.weight,

@@ -3,18 +3,19 @@ different sizes, values mixed across layers and a gate per head (spec: ``NormedA
 
 Per step, with h the mixer's input [T, hidden]:
 
-  1. one product for q | k | v | gate (their matrices are concatenated at load);
+  1. one product for q | k | v | gate (their matrices are concatenated at load; biases are added by the
+     head kernel);
   1b. with ``conv_taps``: a causal convolution over time on every q, k and v channel; the rows
      before a portion come from the request's state record, which is left holding the last
      taps - 1 projected rows;
   2. one kernel: RMS norm of every query and key head (one weight vector each, shared by the
-     heads), rotation on the first ``dims`` elements (neighbouring pairs, or element i with
+     heads; or with ``qk_row_norm`` of all heads of a row together), rotation on the first ``dims`` elements (neighbouring pairs, or element i with
      element i + dims / 2), with ``qk_unit_norm`` every rotated head divided by its root mean
      square, q into its buffer, k into the request's pages; the values -- kept for later layers
      ("source") or replaced by (1 - lambda) v + lambda v_source ("mix") -- into the pages, so the
      cache holds what the attention uses;
   3. attention of every query over its request's visible keys, softmax in float32 (scores
-     soft-capped, a sink a head in the denominator: each optional), head h's row times
+     soft-capped, a distance bias, a sink a head in the denominator: each optional), head h's row times
      sigmoid(gate_h); or, with ``weight_fn`` "sigmoid", weights sigmoid(score + a number a head) that
      are not normalized; visible keys: all earlier ones, a window, or the query's own chunk;
   4. the output projection (``out_dtype``: a mixer that norms the result asks for float32).
@@ -50,6 +51,7 @@ def pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
 @register_mixer("normed_attention")
 class NormedAttention(Mixer):
     graph_safe = True
+    splits_projections = True
     padded_steps_safe = True      # the convolution's record is written per request with tokens only
 
     def __init__(self, spec, prefix, env):
@@ -70,16 +72,29 @@ class NormedAttention(Mixer):
             raise ValueError("normed_attention: a number a head on the scores needs sigmoid weights")
         if spec.chunk is not None and (spec.window is not None or spec.chunk < 1):
             raise ValueError("normed_attention: a chunk is at least 1 and goes without a window")
+        if spec.qk_row_norm and (spec.qk_norm or spec.conv_taps):
+            raise ValueError("normed_attention: a norm over the rows goes without one over the heads or a convolution")
+        if spec.qkv_bias and spec.conv_taps:
+            raise ValueError("normed_attention: biases together with a convolution are not built")
+        if spec.distance_slopes and len(spec.distance_slopes) != spec.num_heads:
+            raise ValueError("normed_attention: a slope for every head")
+        if spec.sink_score is not None and (spec.sink or spec.weight_fn != "softmax"):
+            raise ValueError("normed_attention: a constant sink goes without learned ones, in a softmax")
         self.position = build_part(POSITIONS, spec.position, f"{prefix}.rot", env)
         self.out_dtype = None                  # (set by a mixer that wraps this one)
         self.scale = spec.scale if spec.scale is not None else 1.0 / math.sqrt(spec.head_dim)
         self.q_size = spec.num_heads * spec.head_dim
         self.k_size = spec.num_kv_heads * spec.head_dim
         self.v_size = spec.num_kv_heads * spec.value_dim
+        self.out_width = spec.num_heads * spec.value_dim
+        self.slopes = None
+        if spec.distance_slopes:
+            self.slopes = torch.tensor(list(spec.distance_slopes), dtype=torch.float64).to(torch.float32).to(env.device)
         A.check_kv_supported(spec.head_dim, spec.value_dim)
         A.prepare_kv_attention(spec.head_dim, spec.value_dim, env.dtype)
         if (spec.head_dim == spec.value_dim and env.dtype == torch.bfloat16 and spec.head_dim in (64, 128)
-                and spec.softcap is None and not spec.sink and spec.weight_fn == "softmax" and spec.chunk is None
+                and spec.softcap is None and not spec.sink and spec.sink_score is None
+                and not spec.distance_slopes and spec.weight_fn == "softmax" and spec.chunk is None
                 and torch.cuda.is_available()):
             from ..ops import library
             library.attention(spec.head_dim)      # the kernels for equal sizes, built now
@@ -97,6 +112,13 @@ class NormedAttention(Mixer):
                TensorDecl(n["v"], (G * Dv, h), MATRIX), TensorDecl(n["o"], (h, H * Dv), MATRIX)]
         if spec.qk_norm:
             out += [TensorDecl(n["q_norm"], (D,), NORM), TensorDecl(n["k_norm"], (D,), NORM)]
+        if spec.qk_row_norm:
+            out += [TensorDecl(n["q_norm"], (H * D,), NORM), TensorDecl(n["k_norm"], (G * D,), NORM)]
+        if spec.qkv_bias:
+            out += [TensorDecl(n[x] + spec.bias_suffix, (rows,), BIAS)
+                    for x, rows in (("q", H * D), ("k", G * D), ("v", G * Dv))]
+        if spec.out_bias:
+            out.append(TensorDecl(n["o"] + spec.bias_suffix, (h,), BIAS))
         if spec.value_mix == "mix":
             out.append(TensorDecl(n["value_mix"], (), POSITIVE))
         if spec.head_gate:
@@ -124,8 +146,11 @@ class NormedAttention(Mixer):
         n = self._names(s, self.prefix)
         self.w_in = pad_rows(store.cat([n["q"], n["k"], n["v"]] + ([n["gate"]] if s.head_gate else [])))
         self.w_o = store.get(n["o"])
-        self.q_norm = store.get(n["q_norm"]) if s.qk_norm else None
-        self.k_norm = store.get(n["k_norm"]) if s.qk_norm else None
+        self.q_norm = store.get(n["q_norm"]) if s.qk_norm or s.qk_row_norm else None
+        self.k_norm = store.get(n["k_norm"]) if s.qk_norm or s.qk_row_norm else None
+        self.biases = [store.get(n[x] + s.bias_suffix) if s.qkv_bias else None for x in ("q", "k", "v")]
+        self.o_bias = store.get(n["o"] + s.bias_suffix) if s.out_bias else None
+        self.o_bias_cast = self.o_bias.to(self.env.dtype) if s.out_bias else None
         self.lam = store.get(n["value_mix"]).reshape(1) if s.value_mix == "mix" else None
         self.taps = None
         if s.conv_taps >= 1:
@@ -136,12 +161,21 @@ class NormedAttention(Mixer):
             self.sigmoid_bias = (store.get(f"{self.prefix}.{s.score_bias_name}") if s.score_bias
                                  else torch.zeros(s.num_heads, dtype=torch.float32, device=self.env.device))
         self.sink = store.get(f"{self.prefix}.{s.sink_name}").to(torch.float32).contiguous() if s.sink else None
+        if s.sink_score is not None:
+            self.sink = torch.full((s.num_heads,), float(s.sink_score), dtype=torch.float32, device=self.env.device)
 
     def forward(self, ctx, x, cache, owns_cache):
+        proj = K.plain_unless(None, linear(x, self.w_in))             # [T, q | k | v | gate]
+        out = torch.empty((x.shape[0], self.out_width), dtype=x.dtype, device=x.device)
+        self.core(ctx, x, proj, cache, owns_cache, out)
+        if self.out_dtype is not None:
+            return linear(out, self.w_o, self.o_bias, out_dtype=self.out_dtype)
+        return linear(out, self.w_o, self.o_bias, consumer="norm", bias_cast=self.o_bias_cast)
+
+    def core(self, ctx, x, proj, cache, owns_cache, out, factor=1.0):
         s = self.spec
         T = x.shape[0]
         table = ctx.block_tables[cache.group]
-        proj = K.plain_unless(None, linear(x, self.w_in))             # [T, q | k | v | gate]
         gate = proj[:, self.q_size + self.k_size + self.v_size:] if s.head_gate else None
         if self.taps is not None:
             if not owns_cache:
@@ -176,11 +210,8 @@ class NormedAttention(Mixer):
                     freq=freq, rot_dims=rot_dims, rot_mag=mag, eps=s.qk_norm_eps, q_out=q,
                     k_cache=cache.k if owns_cache else None, v_cache=cache.v if owns_cache else None,
                     lam=self.lam, v_first=v_first, v_keep=v_keep, rot_half=halves,
-                    q_unit_dims=unit_dims, k_unit_dims=unit_dims)
-        out = torch.empty((T, s.num_heads * s.value_dim), dtype=x.dtype, device=x.device)
+                    q_unit_dims=unit_dims, k_unit_dims=unit_dims, q_bias=self.biases[0], k_bias=self.biases[1],
+                    v_bias=self.biases[2], row_norm=s.qk_row_norm)
         A.kv_attention(ctx, q, cache.k, cache.v, s.value_dim, out, table, s.num_heads, s.num_kv_heads,
                        s.head_dim, s.value_dim, cache.page_size, self.scale, s.window or 0, gate,
-                       s.softcap, self.sink, s.chunk or 0, self.sigmoid_bias)
-        if self.out_dtype is not None:
-            return linear(out, self.w_o, out_dtype=self.out_dtype)
-        return linear(out, self.w_o, consumer="norm")
+                       s.softcap, self.sink, s.chunk or 0, self.sigmoid_bias, self.slopes, factor)

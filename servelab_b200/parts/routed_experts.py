@@ -1,4 +1,4 @@
-"""Routed experts with a softmax router, group-limited choice and an optional shared expert
+"""Routed experts with a softmax or sigmoid router, group-limited choice and an optional shared expert
 (spec: ``RoutedExpertsSpec``).
 
 Per step: the router's logits in float32 (a float32 matrix against the step's rows), one kernel
@@ -30,6 +30,10 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: top experts must fit into the kept groups")
         if spec.score_fn not in ("softmax", "sigmoid") or spec.group_best < 1:
             raise ValueError("routed_experts: score_fn is 'softmax' or 'sigmoid'; group_best at least 1")
+        if spec.activation not in K.GATED_ACTIVATIONS:
+            raise ValueError(f"routed_experts: activation {spec.activation!r} ({', '.join(K.GATED_ACTIVATIONS)})")
+        if spec.activation == "swish_clamped" and not (spec.limit is not None and spec.limit > 0):
+            raise ValueError("routed_experts: the clamped activation needs a positive limit")
         self.shared = (build_part(FEED_FORWARDS, spec.shared, f"{prefix}.{spec.shared_name}", env)
                        if spec.shared is not None else None)
 
@@ -73,4 +77,5 @@ class RoutedExperts(FeedForward):
                                               s.renormalize, s.score_fn, self.correction, s.group_best,
                                               s.norm_eps)
         shared = K.plain_unless(None, self.shared.forward(ctx, x)) if self.shared is not None else None
-        return K.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, shared)
+        return K.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, shared, s.activation,
+                             s.limit, s.swish_alpha, s.weight_inputs)
