@@ -504,6 +504,121 @@ def _vufadra_rooflines(size, res, peaks) -> Dict[str, object]:
     return out
 
 
+# Sunutar: four parallel layers -- a windowed attention with a soft cap, a distance bias and the added one beside a
+# selective state space -- each followed by a dense feed-forward or by routed experts.  Beside the dense sizes:
+# Sumolorn with its soft-capped attention in the first layer and its parallel layer (windowed attention beside a
+# linear attention with learned decays, a state of as many numbers) in the others, the same feed-forward.
+# Beside the sizes with experts: Zimupel without streams (linear attention with a fixed decay a head, a state of
+# as many numbers, and differential attention, alternating), the same experts.
+# width, heads, kv heads, head size, feed-forward or expert size, heads / value size / state size / groups of the
+# state space, experts (0: dense), top
+SUNUTAR_SIZES = {
+    "1b-like": (2048, 16, 4, 128, 5632, 32, 64, 128, 4, 0, 0),
+    "small-1024": (1024, 8, 2, 64, 2816, 16, 64, 64, 2, 0, 0),
+    "moe-2048": (2048, 16, 4, 128, 1408, 32, 64, 128, 4, 32, 4),
+    "moe-1024": (1024, 8, 2, 64, 512, 8, 64, 64, 2, 16, 2),
+}
+
+
+def sunutar_config(width, heads, kv, dim, ff, rh, rp, rn, rg, experts, top, layers=LAYERS) -> dict:
+    mlp = ({"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top}} if experts
+           else {"kind": "dense", "ff": ff, "limit": 7.0})
+    left = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+            "mask": {"size": WINDOW}}
+    right = {"heads": rh, "vdim": rp, "state": rn, "groups": rg, "conv": 4, "norm_groups": rg}
+    mixer = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.6}
+    return {"architecture": "Sunutar", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.9,
+            "layers": [{"type": "parallel", "mixer": mixer, "mlp": mlp} for _ in range(layers)]}
+
+
+def sumolorn_like_sunutar(width, heads, kv, dim, ff, rh, rp, rn, rg, experts, top, layers=LAYERS) -> dict:
+    # (a state of rh * rn * rp numbers as heads of dim x dim)
+    return sumolorn_like_vufadra(width, heads, kv, dim, ff, rh * rn * rp // (dim * dim), 64, layers)
+
+
+def zimupel_like_sunutar(width, heads, kv, dim, ff, rh, rp, rn, rg, experts, top, layers=LAYERS) -> dict:
+    cfg = zimupel_config(width, heads, kv, dim, experts, 1, 1, top, ff, 1, layers)
+    cfg.pop("streams")
+    return cfg
+
+
+def _sunutar_rooflines(size, res, peaks) -> Dict[str, object]:
+    """Microseconds a layer and achieved fractions of the measured peaks for the kernels of the Sunutar layers
+    beside their counterparts, from the eager profiles.  Attention, prefill: 2 (Dk + Dv) flops per visible
+    pair and head of the bf16 peak; decode: the cached rows the requests may see of the copy bandwidth.
+    Recurrences, prefill: 4 flops a state element and token (decay, update, output) of the bf16 peak; decode:
+    the state read and written once.  Experts, prefill: 6 T top width size flops; decode: the weights that
+    the step's pairs can touch.  Elementwise kernels: the bytes they must move."""
+    width, heads, kv, dim, ff, rh, rp, rn, rg, experts, top = SUNUTAR_SIZES[size]
+    other = "zimupel" if experts else "sumolorn"
+    up, op = (res[a]["prefill_kernels_us"] for a in ("sunutar", other))
+    out: Dict[str, object] = {}
+
+    def hbm(nbytes, us):
+        return round(nbytes / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 4)
+
+    def tf(flops, us):
+        return round(flops / (us * 1e-6) / 1e12 / peaks["bf16_tflops"], 4)
+
+    def row(name, table, key, layers, frac):
+        us = sum(table.get(k) or 0 for k in ((key,) if isinstance(key, str) else key))
+        if us:
+            out[name] = {"us": round(us / layers, 2), "frac": frac(us / layers)}
+    state, inner = rh * rn * rp, rh * rp
+    chans = inner + 2 * rg * rn
+    win_pairs = sum(min(t + 1, WINDOW) for t in range(PROMPT))
+    full_pairs = PROMPT * (PROMPT + 1) / 2
+    kvk = ("attention_kv_tc", "attention_kv_mma", "attention_kv")
+    plain = ("prefill_attention_tc", "prefill_attention")
+    lin = ("decay_attention (gated chunks)", "decay_attention (chunked)", "decay_attention")
+    n_lin = 2 if experts else 3                       # layers of the other model with a recurrence
+    row("sunutar_attention_prefill", up, kvk, LAYERS, lambda us: tf(win_pairs * heads * 4 * dim, us))
+    row("sunutar_state_space_prefill", up, ("state_space (chunks)", "state_space"), LAYERS,
+        lambda us: tf(4.0 * PROMPT * state, us))
+    row(f"{other}_decay_prefill", op, lin, n_lin, lambda us: tf(4.0 * PROMPT * state, us))
+    if experts:
+        row("zimupel_differential_prefill", op, kvk + plain, 2,
+            lambda us: tf(full_pairs * (heads // 2) * 2 * 2 * (dim + 2 * dim), us))
+    else:
+        row("sumolorn_capped_attention_prefill", op, kvk, 1, lambda us: tf(win_pairs * heads * 4 * dim, us))
+        row("sumolorn_plain_attention_prefill", op, plain, 3, lambda us: tf(win_pairs * heads * 4 * dim, us))
+        row("sumolorn_conv_prefill", op, "short_conv", 3, lambda us: hbm(PROMPT * (heads + 2 * kv) * dim * 4, us))
+    row("sunutar_conv_prefill", up, "short_conv", LAYERS, lambda us: hbm(PROMPT * chans * 4, us))
+    row("sunutar_norm_prefill", up, "post_add_rmsnorm", 2 * LAYERS, lambda us: hbm(PROMPT * width * 12, us))
+    row(f"{other}_norm_prefill", op, "add_rmsnorm", 2 * LAYERS, lambda us: hbm(PROMPT * width * 12, us))
+    row("sunutar_head_prep_prefill", up, "head_prep", LAYERS, lambda us: hbm(PROMPT * 4 * (heads + 2 * kv) * dim, us))
+    # (Zimupel: two layers, of which one writes no keys and values)
+    row(f"{other}_head_prep_prefill", op, "head_prep", 2 if experts else LAYERS,
+        lambda us: hbm(PROMPT * 4 * (heads + (1.5 if experts else 2) * kv) * dim, us))
+    row("sunutar_gated_norm_prefill", up, "gate_group_norm", LAYERS, lambda us: hbm(PROMPT * inner * 8, us))
+    row(f"{other}_norm_gate_prefill", op, "group_norm_gate", 4 if experts else 3,
+        lambda us: hbm(PROMPT * heads * dim * (9 if experts else 8), us))
+    for name, share in (("moe_gate_up", 2.0 / 3.0), ("moe_down", 1.0 / 3.0)):
+        for arch, table in (("sunutar", up), (other, op)):
+            row(f"{arch}_{name}_prefill", table, name, LAYERS, lambda us: tf(share * 6.0 * PROMPT * top * width * ff, us))
+    for arch, table in (("sunutar", up), (other, op)):
+        row(f"{arch}_activation_prefill", table, ("gated_act", "swiglu"), LAYERS,
+            lambda us: hbm(PROMPT * (ff * max(top, 1)) * 6, us))
+        row(f"{arch}_moe_combine_prefill", table, "moe_combine", LAYERS, lambda us: hbm(PROMPT * width * (4 * top + 2), us))
+    for b in (8, 64):
+        ud, od = (res[a][f"decode_b{b}_kernels_us"] for a in ("sunutar", other))
+        dec = ("attention_kv_mma", "attention_kv", "decode_attention")
+        seen = min(CONTEXT, WINDOW)
+        row(f"sunutar_attention_decode_b{b}", ud, dec, LAYERS, lambda us: hbm(b * seen * kv * 4 * dim, us))
+        if experts:
+            row(f"zimupel_differential_decode_b{b}", od, dec, 2, lambda us: hbm(b * CONTEXT * max(1, kv // 2) * 8 * dim, us))
+        else:
+            row(f"sumolorn_capped_attention_decode_b{b}", od, dec[:2], 1, lambda us: hbm(b * seen * kv * 4 * dim, us))
+            row(f"sumolorn_plain_attention_decode_b{b}", od, dec[2:], 3, lambda us: hbm(b * seen * kv * 4 * dim, us))
+        row(f"sunutar_state_space_decode_b{b}", ud, "state_space", LAYERS, lambda us: hbm(b * state * 8, us))
+        row(f"{other}_decay_decode_b{b}", od, "decay_attention", n_lin, lambda us: hbm(b * state * 8, us))
+        for name, share in (("moe_gate_up", 2.0 / 3.0), ("moe_down", 1.0 / 3.0)):
+            for arch, table in (("sunutar", ud), (other, od)):
+                row(f"{arch}_{name}_decode_b{b}", table, name, LAYERS,
+                    lambda us: hbm(share * min(experts, b * top) * 3 * width * ff * 2, us))
+    return out
+
+
 def _measure(cfg: dict, note, graph_prefill: bool = False, queue_ahead: bool = False) -> Dict[str, object]:
     """``graph_prefill``: the prompt's step replays the graph captured for its padded sizes where the
     model allows it (the eager step of a small model is bound by the host's launches); the eager
@@ -645,6 +760,24 @@ def _kernel_rooflines(size, res: Dict[str, Dict[str, object]], peaks) -> Dict[st
 
 
 def run(peaks, note=lambda m: None, sizes=None, design: str = "dezelorn") -> Dict[str, object]:
+    if design == "sunutar":
+        result = {"compare": "sunutar vs sumolorn (dense feed-forward) and vs zimupel without streams (experts) at equal "
+                             "layer sizes", "layers": LAYERS, "prompt": PROMPT, "decode_context": CONTEXT,
+                  "window": WINDOW, "vocab": VOCAB, "dtype": "bf16",
+                  "data": "synthetic: random weights, token ids uniform over the vocabulary",
+                  "peaks": peaks.get("source"), "sizes": {}}
+        for size in (sizes or SUNUTAR_SIZES):
+            dims = SUNUTAR_SIZES[size]
+            res = {}
+            beside = ("zimupel", zimupel_like_sunutar) if dims[9] else ("sumolorn", sumolorn_like_sunutar)
+            for arch, make in (("sunutar", sunutar_config), beside):
+                note(f"{size}: {arch}")
+                res[arch] = _measure(make(*dims), note, graph_prefill=True, queue_ahead=True)
+            res["kernels"] = _sunutar_rooflines(size, res, peaks)
+            res["dims"] = dict(zip(("width", "heads", "kv_heads", "head_dim", "ff", "state_heads", "state_values",
+                                    "state_size", "groups", "experts", "top"), dims))
+            result["sizes"][size] = res
+        return result
     if design == "vufadra":
         result = {"compare": "vufadra vs sumolorn (attention, and parallel layers with a linear branch of the same "
                              "sizes) at equal layer sizes", "layers": LAYERS, "prompt": PROMPT,

@@ -35,7 +35,8 @@ CORE_SOURCES = ["elementwise.cu", "rope_cache.cu", "attention_generic.cu", "gemm
                 "sampling.cu", "gemm_tcgen05.cu", "dynamic_tanh.cu", "short_conv.cu", "layernorm.cu",
                 "head_prep.cu", "attention_kv.cu", "moe.cu", "hyper.cu", "decay_attention.cu", "decay_attention_mma.cu",
                 "decay_gated_chunk.cu", "token_mix.cu", "delta_rule.cu", "delta_rule_chunk.cu",
-                "gated_recurrence.cu", "bottleneck.cu", "state_space.cu"]
+                "gated_recurrence.cu", "bottleneck.cu", "state_space.cu",
+                "state_space_chunk.cu"]
 HEADERS = ["common.cuh", "no_alloc.h", "mma_util.cuh", "tma_util.cuh", "decay_attention.cuh",
            "delta_rule.cuh", "gated_act.cuh", "state_space.cuh"]
 

@@ -1370,6 +1370,17 @@ class _StateSpaceArgs(_ct.Structure):
     ]
 
 
+class _StateSpaceChunkArgs(_ct.Structure):
+    _fields_ = [("a", _StateSpaceArgs), ("tile_seq", _ct.c_void_p), ("tile_row0", _ct.c_void_p),
+                ("num_tiles", _ct.c_int), ("work", _ct.c_void_p), ("total", _ct.c_void_p)]
+
+
+# bfloat16 steps that bring portions of prompts take the chunked tensor-core kernels from this many tokens a
+# request on (shorter portions, single tokens and float32: token by token)
+state_space_chunked = True
+state_space_chunk_min_tokens = 16
+
+
 def state_space_max_state() -> int:
     return L.core().slb_state_space_max_state()
 
@@ -1392,6 +1403,18 @@ def state_space(ctx, u: torch.Tensor, dt: torch.Tensor, state: torch.Tensor, out
     a.cu_q, a.state_slots = ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr()
     a.state, a.num_slots, a.state_stride = state.data_ptr(), state.shape[0], state.stride(0)
     a.out, a.ldo = out.data_ptr(), out.stride(0)
+    if (state_space_chunked and u.dtype == _BF16 and not ctx.decode_only
+            and ctx.num_tokens >= state_space_chunk_min_tokens * ctx.num_seqs):
+        c = _StateSpaceChunkArgs()
+        tile_seq, tile_row0, n = ctx.attention_tiles(1, L.core().slb_state_space_chunk_tokens())
+        work = torch.empty((max(n, 1), num_heads, state_dim, value_dim), dtype=_F32, device=u.device)
+        total = torch.empty((max(n, 1), num_heads), dtype=_F32, device=u.device)
+        c.a, c.tile_seq, c.tile_row0, c.num_tiles = a, tile_seq.data_ptr(), tile_row0.data_ptr(), n
+        c.work, c.total = work.data_ptr(), total.data_ptr()
+        L.check(L.core().slb_state_space_chunk_bf16(_ct.byref(c), ctx.num_seqs, _stream()), "state_space (chunks)")
+        global launch_count
+        launch_count += 2
+        return
     fn = getattr(L.core(), "slb_state_space_" + _suffix(u.dtype))
     L.check(fn(_ct.byref(a), ctx.num_seqs, _stream()), "state_space")
 

@@ -112,6 +112,8 @@ _CORE_SIGNATURES = {
     "slb_attention_kv_maps_bf16": [P, I, P, I, I, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
     "slb_hyper_max_streams": [],
     "slb_state_space_max_state": [],
+    "slb_state_space_chunk_tokens": [],
+    "slb_state_space_chunk_bf16": [P, I, P],
     "slb_embed_norm_streams_f32": [P, P, P, F, P, I, I, I, I, P],
     "slb_embed_norm_streams_bf16": [P, P, P, F, P, I, I, I, I, P],
     "slb_hyper_mix_norm_f32": [P, P, I, P, P, P, P, F, P, I, P, I, I, I, P],
