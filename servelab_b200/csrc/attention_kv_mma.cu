@@ -23,6 +23,11 @@
 // long product of a tile is spread over the warps; the Q tile takes 16 rows of shared memory, so
 // that two blocks fit an SM at the largest sizes.
 //
+// Key sizes up to 192 have a kernel of their own for those steps (attention_kv_rows_kernel): a warp takes 16
+// of every 64 keys through a ring of its own and holds all value columns, so that neither the scores nor
+// the loads of a key are repeated and the warps do not wait for one another until they merge their rows at the
+// end.
+//
 // Instead of the softmax (`sig_bias`, one number a head): a visible key's weight is sigmoid(score +
 // sig_bias_h), the weights are not normalized, and key splits simply add up.  Instead of the window
 // (`chunk` > 0): a query at position i sees the keys j <= i with j / chunk == i / chunk.
@@ -397,6 +402,264 @@ __global__ void __launch_bounds__(NTHREADS) attention_kv_mma_kernel(
     }
 }
 
+// ---- steps of single tokens, at most 16 query heads a kv head: a warp a quarter of the keys ----
+constexpr int WK = 16;                                     // keys of a 64-key tile a warp takes
+constexpr size_t rows_ring_bytes(int stages, bool tied) {
+    return (size_t)4 * stages * WK * (tied ? LDK : LDK + LDV) * sizeof(bf16);
+}
+constexpr int ROW_STAGES = rows_ring_bytes(3, false) <= 112 * 1024 ? 3 : 2;
+constexpr size_t rows_smem(int q_rows, bool tied) { return (size_t)q_rows * LDK * sizeof(bf16) + rows_ring_bytes(ROW_STAGES, tied); }
+constexpr bool ROWS_FORM = DK <= 192;
+// (the warps' rows meet in the ring's memory at the end)
+static_assert(!ROWS_FORM || rows_ring_bytes(ROW_STAGES, true) >= (size_t)4 * 16 * (DV + 2) * sizeof(float) || DV > DK,
+              "the ring holds the four warps' rows");
+
+__global__ void __launch_bounds__(NTHREADS) attention_kv_rows_kernel(
+    const bf16* __restrict__ q, int ldq, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
+    int tied, bf16* __restrict__ out, int ldo, const int* __restrict__ block_table, int max_pages,
+    const int* __restrict__ cu_q, const int* __restrict__ ctx_len, const int* __restrict__ tile_seq,
+    int H, int Hkv, int ps, int num_pages, float scale_log2, int window, const bf16* __restrict__ gate, int ldg,
+    int splits, float* __restrict__ part_o, float* __restrict__ part_ml, int q_rows, float softcap, float scale,
+    const float* __restrict__ sink, int chunk, const float* __restrict__ sig_bias, const float* __restrict__ slopes,
+    float out_scale) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, tig = lane & 3;
+    const int kvh = blockIdx.x % Hkv, tile = blockIdx.x / Hkv;
+    const int s = tile_seq[tile];
+    const int g = H / Hkv;
+    const int q0 = cu_q[s];
+    if (cu_q[s + 1] - q0 <= 0) return;                     // (one token a request)
+    const int pos = ctx_len[s] - 1, kend = pos + 1;
+    const int* table = block_table + (size_t)s * max_pages;
+    bf16* Qs = reinterpret_cast<bf16*>(smem_raw);          // [q_rows][LDK]
+    const int stage_elems_w = WK * (tied ? LDK : LDK + LDV);
+    bf16* ring = Qs + q_rows * LDK + (size_t)warp * ROW_STAGES * stage_elems_w;
+
+    for (int idx = tid; idx < q_rows * KCH; idx += NTHREADS) {
+        const int r = idx / KCH, c = idx - r * KCH;
+        const bool ok = r < g;
+        cp_async16(Qs + r * LDK + c * 8, q + (size_t)q0 * ldq + (size_t)(kvh * g + (ok ? r : 0)) * DK + c * 8, ok);
+    }
+    cp_async_commit();
+
+    const int first = window > 0 ? max(0, pos - window + 1) : chunk > 0 ? pos - pos % chunk : 0;
+    int kbeg = first / 64 * 64;
+    int ntiles = (kend - kbeg + 63) / 64;
+    if (splits > 1) {                                      // this block's share of the key tiles
+        const int per = (ntiles + splits - 1) / splits;
+        const int t0 = min(ntiles, (int)blockIdx.y * per);
+        ntiles = min(ntiles, t0 + per) - t0;
+        kbeg += t0 * 64;
+    }
+    kbeg += warp * WK;                                     // the warp's keys of a tile
+    auto load = [&](int t) {
+        if (t < ntiles) {
+            bf16* Ks = ring + (t % ROW_STAGES) * stage_elems_w;
+            bf16* Vs = Ks + WK * LDK;
+            const int kp = kbeg + t * 64 + (lane & 15);
+            int slot = -1;                                 // lane r (and r + 16): where key r lies
+            if (kp >= first && kp < kend) {
+                const int page = table[kp / ps];
+                if (page >= num_pages) atomicCAS(&kv_attn_status_word, 0, 0x40);
+                else if (page >= 0) slot = (page * Hkv + kvh) * ps + kp % ps;
+            }
+#pragma unroll
+            for (int i = 0; i < KCH / 2; ++i) {
+                const int idx = i * 32 + lane, r = idx / KCH, c = idx - r * KCH;
+                const int sl = __shfl_sync(0xffffffffu, slot, r);
+                cp_async16(Ks + r * LDK + c * 8, kc + (size_t)max(sl, 0) * DK + c * 8, sl >= 0);
+            }
+            if (!tied) {
+#pragma unroll
+                for (int i = 0; i < VCH / 2; ++i) {
+                    const int idx = i * 32 + lane, r = idx / VCH, c = idx - r * VCH;
+                    const int sl = __shfl_sync(0xffffffffu, slot, r);
+                    cp_async16(Vs + r * LDV + c * 8, vc + (size_t)max(sl, 0) * DV + c * 8, sl >= 0);
+                }
+            }
+        }
+        cp_async_commit();                                 // (empty groups keep the count)
+    };
+#pragma unroll
+    for (int t = 0; t < ROW_STAGES - 1; ++t) load(t);
+    cp_async_wait<ROW_STAGES - 1>();                       // this thread's part of Q
+    __syncthreads();
+
+    const bool two = q_rows > 8;                           // rows 8..15 exist
+    const int r_lo = lane >> 2, r_hi = r_lo + 8;
+    float bias2[2] = {0.f, 0.f}, slope[2] = {0.f, 0.f};
+    if (sig_bias != nullptr) {
+        if (r_lo < g) bias2[0] = sig_bias[kvh * g + r_lo] * 1.4426950408889634f;
+        if (r_hi < g) bias2[1] = sig_bias[kvh * g + r_hi] * 1.4426950408889634f;
+    }
+    if (slopes != nullptr) {                               // (scores are multiplied by scale * log2 e below)
+        if (r_lo < g) slope[0] = slopes[kvh * g + r_lo] / scale;
+        if (r_hi < g) slope[1] = slopes[kvh * g + r_hi] / scale;
+    }
+    const float cap_in = softcap > 0.f ? scale / softcap : 0.f, cap_back = softcap > 0.f ? softcap / scale : 0.f;
+    unsigned qf[KSTEPS][4];
+    if constexpr (KSTEPS <= 8) {                           // the queries stay in registers
+        const bf16* Qw = Qs + ((lane & 15) & (q_rows - 1)) * LDK + (lane >> 4) * 8;
+#pragma unroll
+        for (int kk = 0; kk < KSTEPS; ++kk) ldmatrix_x4(qf[kk], Qw + kk * 16);
+    }
+    float o[NT_O][4];
+#pragma unroll
+    for (int n = 0; n < NT_O; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+
+    for (int t = 0; t < ntiles; ++t) {
+        cp_async_wait<ROW_STAGES - 2>();
+        __syncwarp();                                      // every lane's copies of this stage are there
+        load(t + ROW_STAGES - 1);                          // (into the stage that was read last time)
+        const int k0 = kbeg + t * 64;
+        if (k0 >= kend || k0 + WK - 1 < first) continue;
+        const bf16* Ks = ring + (t % ROW_STAGES) * stage_elems_w;
+        const bf16* Vs = tied ? Ks : Ks + WK * LDK;
+        const int ldv_s = tied ? LDK : LDV;
+        float sc[2][4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sc[j][e] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < KSTEPS; ++kk) {
+            unsigned bf[4];
+            ldmatrix_x4(bf, Ks + ((lane >> 4) * 8 + (lane & 7)) * LDK + kk * 16 + ((lane >> 3) & 1) * 8);
+            if constexpr (KSTEPS > 8) ldmatrix_x4(qf[kk], Qs + ((lane & 15) & (q_rows - 1)) * LDK + (lane >> 4) * 8 + kk * 16);
+            mma_bf16(sc[0], qf[kk], bf[0], bf[1]);
+            mma_bf16(sc[1], qf[kk], bf[2], bf[3]);
+        }
+        float alpha[2] = {1.f, 1.f};
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            if (h == 1 && !two) {
+                sc[0][2] = sc[0][3] = sc[1][2] = sc[1][3] = 0.f;
+                continue;
+            }
+            float mx = -INFINITY;
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int kp = k0 + j * 8 + tig * 2 + e;
+                    float v = sc[j][2 * h + e];
+                    if (softcap > 0.f) v = cap_back * tanhf(v * cap_in);
+                    v = fmaf(slope[h], (float)(kp - pos), v);
+                    v = (kp < kend && kp >= first) ? v : -INFINITY;
+                    sc[j][2 * h + e] = v;
+                    mx = fmaxf(mx, v);
+                }
+            if (sig_bias != nullptr) {
+                // sigmoid(x) = 1 / (1 + 2^(-x log2 e)); a masked score (-inf) gives 0
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const float v = sc[j][2 * h + e];
+                        sc[j][2 * h + e] = __fdividef(1.f, 1.f + exp2f(fminf(fmaf(v, -scale_log2, -bias2[h]), 126.f))) *
+                                           (v == -INFINITY ? 0.f : 1.f);
+                    }
+                continue;
+            }
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+            const float m_new = fmaxf(m[h], mx * scale_log2);
+            const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
+            alpha[h] = exp2f(m[h] - m_use);
+            m[h] = m_new;
+            float sum = 0.f;
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    sc[j][2 * h + e] = exp2f(fmaf(sc[j][2 * h + e], scale_log2, -m_use));
+                    sum += sc[j][2 * h + e];
+                }
+            l[h] = l[h] * alpha[h] + sum;
+        }
+        if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+            for (int n = 0; n < NT_O; ++n) {
+                o[n][0] *= alpha[0];
+                o[n][1] *= alpha[0];
+                o[n][2] *= alpha[1];
+                o[n][3] *= alpha[1];
+            }
+        }
+        unsigned a[4];
+        a[0] = pack_bf16(sc[0][0], sc[0][1]);
+        a[1] = pack_bf16(sc[0][2], sc[0][3]);
+        a[2] = pack_bf16(sc[1][0], sc[1][1]);
+        a[3] = pack_bf16(sc[1][2], sc[1][3]);
+        const bf16* Vw = Vs + ((lane & 7) + ((lane >> 3) & 1) * 8) * ldv_s + (lane >> 4) * 8;
+#pragma unroll
+        for (int np = 0; np < NT_O / 2; ++np) {
+            unsigned vf[4];
+            ldmatrix_x4_trans(vf, Vw + np * 16);
+            mma_bf16(o[2 * np], a, vf[0], vf[1]);
+            mma_bf16(o[2 * np + 1], a, vf[2], vf[3]);
+        }
+    }
+    cp_async_wait<0>();
+    pdl_launch_dependents();
+
+    // the warps' rows meet: [warp][row][DV] results and [warp][row][2] maxima and sums
+    __syncthreads();                                       // (the ring is free)
+    float* ow = reinterpret_cast<float*>(Qs + q_rows * LDK);
+    float* ml = ow + (size_t)4 * q_rows * DV;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        if (h == 1 && !two) continue;
+        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
+        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
+        const int row = h ? r_hi : r_lo;
+        float* dst = ow + (size_t)(warp * q_rows + row) * DV + tig * 2;
+#pragma unroll
+        for (int n = 0; n < NT_O; ++n) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
+        if (tig == 0) {
+            ml[2 * (warp * q_rows + row)] = sig_bias != nullptr ? 0.f : m[h];
+            ml[2 * (warp * q_rows + row) + 1] = l[h];
+        }
+    }
+    __syncthreads();
+    for (int idx = tid; idx < g * (DV / 2); idx += NTHREADS) {
+        const int row = idx / (DV / 2), c = (idx - row * (DV / 2)) * 2;
+        const int head = kvh * g + row;
+        float M = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) M = fmaxf(M, ml[2 * (w * q_rows + row)]);
+        float L = 0.f, a0 = 0.f, a1 = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+            const float mw = ml[2 * (w * q_rows + row)];
+            const float f = mw == -INFINITY ? 0.f : exp2f(mw - M);
+            const float2 v = *reinterpret_cast<const float2*>(ow + (size_t)(w * q_rows + row) * DV + c);
+            L += ml[2 * (w * q_rows + row) + 1] * f;
+            a0 += v.x * f;
+            a1 += v.y * f;
+        }
+        if (splits > 1) {
+            const size_t pi = ((size_t)q0 * H + head) * splits + blockIdx.y;
+            if (c == 0) {
+                part_ml[2 * pi] = M;
+                part_ml[2 * pi + 1] = L;
+            }
+            *reinterpret_cast<float2*>(part_o + pi * DV + c) = make_float2(a0, a1);
+            continue;
+        }
+        if (sink != nullptr) L += (M == -INFINITY) ? 1.f : exp2f(sink[head] * 1.4426950408889634f - M);
+        float inv = L > 0.f ? 1.f / L : 0.f;
+        if (sig_bias != nullptr) inv = 1.f;
+        inv *= out_scale;
+        if (gate != nullptr) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)q0 * ldg + head])));
+        *reinterpret_cast<unsigned*>(out + (size_t)q0 * ldo + (size_t)head * DV + c) = pack_bf16(a0 * inv, a1 * inv);
+    }
+}
+
 // out[t][h] = sum_s o_s 2^(m_s - M) / sum_s l_s 2^(m_s - M) (times the gate): one block a (token,
 // head), a thread two neighbouring columns; the splits' weights are formed once per block.
 __global__ void __launch_bounds__(128) attention_kv_combine_kernel(
@@ -459,8 +722,16 @@ int slb_attention_kv_mma_status(int reset) {
     return v;
 }
 // Blocks of the kernel an SM holds at once (separate keys and values), for the choice of splits:
-// `group` rows a tile in the narrow form.
+// `group` rows a tile in the narrow form (`narrow` 2: the form with a quarter of the keys a warp, where it exists).
 int slb_attention_kv_mma_resident(int narrow, int group) {
+    if (narrow == 2 && ROWS_FORM) {
+        static unsigned long long configured_rows = 0;
+        if (slb_configure(&configured_rows, attention_kv_rows_kernel, rows_smem(16, false)) != 0) return 1;
+        int n = 0;
+        const cudaError_t e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_kv_rows_kernel, NTHREADS,
+                                                                            rows_smem(group <= 8 ? 8 : 16, false));
+        return e == cudaSuccess && n > 0 ? n : 1;
+    }
     const int q_rows = narrow ? (group <= 8 ? 8 : 16) : BM;
     const size_t smem = ((size_t)q_rows * LDK + 2 * stage_elems(false)) * sizeof(bf16);
     static unsigned long long configured = 0, configured_narrow = 0;       // (sizes above 48 KB need the opt-in first)
@@ -485,7 +756,8 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
                                    const float* slopes = nullptr, float out_scale = 1.f) {
     // `fold` > 1: H counts (head, map) pairs, `maps` is 1, DK is fold times a map's key size.
     // `narrow`: every tile of the list holds at most 16 rows (a step of single tokens with at most
-    // 16 query heads a kv head).
+    // 16 query heads a kv head).  2: the same by the kernel with a quarter of the keys a warp, for one map and
+    // key sizes up to 192 (other sizes: as 1).
     // `splits` > 1 (steps of single tokens only: a tile is one token's heads): scratch part_o
     // [tokens][H * maps][splits][DV] and part_ml [tokens][H * maps][splits][2], float32.
     if (num_tiles <= 0) return 0;
@@ -500,6 +772,21 @@ static int launch_attention_kv_mma(const bf16* q, int ldq, const bf16* kc, const
         (fold > 1 && (maps != 1 || tied || DK % (8 * fold) != 0 || H % fold != 0)))
         return SLB_ERR_BAD_ARG;
     if ((long long)num_tiles * Hkv * maps > 2147483647LL) return SLB_ERR_TOO_LARGE;
+    if (narrow == 2 && ROWS_FORM && maps == 1 && fold == 1 && out_f32 == nullptr) {
+        const int qr = H / Hkv <= 8 ? 8 : 16;
+        static unsigned long long configured_rows = 0;
+        const int rcr = slb_configure(&configured_rows, attention_kv_rows_kernel, rows_smem(16, false));
+        if (rcr != 0) return rcr;
+        const int er = slb_launch(attention_kv_rows_kernel, dim3(num_tiles * Hkv, splits), dim3(NTHREADS),
+                                  rows_smem(qr, tied != 0 && DV <= DK), st, q, ldq, kc, tied ? kc : vc, tied, out, ldo, block_table,
+                                  max_pages, cu_q, ctx_len, tile_seq, H, Hkv, ps, num_pages, scale * 1.4426950408889634f,
+                                  window, gate, ldg, splits, part_o, part_ml, qr, softcap, scale, sink, chunk, sig_bias,
+                                  slopes, out_scale);
+        if (er != 0 || splits == 1) return er;
+        return slb_launch(attention_kv_combine_kernel, dim3(num_tiles, H), dim3(128), 0, st, (const float*)part_o,
+                          (const float*)part_ml, splits, out, ldo, H, gate, ldg, out_f32, sink,
+                          sig_bias != nullptr ? 1 : 0, out_scale);
+    }
     // (a narrow tile of at most 8 rows keeps 8 rows of Q: a third block fits an SM at the largest sizes)
     const int q_rows = narrow ? (H / Hkv <= 8 ? 8 : 16) : BM;
     const size_t smem = ((size_t)q_rows * LDK + 2 * stage_elems(tied != 0)) * sizeof(bf16);

@@ -145,14 +145,34 @@ __global__ void __launch_bounds__(128) group_norm_gate_kernel(
 
 // The gate before the norm: v = x * act(gate), every one of `groups` equal parts of a row divided by its own root
 // mean square, times a weight over the row and a factor.  A block a (token, part); x float32, float32 arithmetic;
-// up to GGN_NV elements a thread stay in registers, longer parts are formed again.
+// a thread keeps GGN_NV vectors of V elements in registers, longer parts are formed again.
 #define GGN_THREADS 256
-#define GGN_NV 8
+#define GGN_NV 4
 __device__ __forceinline__ float gated_by(float x, float z, int gate_act) {
     const float sg = 1.0f / (1.0f + expf(-z));
     return x * (gate_act == 2 ? z * sg : sg);
 }
-template <typename T>
+__device__ __forceinline__ void ggn_load(const float* p, float (&v)[4]) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+}
+__device__ __forceinline__ void ggn_load(const bf16* p, float (&v)[4]) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+template <typename T> __device__ __forceinline__ void ggn_load(const T* p, float (&v)[1]) { v[0] = to_float(p[0]); }
+__device__ __forceinline__ void ggn_store(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void ggn_store(bf16* p, const float (&v)[4]) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+}
+template <typename T> __device__ __forceinline__ void ggn_store(T* p, const float (&v)[1]) { p[0] = from_float<T>(v[0]); }
+
+template <typename T, int V>
 __global__ void __launch_bounds__(GGN_THREADS) gate_group_norm_kernel(
     const float* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, int gate_act, const float* __restrict__ w,
     float eps, float factor, T* __restrict__ out, int ldo, int size) {
@@ -164,25 +184,44 @@ __global__ void __launch_bounds__(GGN_THREADS) gate_group_norm_kernel(
     const float* xr = x + t * ldx + c0;
     const T* gr = gate + t * ldg + c0;
     T* o = out + t * ldo + c0;
-    float v[GGN_NV];
+    float v[GGN_NV][V], z[GGN_NV][V];
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < GGN_NV; ++j) {
-        const int c = threadIdx.x + j * blockDim.x;
-        v[j] = c < size ? gated_by(xr[c], to_float(gr[c]), gate_act) : 0.f;
-        ss += v[j] * v[j];
+        const int c = (threadIdx.x + j * blockDim.x) * V;
+        if (c < size) {
+            ggn_load(xr + c, v[j]);
+            ggn_load(gr + c, z[j]);
+        }
     }
-    for (int c = threadIdx.x + GGN_NV * blockDim.x; c < size; c += blockDim.x) {
+#pragma unroll
+    for (int j = 0; j < GGN_NV; ++j) {
+        const int c = (threadIdx.x + j * blockDim.x) * V;
+        if (c < size) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                v[j][e] = gated_by(v[j][e], z[j][e], gate_act);
+                ss += v[j][e] * v[j][e];
+            }
+        }
+    }
+    for (int c = threadIdx.x + GGN_NV * V * blockDim.x; c < size; c += blockDim.x) {
         const float u = gated_by(xr[c], to_float(gr[c]), gate_act);
         ss += u * u;
     }
     const float rstd = factor / sqrtf(block_sum(ss, scratch) / (float)size + eps);
 #pragma unroll
     for (int j = 0; j < GGN_NV; ++j) {
-        const int c = threadIdx.x + j * blockDim.x;
-        if (c < size) o[c] = from_float<T>(v[j] * rstd * (w != nullptr ? w[c0 + c] : 1.f));
+        const int c = (threadIdx.x + j * blockDim.x) * V;
+        if (c < size) {
+            float wv[V];
+            if (w != nullptr) ggn_load(w + c0 + c, wv);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[j][e] *= rstd * (w != nullptr ? wv[e] : 1.f);
+            ggn_store(o + c, v[j]);
+        }
     }
-    for (int c = threadIdx.x + GGN_NV * blockDim.x; c < size; c += blockDim.x)
+    for (int c = threadIdx.x + GGN_NV * V * blockDim.x; c < size; c += blockDim.x)
         o[c] = from_float<T>(gated_by(xr[c], to_float(gr[c]), gate_act) * rstd * (w != nullptr ? w[c0 + c] : 1.f));
 }
 
@@ -194,10 +233,17 @@ static int launch_gate_group_norm(const float* x, int ldx, const T* gate, int ld
     if (groups <= 0 || groups > 65535 || size <= 0 || gate == nullptr || gate_act < 1 || gate_act > 2 ||
         ldx < groups * size || ldg < groups * size || ldo < groups * size)
         return SLB_ERR_BAD_ARG;
-    int threads = (size + 31) / 32 * 32;
+    const uintptr_t half = (uintptr_t)gate | (uintptr_t)out;
+    const bool vec = ((size | ldx | ldg | ldo) & 3) == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0 &&
+                     (half & (4 * sizeof(T) - 1)) == 0;
+    const int units = vec ? size / 4 : size;
+    int threads = (units + 31) / 32 * 32;
     threads = threads > GGN_THREADS ? GGN_THREADS : threads;
-    return slb_launch(gate_group_norm_kernel<T>, dim3(T_, groups), dim3(threads), 0, st, x, ldx, gate, ldg, gate_act, w,
-                      eps, factor, out, ldo, size);
+    if (vec)
+        return slb_launch(gate_group_norm_kernel<T, 4>, dim3(T_, groups), dim3(threads), 0, st, x, ldx, gate, ldg,
+                          gate_act, w, eps, factor, out, ldo, size);
+    return slb_launch(gate_group_norm_kernel<T, 1>, dim3(T_, groups), dim3(threads), 0, st, x, ldx, gate, ldg, gate_act,
+                      w, eps, factor, out, ldo, size);
 }
 
 template <typename T>

@@ -999,12 +999,20 @@ def attention_kv_splits(num_seqs: int, num_kv_heads: int, longest_context: int, 
 _kv_resident = {}
 
 
-def attention_kv_resident(lib, k_dim: int, v_dim: int, narrow: bool, group: int) -> int:
+def attention_kv_resident(lib, k_dim: int, v_dim: int, narrow: int, group: int) -> int:
     """Blocks of the tensor-core kernel for these sizes that an SM holds at once."""
-    key = (k_dim, v_dim, bool(narrow), group <= 8)
+    key = (k_dim, v_dim, int(narrow), group <= 8)
     if key not in _kv_resident:
-        _kv_resident[key] = int(lib.slb_attention_kv_mma_resident(1 if narrow else 0, group))
+        _kv_resident[key] = int(lib.slb_attention_kv_mma_resident(int(narrow), group))
     return _kv_resident[key]
+
+
+def _kv_narrow_form(ctx, group: int, k_dim: int, seen: int) -> int:
+    """The form of the tensor-core kernel for a step whose requests see at most ``seen`` keys: 0 (a warp 16 rows),
+    1 (the warps share at most 16 rows) or 2 (the same rows, a quarter of the keys a warp)."""
+    if not (ctx.decode_only and attention_kv_narrow and group <= 16):
+        return 0
+    return 2 if k_dim <= ATTENTION_KV_WARP_KEYS_MAX_DIM and seen >= attention_kv_warp_keys_min else 1
 
 
 def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num_heads: int,
@@ -1021,11 +1029,11 @@ def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num
     rows = lib.slb_attention_kv_mma_tile_rows()
     tile_seq, tile_row0, n = ctx.attention_tiles(num_heads // num_kv_heads, rows)
     splits, part_o, part_ml = 1, None, None
+    # (a chunk's keys fill up from its start: at most ``chunk`` of them, half on average)
+    longest = min(ctx.split_hint_len, chunk) if chunk else ctx.split_hint_len
+    narrow = _kv_narrow_form(ctx, num_heads // num_kv_heads, k_dim, min(longest, window) if window > 0 else longest)
     if ctx.decode_only and attention_kv_split and num_heads // num_kv_heads <= rows:
-        narrow = attention_kv_narrow and num_heads // num_kv_heads <= 16
-        # (a chunk's keys fill up from its start: at most ``chunk`` of them, half on average)
-        splits = attention_kv_splits(ctx.num_seqs, num_kv_heads,
-                                     min(ctx.split_hint_len, chunk) if chunk else ctx.split_hint_len, window,
+        splits = attention_kv_splits(ctx.num_seqs, num_kv_heads, longest, window,
                                      max_splits=lib.slb_attention_kv_mma_max_splits(),
                                      resident=attention_kv_resident(lib, k_dim, v_dim, narrow,
                                                                     num_heads // num_kv_heads))
@@ -1038,7 +1046,7 @@ def attention_kv_mma(ctx, q, k_cache, v_cache, tied: bool, out, block_table, num
             ctx.ctx_len.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), n, num_heads, num_kv_heads,
             page_size, k_cache.shape[0], float(scale), int(window), _p(head_gate),
             head_gate.stride(0) if head_gate is not None else 0, splits, _p(part_o), _p(part_ml),
-            1 if ctx.decode_only and attention_kv_narrow and num_heads // num_kv_heads <= 16 else 0)
+            narrow)
     if (softcap or sink is not None or chunk or sigmoid_bias is not None or slopes is not None
             or out_scale != 1.0):
         L.check(lib.slb_attention_kv_mma_capped_bf16(*args, float(softcap or 0.0), _p(sink), int(chunk),
@@ -1051,6 +1059,10 @@ attention_kv_split = True      # (off: one block a request and kv head, the twin
 # steps of single tokens with at most 16 query heads a kv head: the block's warps share the rows
 # and split the value columns (off: a warp 16 rows, the twin)
 attention_kv_narrow = True
+# ... and with keys of up to 192 elements a quarter of the keys a warp, from contexts on that are worth the merge of
+# the warps' rows at the end (below: the twin that repeats the scores in every warp)
+attention_kv_warp_keys_min = 512
+ATTENTION_KV_WARP_KEYS_MAX_DIM = 192
 
 
 # steps of single tokens with several maps a head: the maps become rows of one block (a library

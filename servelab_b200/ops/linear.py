@@ -208,11 +208,15 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
 narrow_logits_max_tokens = 512     # from here on the library's product
 
 
+def narrow_logits_by_library(x: torch.Tensor) -> bool:
+    return x.dtype != torch.float32 and x.shape[0] >= narrow_logits_max_tokens
+
+
 def narrow_logits(x: torch.Tensor, w: torch.Tensor, w_f32: torch.Tensor) -> torch.Tensor:
     """float32 x W^T for a matrix of few rows: [T, >= rows].  ``w`` in the compute type with its rows padded to
     a multiple of 8, ``w_f32`` float32 [rows, hidden].  Steps of few tokens: one launch of this package's
     kernel for narrow matrices (a product of wide tiles would split K and reduce)."""
-    if x.dtype == torch.float32 or x.shape[0] >= narrow_logits_max_tokens:
+    if x.dtype == torch.float32 or narrow_logits_by_library(x):
         return linear(x, w, out_dtype=torch.float32)
     return K.router_logits(x, w_f32)
 

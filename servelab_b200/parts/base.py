@@ -40,8 +40,10 @@ not set it always gets plain tensors.
 A mixer with ``splits_projections = True`` lets a mixer around it merge its products with those of
 another: after ``load`` it holds ``w_in`` (the matrix of its first product, [a multiple of 8, hidden]),
 ``w_o`` and ``o_bias`` (None: none) of its last one, and ``core(ctx, x, proj, cache, owns_cache, out,
-factor)`` turns the first product's rows ``proj`` (columns of a wider row) into ``factor`` times the rows
-that the last product reads, written to ``out`` [T, out_width] (columns of a wider row too).
+factor, early)`` turns the first product's rows ``proj`` (columns of a wider row) into ``factor`` times the
+rows that the last product reads, written to ``out`` [T, out_width] (columns of a wider row too).  ``core`` may
+run on a stream of its own and launches this package's kernels only; ``early(ctx, x)`` runs what it needs of
+the library's products before it, on the step's stream, and what it returns is handed to ``core``.
 """
 
 from __future__ import annotations

@@ -172,7 +172,10 @@ class NormedAttention(Mixer):
             return linear(out, self.w_o, self.o_bias, out_dtype=self.out_dtype)
         return linear(out, self.w_o, self.o_bias, consumer="norm", bias_cast=self.o_bias_cast)
 
-    def core(self, ctx, x, proj, cache, owns_cache, out, factor=1.0):
+    def early(self, ctx, x):
+        return None
+
+    def core(self, ctx, x, proj, cache, owns_cache, out, factor=1.0, early=None):
         s = self.spec
         T = x.shape[0]
         table = ctx.block_tables[cache.group]

@@ -11,7 +11,9 @@ Both branches are mixers of the registry, built from their own specs under
 float32 and one kernel norms both over the model width and adds them.  Without norms the sum is linear in
 what the branches' last products read, so both first products are one product and both last products are
 one: the matrices are concatenated at load, each branch works on its columns of the two rows and
-multiplies its own by its factor (``splits_projections``, see ``parts/base.py``).
+multiplies its own by its factor (``splits_projections``, see ``parts/base.py``).  Between the two products
+the branches have nothing to do with one another: in a captured step the right one runs on a stream of
+its own, so that two chains of short kernels run side by side.
 
 What the branches ask of the cache is merged into one request of this mixer: pages from the one
 branch that wants pages (two paged branches would need two block tables a layer, which is not
@@ -30,6 +32,17 @@ from ..ops.linear import linear
 from ..weights.source import NORM, TensorDecl
 from .base import LayerCache, Mixer
 from .registry import MIXERS, build_part, part_class, register_mixer
+
+
+overlap_branches = True       # (captured steps; off: one after the other, as in steps launched one by one)
+_side_streams = {}
+
+
+def _side_stream(device) -> torch.cuda.Stream:
+    key = torch.device(device)
+    if key not in _side_streams:
+        _side_streams[key] = torch.cuda.Stream(device=key)
+    return _side_streams[key]
 
 
 def _record_sizes(spec):
@@ -123,8 +136,23 @@ class ParallelMixers(Mixer):
         proj = K.plain_unless(None, linear(x, self.w_in))
         make = torch.zeros if self.row_padding else torch.empty
         row = make((x.shape[0], self.row_width), dtype=x.dtype, device=x.device)
-        self.left.core(ctx, x, proj[:, :self.right_rows], self._branch_cache(cache, 0), owns_cache,
-                       row[:, :self.left.out_width], self.spec.left_factor)
-        self.right.core(ctx, x, proj[:, self.right_rows:], self._branch_cache(cache, 1), owns_cache,
-                        row[:, self.right_at:self.right_at + self.right.out_width], self.spec.right_factor)
+        early = self.right.early(ctx, x)
+
+        def left():
+            self.left.core(ctx, x, proj[:, :self.right_rows], self._branch_cache(cache, 0), owns_cache,
+                           row[:, :self.left.out_width], self.spec.left_factor, self.left.early(ctx, x))
+
+        def right():
+            self.right.core(ctx, x, proj[:, self.right_rows:], self._branch_cache(cache, 1), owns_cache,
+                            row[:, self.right_at:self.right_at + self.right.out_width], self.spec.right_factor, early)
+        if overlap_branches and torch.cuda.is_current_stream_capturing():
+            main, side = torch.cuda.current_stream(), _side_stream(x.device)
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                right()
+            left()
+            main.wait_stream(side)
+        else:
+            left()
+            right()
         return linear(row, self.w_o, self.o_bias, consumer="norm", bias_cast=self.o_bias_cast)

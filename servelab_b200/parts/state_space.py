@@ -19,7 +19,7 @@ import torch
 
 from ..cache.manager import FixedStateRequest
 from ..ops import kernels as K
-from ..ops.linear import linear, narrow_logits
+from ..ops.linear import linear, narrow_logits, narrow_logits_by_library
 from ..weights.source import BIAS, MATRIX, NORM, TensorDecl
 from .base import Mixer
 from .normed_attention import pad_rows
@@ -104,12 +104,16 @@ class StateSpace(Mixer):
             return linear(out, self.w_o, out_dtype=self.out_dtype)
         return linear(out, self.w_o, consumer="norm")
 
-    def core(self, ctx, x, proj, cache, owns_cache, out, factor=1.0):
+    def early(self, ctx, x):
+        """The step sizes' logits, where they come from a product of the library."""
+        return narrow_logits(x, self.w_dt, self.w_dt_f32) if narrow_logits_by_library(x) else None
+
+    def core(self, ctx, x, proj, cache, owns_cache, out, factor=1.0, early=None):
         s = self.spec
         T = x.shape[0]
         if not owns_cache:
             raise NotImplementedError("state_space: a run that reads another run's cache")
-        dt = narrow_logits(x, self.w_dt, self.w_dt_f32)
+        dt = narrow_logits(x, self.w_dt, self.w_dt_f32) if early is None else early
         state = cache.state if cache.state.dim() == 2 else cache.state.view(cache.state.shape[0], -1)
         rows = state[:, self.state_floats:] if s.conv_taps > 1 else None
         u = torch.empty((T, self.channels), dtype=x.dtype, device=x.device)

@@ -231,15 +231,28 @@ def test_attention_with_a_distance_bias(dtype, spike, shape, decode):
             _close(run(), want, tol, "mma")
         finally:
             A.use_kv_tc_capped = True
+        if decode:                                     # ... as are the two forms for single tokens
+            saved = K.attention_kv_warp_keys_min
+            try:
+                for least in (0, 1 << 30):
+                    K.attention_kv_warp_keys_min = least
+                    _close(run(), want, tol, least)
+            finally:
+                K.attention_kv_warp_keys_min = saved
         if Dk % 64 == 0 and Dv % 64 == 0:
             assert K.attention_kv_tc_status(Dk, Dv) == 0 and K.attention_kv_mma_status(Dk, Dv) == 0
 
 
 @pytest.mark.parametrize("window,ctxs", [(None, [1500, 900, 1]), (1100, [1100, 2201, 900])])
-def test_attention_single_tokens_with_key_splits_and_a_distance_bias(window, ctxs):
-    """Few requests with long contexts: the keys are split over blocks; the added one counts once."""
+@pytest.mark.parametrize("least", [0, 1 << 30])
+@pytest.mark.parametrize("shape", [(8, 2, 64, 48, 16), (12, 1, 192, 256, 8), (3, 1, 128, 128, 32)])
+def test_attention_single_tokens_with_key_splits_and_a_distance_bias(window, ctxs, least, shape, monkeypatch):
+    """Few requests with long contexts: the keys are split over blocks; the added one counts once.  Both forms of the
+    kernel."""
     from servelab_b200.ops import attention as A
-    Hq, G, Dk, Dv, ps = 8, 2, 64, 48, 16
+    from servelab_b200.ops import kernels as K
+    monkeypatch.setattr(K, "attention_kv_warp_keys_min", least)
+    Hq, G, Dk, Dv, ps = shape
     for spike in ("in", "far", None):
         case = _attention_case(5, Hq, G, Dk, Dv, window, ctxs, [1, 1, 1], ps, torch.bfloat16, spike, 0.3, 14.0)
         ctx = _ctx(case["entries"])
@@ -248,6 +261,32 @@ def test_attention_single_tokens_with_key_splits_and_a_distance_bias(window, ctx
                        window or 0, None, 14.0, torch.zeros(Hq, device=DEV), slopes=plain.head_slopes(Hq).float().to(DEV),
                        out_scale=1.5)
         _close(out, case["want"] * 1.5, 1.5e-2, spike)
+
+
+@pytest.mark.parametrize("chunk", [0, 700])
+def test_single_token_forms_agree_on_gates_sigmoid_weights_and_tied_values(chunk, monkeypatch):
+    """What other designs ask of the kernel for single tokens: weights that are not normalized in chunks, a gate a
+    head, values that are a prefix of the keys, a learned sink -- the two forms against each other."""
+    from servelab_b200.ops import attention as A
+    from servelab_b200.ops import kernels as K
+    Hq, G, Dk, Dv, ps = 6, 2, 96, 64, 16
+    case = _attention_case(9, Hq, G, Dk, Dv, None, [1400, 650, 40], [1, 1, 1], ps, torch.bfloat16, None, 0.2, None)
+    ctx = _ctx(case["entries"])
+    gate = torch.randn(3, Hq, device=DEV).to(torch.bfloat16)
+    extra = torch.linspace(-2.0, 2.0, Hq, device=DEV)
+
+    def run(least, tied, **kw):
+        monkeypatch.setattr(K, "attention_kv_warp_keys_min", least)
+        out = torch.empty(3, Hq * Dv, dtype=torch.bfloat16, device=DEV)
+        v = case["kc"] if tied else case["vc"]
+        A.kv_attention(ctx, case["q"], case["kc"], v, Dk if tied else Dv, out, ctx.block_tables[0], Hq, G, Dk, Dv, ps, 0.2,
+                       0, **kw)
+        return out.double().cpu()
+    for tied in (False, True):
+        for kw in (dict(head_gate=gate, chunk=chunk), dict(head_gate=gate, sink=extra, softcap=5.0, chunk=chunk),
+                   dict(head_gate=None, sigmoid_bias=extra, chunk=chunk)):
+            a, b = run(0, tied, **kw), run(1 << 30, tied, **kw)
+            assert (a - b).abs().max() < 1e-2 * max(1.0, float(b.abs().max())), (tied, list(kw))
 
 
 # ------------------------------------------------------- convolution with SiLU
