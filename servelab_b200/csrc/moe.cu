@@ -466,19 +466,75 @@ __global__ void __launch_bounds__(128) moe_product_mma_kernel(
 }
 
 // ----------------------------------------------------------------- combine
-template <typename T, typename TY>
+__device__ __forceinline__ void combine_load(const float* p, float (&v)[4]) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+}
+__device__ __forceinline__ void combine_load(const bf16* p, float (&v)[4]) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+template <typename T> __device__ __forceinline__ void combine_load(const T* p, float (&v)[1]) { v[0] = to_float(p[0]); }
+__device__ __forceinline__ void combine_store(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void combine_store(bf16* p, const float (&v)[4]) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(slb_mma::pack_bf16(v[0], v[1]), slb_mma::pack_bf16(v[2], v[3]));
+}
+template <typename T> __device__ __forceinline__ void combine_store(T* p, const float (&v)[1]) { p[0] = from_float<T>(v[0]); }
+
+// a thread V neighbouring columns; the experts' rows of four choices are in flight at once, the additions keep the
+// order of the choice
+template <typename T, typename TY, int V>
 __global__ void __launch_bounds__(256) moe_combine_kernel(
     const TY* __restrict__ y, int ldy, const float* __restrict__ weights, const T* __restrict__ shared,
     int lds, T* __restrict__ out, int ldo, int top, int N) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < N; c += gridDim.y * blockDim.x) {
-        float v = 0.f;
-        for (int k = 0; k < top; ++k) v += (weights != nullptr ? weights[(size_t)t * top + k] : 1.f) * to_float(y[((size_t)t * top + k) * ldy + c]);
-        if (shared != nullptr) v += to_float(shared[(size_t)t * lds + c]);
-        out[(size_t)t * ldo + c] = from_float<T>(v);
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * V; c < N; c += gridDim.y * blockDim.x * V) {
+        float v[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = 0.f;
+        for (int k0 = 0; k0 < top; k0 += 4) {
+            float r[4][V], w[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                if (k0 + k >= top) continue;
+                combine_load(y + ((size_t)t * top + k0 + k) * ldy + c, r[k]);
+                w[k] = weights != nullptr ? weights[(size_t)t * top + k0 + k] : 1.f;
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                if (k0 + k >= top) continue;
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] += w[k] * r[k][e];
+            }
+        }
+        if (shared != nullptr) {
+            float r[V];
+            combine_load(shared + (size_t)t * lds + c, r);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] += r[e];
+        }
+        combine_store(out + (size_t)t * ldo + c, v);
     }
+}
+
+template <typename T, typename TY>
+static int launch_moe_combine(const TY* y, int ldy, const float* weights, const T* shared, int lds, T* out, int ldo,
+                              int T_, int top, int N, cudaStream_t st) {
+    if (T_ <= 0) return 0;
+    const uintptr_t half = (uintptr_t)shared | (uintptr_t)out;
+    const bool vec = ((N | ldy | ldo | (shared != nullptr ? lds : 0)) & 3) == 0 && ((uintptr_t)y & (4 * sizeof(TY) - 1)) == 0 &&
+                     (half & (4 * sizeof(T) - 1)) == 0;
+    const int units = vec ? (N + 3) / 4 : N;
+    const dim3 grid(T_, T_ < 256 ? (units + 255) / 256 : 1);
+    if (vec)
+        return slb_launch(moe_combine_kernel<T, TY, 4>, grid, dim3(256), 0, st, y, ldy, weights, shared, lds, out, ldo, top, N);
+    return slb_launch(moe_combine_kernel<T, TY, 1>, grid, dim3(256), 0, st, y, ldy, weights, shared, lds, out, ldo, top, N);
 }
 
 static int moe_num_tiles(int P, int E) { return (P + MOE_BM - 1) / MOE_BM + E; }
@@ -597,21 +653,15 @@ int slb_moe_down_bf16(const bf16* act, int lda, const bf16* w_down, int ldw, flo
 }
 int slb_moe_combine_f32(const float* y, int ldy, const float* weights, const float* shared, int lds,
                         float* out, int ldo, int T, int top, int N, cudaStream_t st) {
-    if (T <= 0) return 0;
-    return slb_launch(moe_combine_kernel<float, float>, dim3(T, T < 256 ? (N + 255) / 256 : 1), dim3(256), 0, st, y, ldy, weights, shared, lds,
-                      out, ldo, top, N);
+    return launch_moe_combine<float, float>(y, ldy, weights, shared, lds, out, ldo, T, top, N, st);
 }
 int slb_moe_combine_bf16(const float* y, int ldy, const float* weights, const bf16* shared, int lds,
                          bf16* out, int ldo, int T, int top, int N, cudaStream_t st) {
-    if (T <= 0) return 0;
-    return slb_launch(moe_combine_kernel<bf16, float>, dim3(T, T < 256 ? (N + 255) / 256 : 1), dim3(256), 0, st, y, ldy, weights, shared, lds,
-                      out, ldo, top, N);
+    return launch_moe_combine<bf16, float>(y, ldy, weights, shared, lds, out, ldo, T, top, N, st);
 }
 // the experts' rows in bfloat16 (a library product left them so)
 int slb_moe_combine_bf16_rows(const bf16* y, int ldy, const float* weights, const bf16* shared, int lds,
                               bf16* out, int ldo, int T, int top, int N, cudaStream_t st) {
-    if (T <= 0) return 0;
-    return slb_launch(moe_combine_kernel<bf16, bf16>, dim3(T, T < 256 ? (N + 255) / 256 : 1), dim3(256), 0, st,
-                      y, ldy, weights, shared, lds, out, ldo, top, N);
+    return launch_moe_combine<bf16, bf16>(y, ldy, weights, shared, lds, out, ldo, T, top, N, st);
 }
 }
