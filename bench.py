@@ -20,9 +20,9 @@ extra flush is needed.
 ``--impl reference``: the reference's engine cannot run (the line says what its import
 raises); its two GPU kernels can, and are timed beside this package's on the same data.
 
-``--compare dezelorn`` / ``--compare daferax`` / ``--compare zimupel`` / ``--compare sumolorn`` / ``--compare vufadra`` / ``--compare sunutar``: instead of all this, the named
-design beside the Qwen2 decoder (Zimupel: beside Daferax) at a few equal layer sizes (prefill and decode throughput, the times and roofline
-fractions of the kernels that differ), one JSON line.
+``--compare DESIGN`` (dezelorn, daferax, zimupel, sumolorn, vufadra, sunutar): instead of all this, the named design
+beside the closest other model of the package (Dezelorn and Daferax: the Qwen2 decoder) at a few equal layer sizes
+(prefill and decode throughput, the times and roofline fractions of the kernels that differ), one JSON line.
 
 More than one GPU is not supported: one line says so and the exit code is 2.
 """
@@ -177,7 +177,7 @@ def main(argv=None) -> int:
     ap.add_argument("--no-graphs", action="store_true", help="profiling aid: launch kernels eagerly")
     ap.add_argument("--compare", default="", choices=["", "dezelorn", "daferax", "zimupel", "sumolorn", "vufadra", "sunutar"],
                     help="instead of the default workload: prefill and decode throughput of the named "
-                         "design beside the Qwen2 decoder at equal layer sizes (bench/arch_compare.py)")
+                         "design beside the closest other model at equal layer sizes (bench/arch_compare.py)")
     ap.add_argument("--compare-sizes", default="", help="comma-separated subset of the sizes to compare")
     ap.add_argument("--tune", action="append", default=[], metavar="NAME=VALUE",
                     help="measurement aid: set a dispatch tunable: " + TUNABLES)

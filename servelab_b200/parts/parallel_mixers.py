@@ -119,6 +119,8 @@ class ParallelMixers(Mixer):
                 self.o_bias = term if self.o_bias is None else self.o_bias + term
             branch.w_in = branch.w_o = None
         self.o_bias_cast = None if self.o_bias is None else self.o_bias.to(self.env.dtype)
+        if self.w_in.is_cuda:
+            _side_stream(self.w_in.device)                 # (made now, not in a capture)
 
     def _branch_cache(self, cache: LayerCache, index: int) -> LayerCache:
         return cache.with_state_slice(sum(self.sizes[:index]), self.sizes[index])

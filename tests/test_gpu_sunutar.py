@@ -744,6 +744,24 @@ def test_single_token_steps_through_replayed_graphs(model, dtype):
     _compare(model, dtype, graphs)
 
 
+def test_branches_on_two_streams_equal_one_stream(model, monkeypatch):
+    """Captured steps run the two branches side by side; bit for bit the results of one stream."""
+    from servelab_b200.parts import parallel_mixers as PM
+    steps = H.trace_mixed(model["requests"], seed=4)
+    from servelab_b200.replay import TraceSession
+    got = []
+    for overlap in (True, False, True):
+        monkeypatch.setattr(PM, "overlap_branches", overlap)
+        sess = TraceSession(model["folder"], "bfloat16", H.peak_tokens(steps), page_size=model["page"], max_live=4,
+                            poison_cache=True, cuda_graphs=True)
+        sess.runner.portion_graph_after = 1
+        got.append(H.collect(steps, H.run_session(sess, steps), model["cfg"]["vocab"]))
+        assert sess.runner.portion_graph_replays > 0
+    for rid in got[0]:
+        for pos in got[0][rid]:
+            assert np.array_equal(got[0][rid][pos], got[1][rid][pos]) and np.array_equal(got[0][rid][pos], got[2][rid][pos])
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_steps_with_portions_through_graphs_captured_for_padded_sizes(model, dtype):
     """Steps with prompt portions replay graphs captured for padded sizes although the model keeps
