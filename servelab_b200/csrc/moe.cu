@@ -46,7 +46,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 
 // One warp a token.  `score_fn` 0: scores = softmax(logits); 1: scores = sigmoid(logits).  The
 // choice runs on choice scores c = score (+ correction[e], a learned offset that enters the choice
-// only); a group's score is the sum of its `group_best` largest choice scores (1: its maximum);
+// only; sigmoids without offset and groups: c = the logit); a group's score is the sum of its `group_best` largest choice scores (1: its maximum);
 // experts outside the `keep` best groups count as minus infinity (choice scores may be negative);
 // the weights are the chosen experts' scores without the offset, divided by their sum + `norm_eps`
 // with `renormalize`, times `route_scale`.  Ties: the lower index.
@@ -82,7 +82,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(
         for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-z[e]));
     }
     __syncwarp();
-    for (int e = lane; e < E; e += 32) c[e] = correction != nullptr ? s[e] + correction[e] : s[e];
+    // (sigmoids alone: the logits give the same order, also where their sigmoids round to the same number)
+    const bool by_logit = score_fn == 1 && correction == nullptr && groups == 1;
+    for (int e = lane; e < E; e += 32) c[e] = by_logit ? z[e] : correction != nullptr ? s[e] + correction[e] : s[e];
     __syncwarp();
     const int per = E / groups;
     if (groups > 1) {

@@ -532,6 +532,7 @@ def test_router_takes_the_largest_sigmoids_and_keeps_them():
     for E, top in ((5, 2), (1, 1), (64, 7), (300, 32), (3, 3)):
         z = torch.randn(77, E, generator=g) * 3
         z[5] = 0.25                                    # ties: the lower index
+        z[6] = torch.randperm(E, generator=g) / 64.0 + 25.0     # sigmoids that round to 1 in float32
         ids, w = K.moe_route_scored(z.to(DEV), 1, 1, top, 1.0, False, "sigmoid")
         wi, ww = plain.route(z.double(), top)
         assert torch.equal(ids.cpu().long(), wi)
